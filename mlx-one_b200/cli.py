@@ -10,7 +10,7 @@ from dataclasses import asdict
 import click
 
 
-@click.group(help="B200-native inference engine (LFM2, Galarax, Farorax, Lamisun and Tirudra models).")
+@click.group(help="B200-native inference engine (LFM2, Galarax, Farorax, Lamisun, Tirudra and Susalorn models).")
 def main() -> None:
     pass
 

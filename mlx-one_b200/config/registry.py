@@ -33,6 +33,7 @@ _BUILTIN = {
     "farorax": "mlx_one_b200.architectures.farorax:ARCHITECTURE",
     "lamisun": "mlx_one_b200.architectures.lamisun:ARCHITECTURE",
     "tirudra": "mlx_one_b200.architectures.tirudra:ARCHITECTURE",
+    "susalorn": "mlx_one_b200.architectures.susalorn:ARCHITECTURE",
 }
 _REGISTERED: dict[str, Architecture] = {}
 

@@ -167,10 +167,11 @@ class Part:
         self.runtime = runtime
         self.ops = runtime.ops
         expected = self.tensors(spec)
+        sizes: dict[str, int] = {}
         for name, want in expected.items():
             if name not in tensors:
                 raise KeyError(f"{type(self).__name__}: tensor {name!r} was not given")
-            if tuple(tensors[name].shape) != tuple(want.shape):
+            if not want.fits(tuple(tensors[name].shape), sizes):
                 raise ValueError(f"{type(self).__name__}: {name} has shape "
                                  f"{tuple(tensors[name].shape)}, expected {want.shape}")
 
@@ -263,6 +264,21 @@ class Embedding(Part):
         raise NotImplementedError
 
 
+class StreamUpdate:
+    """The output of a sublayer that has not been written into parallel streams yet: new stream t
+    is sum_s mix[s, t] X_s + out[t] * output, all from the old streams X. ``mix`` [streams before,
+    streams after] and ``out`` [streams after] are 32-bit."""
+
+    def __init__(self, output: torch.Tensor, mix: torch.Tensor, out: torch.Tensor) -> None:
+        self.output, self.mix, self.out = output, mix, out
+
+    def applied(self, streams: torch.Tensor) -> torch.Tensor:
+        """The streams [tokens, streams after, hidden] after the update, computed plainly (for
+        observers; the engine's kernels never write the update on its own)."""
+        mixed = torch.einsum("nsc,st->ntc", streams.float(), self.mix)
+        return mixed + self.out[:, None] * self.output.float()[:, None, :]
+
+
 class Block(Part):
     """Arranges a layer's parts. Gets the built parts by role."""
 
@@ -282,6 +298,10 @@ class Block(Part):
     # place; the block leaves what the next call reads in kept[place + 2] and returns
     # (that stream, pending output) instead of the pending output alone.
     keeps_streams = False
+    # True: the block works on several parallel streams [tokens, streams, hidden] (one stream, the
+    # embedding's output, ahead of the first block): ``residual`` has that shape, ``delta`` is a
+    # ``StreamUpdate`` or None, and ``forward`` returns (streams, StreamUpdate).
+    parallel_streams = False
 
     @classmethod
     def cache_need(cls, spec: PartSpec):

@@ -2,7 +2,7 @@
 
 from __future__ import annotations
 
-from .base import Block, FixedState
+from .base import Block, FixedState, StreamUpdate
 from .registry import BLOCKS
 from .spec import TensorSpec
 
@@ -165,3 +165,62 @@ class SandwichBlock(Block):
             out = self.feed_forward.forward(normed, ctx)
             self.ops.normed_mean_add(residual, [out], [self.post_feed_forward], self.eps)
         return None
+
+
+@BLOCKS.register("hyper")
+class HyperConnectedBlock(Block):
+    """Hyper-connections: ``streams`` residual streams X_1 .. X_n instead of one, all equal to the
+    embedding's output at the start. A sublayer reads u = sum_s in[s] X_s, and with y =
+    part(norm(u)) every stream is replaced at once: X_t <- sum_s mix[s, t] X_s + out[t] y. The
+    stored ``in1``, ``out1`` [streams] and ``mix1`` [streams, streams] (indexed [from, to]) belong
+    to the mixer, ``in2``, ``out2``, ``mix2`` to the feed-forward. A layer without a feed-forward
+    ends after the mixer. Parameters: ``streams``, ``feed_forward`` (True: the layer has one).
+
+    The streams are 32-bit [tokens, streams, hidden]. One kernel stands between two sublayers: it
+    writes the last one's output into the streams, reads the next one's input from them and norms
+    it, so each stream is read and written once per sublayer. Ahead of the first sublayer there is
+    one stream that stands for all: reading it takes the sum of ``in``, and the first write makes
+    ``streams`` of it with the sums of ``mix``'s columns."""
+
+    parallel_streams = True
+
+    @classmethod
+    def tensors(cls, spec):
+        count = spec["streams"]
+        out = {}
+        for which in ("1", "2") if spec.get("feed_forward", True) else ("1",):
+            out["in" + which] = TensorSpec((count,), "wide")
+            out["out" + which] = TensorSpec((count,), "norm")
+            out["mix" + which] = TensorSpec((count, count), "mix")
+        return out
+
+    def __init__(self, spec, tensors, runtime, **roles):
+        super().__init__(spec, tensors, runtime, **roles)
+        self.streams = int(spec["streams"])
+        if (self.feed_forward is None) == bool(spec.get("feed_forward", True)):
+            raise ValueError("a feed-forward and its connections come together")
+        for norm in (self.mixer_norm, self.feed_forward_norm):
+            if norm is not None and not hasattr(norm, "read_streams"):
+                raise ValueError("this block needs norms that can read parallel streams")
+        # per sublayer: (reading weights, mix, out), for all streams and for the one at the start
+        self.connections = []
+        for which in ("1", "2") if self.feed_forward is not None else ("1",):
+            read, mix = self.vector(tensors["in" + which]), self.vector(tensors["mix" + which])
+            out = self.vector(tensors["out" + which])
+            self.connections.append({
+                self.streams: (read, mix, out),
+                1: (read.sum(0, keepdim=True), mix.sum(0, keepdim=True).contiguous(), out)})
+
+    def _sublayer(self, which, norm, residual, delta, run):
+        before = residual.shape[1] if delta is None else delta.mix.shape[1]
+        read, mix, out = self.connections[which][before]
+        residual, normed = norm.read_streams(residual, delta, read)
+        return residual, StreamUpdate(run(normed), mix, out)
+
+    def forward(self, residual, delta, ctx, cache, write):
+        residual, delta = self._sublayer(0, self.mixer_norm, residual, delta,
+                                         lambda x: self.mixer.forward(x, ctx, cache, write))
+        if self.feed_forward is not None:
+            residual, delta = self._sublayer(1, self.feed_forward_norm, residual, delta,
+                                             lambda x: self.feed_forward.forward(x, ctx))
+        return residual, delta

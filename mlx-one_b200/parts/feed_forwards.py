@@ -93,14 +93,15 @@ class DenseFeedForward(FeedForward):
 
 @FEED_FORWARDS.register("routed")
 class RoutedExperts(FeedForward):
-    """A mixture of gated feed-forwards. Parameters: ``hidden``, ``width`` (of an expert),
-    ``experts``, ``top`` (experts a token uses), ``groups`` and ``keep`` (experts form ``groups``
-    equal runs of neighbours; a group's score is the sum of its ``group_score`` largest scores,
-    and only experts of the ``keep`` best groups can be chosen), ``shared_width`` (None: no
-    shared expert), ``activation`` of the gates, ``scores`` (``sigmoid``, or ``softmax`` over all
-    outputs of the router), ``correction`` (True: the stored ``correction``, one number per
-    output of the router, is added to the scores where experts are chosen, and only there),
-    ``normalize`` (True; False: the chosen experts keep their scores as weights), ``identity``
+    """A mixture of feed-forwards. Parameters: ``hidden``, ``width`` (of an expert),
+    ``gated`` (True; False: an expert is down(act(up x))), ``experts``, ``top`` (experts a token
+    uses), ``groups`` and ``keep`` (experts form ``groups`` equal runs of neighbours; a group's
+    score is the sum of its ``group_score`` largest scores, and only experts of the ``keep`` best
+    groups can be chosen), ``scale`` (1: a factor on the weights), ``shared_width`` (None: no
+    shared expert), ``activation`` (of the gates, or of experts without one), ``scores``
+    (``sigmoid``, or ``softmax`` over all outputs of the router), ``correction`` (True: the
+    stored ``correction``, one number per output of the router, is added to the scores where
+    experts are chosen, and only there), ``normalize`` (True; False: the chosen experts keep their scores as weights), ``identity``
     (0: that many further outputs of the router, behind the experts', stand for experts without
     tensors whose output is the input itself), ``shared_gate`` (True: the shared expert's output
     is multiplied by sigmoid(w x), one number per token, with the stored ``shared.sg`` [1,
@@ -110,8 +111,8 @@ class RoutedExperts(FeedForward):
     with the largest scores are chosen and weighted with s / (sum of the chosen s + 1e-20). The
     output is the weighted sum of the chosen experts' down(act(gate x) * up x), plus the shared
     expert's, which every token uses with weight 1. The options above (softmax scores, a
-    correction, weights that are not normalised, identity outputs, a gated shared expert) go
-    through a second routing kernel that has no groups.
+    correction, a scale, weights that are not normalised, identity outputs, a gated shared
+    expert) go through a second routing kernel.
 
     The experts' gate and up matrices are stacked into one matrix and their down matrices side
     by side into another (the shared expert last). Small steps run every token through all of
@@ -132,8 +133,12 @@ class RoutedExperts(FeedForward):
             if not spec.get("shared_width"):
                 raise ValueError("a gate of the shared expert needs a shared expert")
             out["shared.sg"] = TensorSpec((1, hidden), "wide")
+        gated = spec.get("gated", True)
+        if not gated and spec.get("shared_width"):
+            raise ValueError("a shared expert goes with gated experts")
         for e in range(spec["experts"]):
-            out[f"e{e}.gate"] = TensorSpec((width, hidden))
+            if gated:
+                out[f"e{e}.gate"] = TensorSpec((width, hidden))
             out[f"e{e}.up"] = TensorSpec((width, hidden))
             out[f"e{e}.down"] = TensorSpec((hidden, width))
         if spec.get("shared_width"):
@@ -160,20 +165,28 @@ class RoutedExperts(FeedForward):
             raise ValueError("experts must form equal groups")
         # what the first routing kernel does not know goes to the second one
         self.general = None
+        scale = float(spec.get("scale", 1.0))
         if (scores != "sigmoid" or spec.get("correction") or not normalize or self.identity
-                or self.shared_gate):
-            if self.routing["groups"] != 1:
-                raise ValueError("groups of experts go with sigmoid scores, normalised weights "
-                                 "and no identity outputs")
+                or self.shared_gate or scale != 1.0):
+            if self.routing["groups"] != 1 and (self.identity or spec.get("correction")):
+                raise ValueError("groups of experts go without identity outputs and correction")
             self.general = dict(experts=self.experts, identity=self.identity, top=spec["top"],
                                 scores=scores, normalize=bool(normalize),
                                 shared_gate=self.shared_gate)
+            if self.routing["groups"] != 1:
+                self.general.update({key: self.routing[key] for key in ("groups", "keep", "group_score")})
+            if scale != 1.0:
+                self.general["scale"] = scale
             self.correction = None
             if spec.get("correction"):
                 self.correction = tensors["correction"].to(torch.float32).contiguous()
         names = [f"e{e}." for e in range(self.experts)] + (["shared."] if self.shared_width else [])
-        self.gate_up = self.matrix(torch.cat([tensors[name + "gate"] for name in names] +
-                                             [tensors[name + "up"] for name in names], dim=0))
+        # [gate rows; up rows], or the up rows alone
+        self.gated = bool(spec.get("gated", True))
+        self.gate_up = self.matrix(torch.cat(
+            ([tensors[name + "gate"] for name in names] if self.gated else []) +
+            [tensors[name + "up"] for name in names], dim=0))
+        self.stack = sum(tensors[name + "up"].shape[0] for name in names)
         self.down = self.matrix(torch.cat([tensors[name + "down"] for name in names], dim=1))
         self.router = tensors["router"].to(torch.float32).contiguous()
         if self.shared_gate:
@@ -182,8 +195,10 @@ class RoutedExperts(FeedForward):
                                      .reshape(1, -1)], dim=0).contiguous()
         # the shared expert once more on its own, for steps that sort their tokens by expert
         self.shared = {}
-        self.sortable = (self.activation == "silu" and hasattr(self.ops, "sorts_experts")
+        sorted_kinds = ("silu",) if self.gated else ("relu2",)
+        self.sortable = (self.activation in sorted_kinds and hasattr(self.ops, "sorts_experts")
                          and runtime.dtype == torch.bfloat16)
+        self.sorted_form = {} if self.gated else dict(activation=self.activation)
         if self.sortable and self.shared_width:
             self.shared = dict(
                 shared_gate_up=self.matrix(torch.cat([tensors["shared.gate"], tensors["shared.up"]], dim=0)),
@@ -192,23 +207,30 @@ class RoutedExperts(FeedForward):
     fuses_residual = True
     scales_residual = True
 
+    def _hidden(self, x):
+        """All experts' hidden values [tokens, stack] (the shared expert's last)."""
+        if not self.gated:
+            return self.ops.linear_act(x, self.gate_up, self.activation)
+        if self.activation == "silu":
+            return self.ops.linear_swiglu(x, self.gate_up)
+        return self.ops.linear_gated(x, self.gate_up, self.activation)
+
+    def _sorts(self, x):
+        return self.sortable and self.ops.sorts_experts(
+            x, experts=self.experts, width=self.width, top=self.routing["top"], stack=self.stack)
+
     def _forward_general(self, x, ctx):
         """Routing with the second kernel: weights [tokens, experts] of the experts that have
         tensors, and per token the sum of the chosen identity outputs' weights and the shared
         expert's gate."""
         weights, others = self.ops.route_general(x, self.router, self.correction, **self.general)
         shared_scale = others[1] if self.shared_gate else None
-        if self.sortable and self.ops.sorts_experts(x, experts=self.experts, width=self.width,
-                                                    top=self.routing["top"],
-                                                    stack=self.gate_up.shape[0] // 2):
+        if self._sorts(x):
             out = self.ops.routed_experts_sorted(
                 x, weights, self.gate_up, self.down, experts=self.experts, width=self.width,
-                top=self.routing["top"], shared_scale=shared_scale, **self.shared)
+                top=self.routing["top"], shared_scale=shared_scale, **self.shared, **self.sorted_form)
         else:
-            if self.activation == "silu":
-                gated = self.ops.linear_swiglu(x, self.gate_up)
-            else:
-                gated = self.ops.linear_gated(x, self.gate_up, self.activation)
+            gated = self._hidden(x)
             # (the shared expert's columns, behind the experts', times its gate in the same pass)
             self.ops.scale_expert_columns(gated, weights, self.width, tail=shared_scale)
             out = self.ops.linear(gated, self.down)
@@ -221,16 +243,11 @@ class RoutedExperts(FeedForward):
             out = self._forward_general(x, ctx)
             return out          # (the caller adds it, with its factor, where it norms next)
         weights = self.ops.route_experts(x, self.router, **self.routing)
-        if self.sortable and self.ops.sorts_experts(x, experts=self.experts, width=self.width,
-                                                    top=self.routing["top"],
-                                                    stack=self.gate_up.shape[0] // 2):
+        if self._sorts(x):
             return self.ops.routed_experts_sorted(
                 x, weights, self.gate_up, self.down, experts=self.experts, width=self.width,
-                top=self.routing["top"], **self.shared)
-        if self.activation == "silu":
-            gated = self.ops.linear_swiglu(x, self.gate_up)
-        else:
-            gated = self.ops.linear_gated(x, self.gate_up, self.activation)
+                top=self.routing["top"], **self.shared, **self.sorted_form)
+        gated = self._hidden(x)
         self.ops.scale_expert_columns(gated, weights, self.width)
         if residual is None:
             return self.ops.linear(gated, self.down)

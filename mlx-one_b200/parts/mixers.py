@@ -1,6 +1,6 @@
 """Sequence mixers: grouped-query attention over paged keys and values, the gated short
-convolution with a fixed-size state, the gated delta rule with a matrix state per head,
-several mixers side by side on one input, attention over one latent row per token, and
+convolution with a fixed-size state, the gated delta rule with a matrix state per head (one
+decay per head, or one per key channel), several mixers side by side on one input, attention over one latent row per token, and
 attention with two score maps per head."""
 
 from __future__ import annotations
@@ -9,7 +9,7 @@ import torch
 
 from .base import FixedState, Mixer, PagedKeyValues
 from .registry import MIXERS, NORMS, POSITIONS
-from .spec import PartSpec, TensorSpec
+from .spec import FreeSize, PartSpec, TensorSpec
 
 
 @MIXERS.register("attention")
@@ -387,6 +387,97 @@ class GatedDeltaRule(Mixer):
         return self.ops.linear_add(mixed, self.out, None, residual)
 
 
+@MIXERS.register("channel_delta")
+class ChannelDeltaRule(Mixer):
+    """The gated delta rule with a decay per key channel and an output gate, both through small
+    inner projections. Parameters: ``hidden``, ``heads`` (value heads), ``kv_heads`` (query/key
+    heads; value head h reads query/key head h // (heads / kv_heads)), ``key_dim``,
+    ``value_dim``, ``taps``, ``eps`` (of the output norm), ``decay_rank`` and ``gate_rank`` (inner
+    sizes of the two pairs of projections for random weights; stored tensors bring their own).
+
+    q, k, v, their convolutions with silu, unit lengths and beta are those of ``gated_delta``. The
+    decay is one number per head and key channel, g = exp(-exp(A_log_h) softplus(W_a2 (W_a1 x) +
+    dt_bias)) [heads, key_dim], and multiplies the rows of S: S = g * S; u = beta (v - S^T k);
+    S = S + k u^T; o = S^T q. The output is o / rms(o) (over value_dim, with ``eps``) * norm *
+    sigmoid(W_g2 (W_g1 x)), projected by W_o. Everything after the convolutions' silu and the
+    projections is 32-bit, and W_a2's output is kept in 32-bit. The state slot is that of
+    ``gated_delta``: S of every head and a ring of the convolutions' inputs."""
+
+    UNIT_EPS = 1e-6
+
+    _channels = GatedDeltaRule._channels
+    state_size = GatedDeltaRule.state_size
+    cache_need = GatedDeltaRule.cache_need
+
+    @classmethod
+    def tensors(cls, spec):
+        hidden, heads, taps = spec["hidden"], spec["heads"], spec["taps"]
+        qk, inner = cls._channels(spec)
+        decays = heads * spec["key_dim"]
+        decay_rank = FreeSize("decay_rank", spec.get("decay_rank") or spec["key_dim"])
+        gate_rank = FreeSize("gate_rank", spec.get("gate_rank") or spec["value_dim"])
+        return {
+            "q": TensorSpec((qk, hidden)), "q.conv": TensorSpec((qk, taps), "wide"),
+            "k": TensorSpec((qk, hidden)), "k.conv": TensorSpec((qk, taps), "wide"),
+            "v": TensorSpec((inner, hidden)), "v.conv": TensorSpec((inner, taps), "wide"),
+            "b": TensorSpec((heads, hidden)), "A_log": TensorSpec((heads,), "wide"),
+            "a1": TensorSpec((decay_rank, hidden)), "a2": TensorSpec((decays, decay_rank)),
+            "dt_bias": TensorSpec((decays,), "wide"), "norm": TensorSpec((spec["value_dim"],), "norm"),
+            "g1": TensorSpec((gate_rank, hidden)), "g2": TensorSpec((inner, gate_rank)),
+            "o": TensorSpec((hidden, inner)),
+        }
+
+    def __init__(self, spec, tensors, runtime):
+        super().__init__(spec, tensors, runtime)
+        self.sizes = dict(heads=spec["heads"], kv_heads=spec["kv_heads"], key_dim=spec["key_dim"],
+                          value_dim=spec["value_dim"], taps=spec["taps"])
+        if spec["heads"] % spec["kv_heads"]:
+            raise ValueError("heads must be a multiple of kv_heads")
+        # One product for everything that reads x: q | k | v | beta, the inner rows of the decay,
+        # the inner rows of the gate, each of the three starting on a multiple of 8 rows (rows of
+        # zeros in between), so that a slice of the result can be another product's operand.
+        pieces, at = [], 0
+        starts = []
+        for group in (("q", "k", "v", "b"), ("a1",), ("g1",)):
+            starts.append(at)
+            pieces += [tensors[name] for name in group]
+            rows = sum(tensors[name].shape[0] for name in group)
+            if rows % 8:
+                pieces.append(tensors["q"].new_zeros((-rows % 8, spec["hidden"])))
+            at += rows + -rows % 8
+        self.project = self.matrix(torch.cat(pieces, dim=0))
+        self.decay_columns = (starts[1], starts[1] + tensors["a1"].shape[0])
+        self.gate_columns = (starts[2], starts[2] + tensors["g1"].shape[0])
+        self.decay_up = self.matrix(tensors["a2"])
+        self.gate_up = self.matrix(tensors["g2"])
+        self.conv = self.vector(torch.cat([tensors[name] for name in
+                                           ("q.conv", "k.conv", "v.conv")], dim=0))
+        self.a_log = self.vector(tensors["A_log"])
+        self.dt_bias = self.vector(tensors["dt_bias"])
+        self.norm = self.vector(tensors["norm"])
+        self.out = self.matrix(tensors["o"])
+        self.eps = float(spec["eps"])
+
+    fuses_residual = True
+    accepts_normed_input = True
+
+    def input_projection(self):
+        return self.project, None
+
+    def forward(self, x, ctx, cache, write, residual=None):
+        return self.forward_projected(self.ops.linear(x, self.project), ctx, cache, write, residual)
+
+    def forward_projected(self, projected, ctx, cache, write, residual=None):
+        mixed = self.ops.channel_delta_rule(
+            projected, self.decay_up, self.gate_up, decay_columns=self.decay_columns,
+            gate_columns=self.gate_columns, conv=self.conv, a_log=self.a_log,
+            dt_bias=self.dt_bias, norm_weight=self.norm, eps=self.eps, unit_eps=self.UNIT_EPS,
+            ctx=ctx, view=cache, write=write, **self.sizes)
+        if residual is None:
+            return self.ops.linear(mixed, self.out)
+        return self.ops.linear_add(mixed, self.out, None, residual)
+
+
 @MIXERS.register("lightning")
 class LightningAttention(Mixer):
     """Linear attention with a constant decay per head. Parameters: ``hidden``, ``heads``,
@@ -533,34 +624,47 @@ class ParallelMixers(Mixer):
 class LatentAttention(Mixer):
     """Softmax attention whose keys and values of all heads come from one small latent per
     token. Parameters: ``hidden``, ``heads``, ``head_dim`` (unrotated query/key dimensions of a
-    head), ``rot_dim`` (rotated ones), ``value_dim``, ``latent`` (size of the latent), ``eps`` (of
-    the latent's norm), ``position`` (a position-encoding PartSpec for the rotated part), ``scale``,
-    ``gate`` (a sigmoid gate on the heads' outputs, computed from the mixer's input).
+    head), ``rot_dim`` (rotated ones), ``value_dim``, ``latent`` (size of the latent),
+    ``query_latent`` (None: queries come straight from the mixer's input; else the size of a
+    latent of their own), ``eps`` (of the latents' norms), ``position`` (a position-encoding
+    PartSpec for the rotated part), ``scale``, ``gate`` (a sigmoid gate on the heads' outputs,
+    computed from the mixer's input), ``sink`` (a stored number per head, ``sink`` [heads], that
+    stands in the softmax's denominator as exp(sink): no key, no value, not scaled).
 
-    q = W_q x, head by head [head_dim unrotated | rot_dim rotated]. W_down x has latent + rot_dim
-    rows: the first ``latent``, divided by their root mean square and multiplied by ``down_norm``,
-    are the latent c; the last rot_dim are one rotated key part r that all heads share. Per head
-    h the key is [W_uk,h c | r] and the value W_uv,h c; causal softmax(q k^T scale) v; the heads
-    side by side are multiplied by sigmoid(W_g x) and projected by W_o.
+    q = W_q x, or with a query latent W_uq c_q with c_q = rms_norm(W_dq x) (``query_down``,
+    ``query_norm``, ``query_up``), head by head [head_dim unrotated | rot_dim rotated]. W_down x
+    has latent + rot_dim rows: the first ``latent``, divided by their root mean square and
+    multiplied by ``down_norm``, are the latent c; the last rot_dim are one rotated key part r that
+    all heads share. Per head h the key is [W_uk,h c | r] and the value W_uv,h c; causal
+    softmax(q k^T scale) v; the heads side by side are multiplied by sigmoid(W_g x) (with a gate)
+    and projected by W_o.
 
     Only c and r are kept per token: one row [c | r] in single-plane pages. The up-projections
     move to the query's side: q_h . (W_uk,h c) = (W_uk,h^T q_h) . c, so every head's query becomes
     [W_uk,h^T q_h | rotated part] against the one shared row, the attention's output is the
     weights' average of c, and the head's value is W_uv,h applied to that average. Scores,
-    weights, the norm and the rotation are 32-bit."""
+    weights, the norms and the rotation are 32-bit."""
 
     @classmethod
     def tensors(cls, spec):
         hidden, heads, latent = spec["hidden"], spec["heads"], spec["latent"]
-        inner = heads * spec["value_dim"]
-        out = {"q": TensorSpec((heads * (spec["head_dim"] + spec["rot_dim"]), hidden)),
-               "down": TensorSpec((latent + spec["rot_dim"], hidden)),
-               "down_norm": TensorSpec((latent,), "norm"),
-               "up_k": TensorSpec((heads * spec["head_dim"], latent)),
-               "up_v": TensorSpec((inner, latent)),
-               "out": TensorSpec((hidden, inner))}
+        inner, queries = heads * spec["value_dim"], heads * (spec["head_dim"] + spec["rot_dim"])
+        rank = spec.get("query_latent")
+        if rank:
+            out = {"query_down": TensorSpec((rank, hidden)),
+                   "query_norm": TensorSpec((rank,), "norm"),
+                   "query_up": TensorSpec((queries, rank))}
+        else:
+            out = {"q": TensorSpec((queries, hidden))}
+        out.update({"down": TensorSpec((latent + spec["rot_dim"], hidden)),
+                    "down_norm": TensorSpec((latent,), "norm"),
+                    "up_k": TensorSpec((heads * spec["head_dim"], latent)),
+                    "up_v": TensorSpec((inner, latent)),
+                    "out": TensorSpec((hidden, inner))})
         if spec.get("gate", True):
             out["gate"] = TensorSpec((inner, hidden))
+        if spec.get("sink"):
+            out["sink"] = TensorSpec((heads,), "wide")
         return out
 
     @classmethod
@@ -576,41 +680,68 @@ class LatentAttention(Mixer):
         self.position = POSITIONS.get(position.kind)(position, {}, runtime)
         self.neighbours = getattr(self.position, "layout", "halves") == "neighbours"
         self.gated = bool(spec.get("gate", True))
-        # one product for everything that reads x: q | latent and shared key part | gate
-        names = ["q", "down"] + (["gate"] if self.gated else [])
+        self.query_latent = int(spec.get("query_latent") or 0)
+        # one product for everything that reads x: queries (or their latent) | latent and shared
+        # key part | gate
+        names = ["query_down" if self.query_latent else "q", "down"] + (["gate"] if self.gated else [])
         self.project = self.matrix(torch.cat([tensors[name] for name in names], dim=0))
+        if self.query_latent:
+            self.query_norm = self.vector(tensors["query_norm"])
+            self.query_up = self.matrix(tensors["query_up"])
         self.down_norm = self.vector(tensors["down_norm"])
         # per head: [latent, head_dim] (the key's up-projection, transposed) and [value_dim, latent]
         up_k = tensors["up_k"].view(self.heads, self.head_dim, self.latent)
         self.up_k = self.matrix(up_k.transpose(1, 2))
         self.up_v = self.matrix(tensors["up_v"].view(self.heads, self.value_dim, self.latent))
         self.out = self.matrix(tensors["out"])
+        # what the plain form of the operations does not cover goes to them as extra arguments
+        amplitude = self.position.amplitude()
+        self.turn = {} if amplitude == 1.0 else dict(amplitude=amplitude)
+        self.sinks = dict(sinks=self.vector(tensors["sink"])) if spec.get("sink") else {}
         self.ops.check_attention_sizes(self.heads, 1, self.latent + self.rot_dim)
 
     def inner_parts(self):
         return (self.position,)
 
-    def forward(self, x, ctx, cache, write):
+    def _queries(self, x, ctx, cache, write):
+        """The projection of x and the finished query rows [tokens, heads, latent + rot_dim]; the
+        tokens' rows [c | r] are in their pages afterwards."""
         heads, latent, rot = self.heads, self.latent, self.rot_dim
         projected = self.ops.linear(x, self.project)
         tokens = projected.shape[0]
         queries = torch.empty((tokens, heads, latent + rot), dtype=projected.dtype,
                               device=projected.device)
-        # the latent's norm, the rotation of the shared key part and of the queries' rotated
-        # parts, the row [c | r] appended to the request's pages
-        self.ops.latent_prepare(projected, queries, heads=heads, head_dim=self.head_dim,
-                                rot_dim=rot, latent=latent, norm_weight=self.down_norm,
-                                eps=self.eps, rotary=self.position.rotary_table(),
-                                neighbours=self.neighbours, ctx=ctx, view=cache, write=write)
-        plain = projected[:, :heads * (self.head_dim + rot)].view(tokens, heads, -1)
+        common = dict(rot_dim=rot, latent=latent, rotary=self.position.rotary_table(),
+                      neighbours=self.neighbours, ctx=ctx, **self.turn)
+        if self.query_latent:
+            rank = self.query_latent
+            # the two latents' norms, the row [c | r] appended to the request's pages
+            small = self.ops.latent_rows(projected, rank=rank, query_norm=self.query_norm,
+                                         norm_weight=self.down_norm, eps=self.eps, view=cache,
+                                         write=write, **common)
+            q = self.ops.linear(small, self.query_up)
+            self.ops.latent_queries(q, queries, heads=heads, head_dim=self.head_dim, **common)
+        else:
+            # the latent's norm, the rotation of the shared key part and of the queries' rotated
+            # parts, the row [c | r] appended to the request's pages
+            self.ops.latent_prepare(projected, queries, heads=heads, head_dim=self.head_dim,
+                                    norm_weight=self.down_norm, eps=self.eps, view=cache,
+                                    write=write, **common)
+            q = projected[:, :heads * (self.head_dim + rot)]
+        plain = q.unflatten(1, (heads, -1))
         self.ops.linear_heads(plain[:, :, :self.head_dim], self.up_k, out=queries[:, :, :latent])
+        return projected, queries
+
+    def forward(self, x, ctx, cache, write):
+        heads, latent = self.heads, self.latent
+        projected, queries = self._queries(x, ctx, cache, write)
+        tokens = queries.shape[0]
         mixed = self.ops.latent_attention(queries, heads=heads, latent=latent, scale=self.scale,
-                                          ctx=ctx, view=cache)
+                                          ctx=ctx, view=cache, **self.sinks)
         values = self.ops.linear_heads(mixed[:, :, :latent], self.up_v)
         values = values.view(tokens, heads * self.value_dim)
         if self.gated:
-            gate = projected[:, heads * (self.head_dim + rot) + latent + rot:]
-            values = self.ops.sigmoid_gate(values, gate)
+            values = self.ops.sigmoid_gate(values, projected[:, projected.shape[1] - values.shape[1]:])
         return self.ops.linear(values, self.out)
 
 

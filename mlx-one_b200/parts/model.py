@@ -13,7 +13,8 @@ from .spec import LayerCall, ModelSpec, PartSpec, TensorSpec
 
 def _part_tensors(registry, spec: PartSpec, prefix: str) -> dict[str, TensorSpec]:
     cls = registry.get(spec.kind)
-    return {prefix + spec.stored_name(local): t for local, t in cls.tensors(spec).items()}
+    return {prefix + spec.stored_name(local): t.within(prefix + spec.prefix)
+            for local, t in cls.tensors(spec).items()}
 
 
 def expected_tensors(spec: ModelSpec) -> dict[str, TensorSpec]:
@@ -184,13 +185,20 @@ class Model:
         self.capturable = all(getattr(part, "capturable", True) for part in parts)
         # blocks that read the streams of the calls before them (see Block.keeps_streams)
         self.keeps_streams = any(block.keeps_streams for block in self.layers)
+        # blocks that work on parallel streams (see Block.parallel_streams)
+        self.parallel_streams = any(block.parallel_streams for block in self.layers)
+        if self.parallel_streams and not (
+                all(block.parallel_streams for block in self.layers)
+                and all(call.inject is None for call in self.order)):
+            raise ValueError("parallel streams run through all layers, and nothing is injected into them")
         self.own_caches = [bool(type(block).cache_need(block.spec)) for block in self.layers]
         # For debugging: called as observer(place, residual, delta) after the embedding
         # (place -1) and after every call of a layer (place = its number in the order); the
         # hidden state there is residual + s * delta, s the block's ``pending_scale`` (1 unless the
-        # architecture gives its parts' outputs a factor). It sees the step's own tensors (a step's
-        # rows may be followed by fillers): copy what is to be kept. Steps that are replayed from
-        # a CUDA graph do not call it.
+        # architecture gives its parts' outputs a factor); with parallel streams it is the sum over
+        # the streams of delta.applied(residual) (of ``residual`` while delta is None). It sees
+        # the step's own tensors (a step's rows may be followed by fillers): copy what is to be
+        # kept. Steps that are replayed from a CUDA graph do not call it.
         self.observer = None
 
     def forward(self, ctx: StepContext):
@@ -209,6 +217,8 @@ class Model:
         if kept is not None:
             # the first call works on a copy: the embedding's output is read again later
             residual = self.ops.stream_average(kept, None, 1, kept[1])
+        if self.parallel_streams:
+            residual = residual.unsqueeze(1)            # one stream as yet: they are all equal
         delta, scale = None, 1.0
         if self.observer is not None:
             self.observer(-1, residual, delta)
@@ -233,7 +243,10 @@ class Model:
             block = self.layers[call.layer]
             if self.own_caches[call.layer]:
                 extra["own_cache"] = block_view_of(ctx.views, call.cache)
-            if block.keeps_streams:
+            if block.parallel_streams:
+                residual, delta = block.forward(
+                    residual, delta, ctx, view_of(ctx.views, call.cache), call.writes_cache, **extra)
+            elif block.keeps_streams:
                 residual, delta = block.forward(
                     residual, delta, ctx, view_of(ctx.views, call.cache), call.writes_cache,
                     streams=(kept, place), **extra)
@@ -251,7 +264,10 @@ class Model:
     def logits(self, residual, delta, rows: torch.Tensor | None) -> torch.Tensor:
         """32-bit logits [len(rows), vocab] at the token rows ``rows`` (int32, device); None:
         at every row, in order (a step of single tokens that all want theirs: nothing to pick)."""
-        if rows is None:
+        if self.parallel_streams:
+            # the wanted rows' streams, with what is pending, added up
+            picked, picked_delta = self.ops.sum_streams(residual, delta, rows), None
+        elif rows is None:
             picked, picked_delta = residual, delta
         else:
             picked, picked_delta = self.ops.gather_rows(residual, delta, rows)

@@ -36,6 +36,13 @@ class RMSNorm(Norm):
         return self.ops.add_rmsnorm(residual, delta, self.weight, self.eps, self.runtime.dtype,
                                     delta_scale=delta_scale)
 
+    def read_streams(self, streams, update, read):
+        """From parallel streams [tokens, n, hidden]: applies the pending ``update`` (a
+        StreamUpdate or None) and norms u = sum_s read[s] X_s. Returns (the streams after the
+        update, the normed u in the compute dtype)."""
+        return self.ops.read_streams(streams, update, read, self.weight, self.eps,
+                                     self.runtime.dtype)
+
     def add_normed(self, residual, x):
         """In place: residual += x * rsqrt(mean(x^2) + eps) * weight, the norm taken over a part's
         output ``x`` (compute dtype) and everything in 32-bit."""

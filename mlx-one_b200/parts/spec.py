@@ -32,14 +32,48 @@ class PartSpec:
         return self.prefix + self.names.get(local, local)
 
 
+class FreeSize(int):
+    """A size that the stored tensor decides (an inner size that config.json does not give).
+    ``name`` ties sizes together: within a layer's part every dimension with that name has the
+    same size. The number itself is what the random-weights mode uses."""
+
+    def __new__(cls, name: str, default: int):
+        size = super().__new__(cls, default)
+        size.name = name
+        return size
+
+    def within(self, prefix: str) -> "FreeSize":
+        return FreeSize(prefix + self.name, int(self))
+
+
 @dataclass(frozen=True)
 class TensorSpec:
     """Shape of a stored tensor and how the random-weights mode fills it:
     ``normal`` ~ N(0, std), ``norm`` ~ 1 + N(0, 0.1), ``bias`` ~ N(0, std), ``norm0`` ~
-    N(0, 0.1) (a norm weight stored around zero), ``wide`` ~ N(0, 0.5)."""
+    N(0, 0.1) (a norm weight stored around zero), ``wide`` ~ N(0, 0.5), ``mix`` (a square matrix
+    near the identity) ~ 1 + N(0, 0.1) on the diagonal and N(0, 0.1) beside it."""
 
     shape: tuple[int, ...]
     init: str = "normal"
+
+    def within(self, prefix: str) -> "TensorSpec":
+        """The same with its free sizes' names made unique to the part stored under ``prefix``."""
+        if not any(isinstance(size, FreeSize) for size in self.shape):
+            return self
+        return TensorSpec(tuple(size.within(prefix) if isinstance(size, FreeSize) else size
+                                for size in self.shape), self.init)
+
+    def fits(self, shape, sizes: dict[str, int]) -> bool:
+        """Whether a stored tensor of ``shape`` is what is wanted. ``sizes`` keeps the free sizes
+        met so far, by name."""
+        if len(shape) != len(self.shape):
+            return False
+        for got, want in zip(shape, self.shape):
+            if isinstance(want, FreeSize):
+                want = sizes.setdefault(want.name, int(got)) if got > 0 else -1
+            if got != want:
+                return False
+        return True
 
 
 @dataclass(frozen=True)

@@ -75,9 +75,11 @@ def check_names(spec: ModelSpec, stored: Mapping[str, tuple[int, ...]]):
         shapes[new_name] = shape
     missing = sorted(set(expected) - set(bound))
     unexpected = sorted(set(bound) - set(expected))
-    mismatched = sorted((name, shapes[name], tuple(expected[name].shape))
-                        for name in set(bound) & set(expected)
-                        if shapes[name] != tuple(expected[name].shape))
+    sizes: dict[str, int] = {}          # sizes that the stored tensors decide, by name
+    mismatched = sorted((name, shapes[name], tuple(sizes.get(getattr(size, "name", None), size)
+                                                   for size in want.shape))
+                        for name, want in expected.items()
+                        if name in bound and not want.fits(shapes[name], sizes))
     if missing or unexpected or mismatched or duplicates:
         raise WeightError(missing, unexpected, mismatched, sorted(duplicates))
     return bound

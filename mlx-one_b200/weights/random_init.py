@@ -4,7 +4,8 @@ Every tensor is drawn in 32-bit on the host from a generator seeded by (seed, te
 name), so the same folder comes out on every machine and for every order of tensors:
 matrices, tables, convolution kernels and biases ~ N(0, std); norm weights ~ 1 + N(0, 0.1)
 (``norm0``, a weight stored around zero: N(0, 0.1); ``wide``, small per-channel kernels and
-per-head constants that should differ visibly: N(0, 0.5)).
+per-head constants that should differ visibly: N(0, 0.5); ``mix``, a square matrix near the
+identity: the identity + N(0, 0.1)).
 """
 
 from __future__ import annotations
@@ -48,6 +49,8 @@ def random_tensors(spec, seed: int, dtype: torch.dtype = torch.bfloat16, device=
             values = 0.1 * values
         elif want.init == "wide":
             values = 0.5 * values
+        elif want.init == "mix":
+            values = torch.eye(want.shape[0], dtype=torch.float32, device=device) + 0.1 * values
         else:
             values = spec.init_std * values
         out[name] = values.to(dtype)

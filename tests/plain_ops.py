@@ -296,46 +296,67 @@ class PlainOps:
 
     # ---- attention over one latent row per token
 
-    def latent_prepare(self, projected, queries, *, heads, head_dim, rot_dim, latent, norm_weight,
-                       eps, rotary, neighbours, ctx, view, write):
-        tokens = projected.shape[0]
-        flat = projected.float()
-        per_head = head_dim + rot_dim
-        q_rot = flat[:, :heads * per_head].view(tokens, heads, per_head)[:, :, head_dim:]
-        down = flat[:, heads * per_head:heads * per_head + latent + rot_dim]
-        c = down[:, :latent]
-        c = c * torch.rsqrt(c.pow(2).mean(dim=-1, keepdim=True) + eps) * norm_weight
-        shared = down[:, latent:]
+    @staticmethod
+    def _rotated(x, rotary, neighbours, ctx, amplitude):
+        """x [tokens, (heads,) values]: its first dims values turned by position * frequency."""
+        if rotary is None:
+            return x
+        inv_freq, dims = rotary
+        angles = ctx.positions.float()[:, None] * inv_freq[None, :]
+        cos, sin = torch.cos(angles) * amplitude, torch.sin(angles) * amplitude
+        if x.dim() == 3:
+            cos, sin = cos[:, None, :], sin[:, None, :]
+        out = x.clone()
+        if neighbours:
+            a, b = x[..., 0:dims:2], x[..., 1:dims:2]
+            out[..., 0:dims:2] = a * cos - b * sin
+            out[..., 1:dims:2] = b * cos + a * sin
+        else:
+            half = dims // 2
+            a, b = x[..., :half], x[..., half:dims]
+            out[..., :half] = a * cos - b * sin
+            out[..., half:dims] = b * cos + a * sin
+        return out
 
-        def rotate(x):
-            if rotary is None:
-                return x
-            inv_freq, dims = rotary
-            angles = ctx.positions.float()[:, None] * inv_freq[None, :]
-            cos, sin = torch.cos(angles), torch.sin(angles)
-            if x.dim() == 3:
-                cos, sin = cos[:, None, :], sin[:, None, :]
-            out = x.clone()
-            if neighbours:
-                a, b = x[..., 0:dims:2], x[..., 1:dims:2]
-                out[..., 0:dims:2] = a * cos - b * sin
-                out[..., 1:dims:2] = b * cos + a * sin
-            else:
-                half = dims // 2
-                a, b = x[..., :half], x[..., half:dims]
-                out[..., :half] = a * cos - b * sin
-                out[..., half:dims] = b * cos + a * sin
-            return out
+    @staticmethod
+    def _normed(x, weight, eps):
+        return x * torch.rsqrt(x.pow(2).mean(dim=-1, keepdim=True) + eps) * weight
 
-        queries[:, :, latent:] = rotate(q_rot).to(queries.dtype)
-        row = torch.cat((c, rotate(shared)), dim=1).to(view.kv.dtype)
+    def _store_latent(self, down, *, latent, norm_weight, eps, rotary, neighbours, amplitude, ctx,
+                      view, write):
+        c = self._normed(down[:, :latent], norm_weight, eps)
+        shared = self._rotated(down[:, latent:], rotary, neighbours, ctx, amplitude)
+        row = torch.cat((c, shared), dim=1).to(view.kv.dtype)
         if write:
             positions, requests = ctx.positions.tolist(), ctx.token_request.tolist()
             table = view.block_table.tolist()
-            for t in range(tokens):
+            for t in range(row.shape[0]):
                 page = table[requests[t]][positions[t] // view.page_size]
                 assert page >= 0, "a row is written to a position without a page"
                 view.kv[0, page, 0, positions[t] % view.page_size] = row[t]
+
+    def latent_prepare(self, projected, queries, *, heads, head_dim, rot_dim, latent, norm_weight,
+                       eps, rotary, neighbours, ctx, view, write, amplitude=1.0):
+        width = heads * (head_dim + rot_dim)
+        self.latent_queries(projected[:, :width], queries, heads=heads, head_dim=head_dim,
+                            rot_dim=rot_dim, latent=latent, rotary=rotary, neighbours=neighbours,
+                            ctx=ctx, amplitude=amplitude)
+        self._store_latent(projected.float()[:, width:width + latent + rot_dim], latent=latent,
+                           norm_weight=norm_weight, eps=eps, rotary=rotary, neighbours=neighbours,
+                           amplitude=amplitude, ctx=ctx, view=view, write=write)
+
+    def latent_queries(self, q, queries, *, heads, head_dim, rot_dim, latent, rotary, neighbours,
+                       ctx, amplitude=1.0):
+        parts = q.float().reshape(q.shape[0], heads, head_dim + rot_dim)[:, :, head_dim:]
+        queries[:, :, latent:] = self._rotated(parts, rotary, neighbours, ctx, amplitude).to(queries.dtype)
+
+    def latent_rows(self, projected, *, rank, query_norm, norm_weight, eps, rot_dim, latent, rotary,
+                    neighbours, ctx, view, write, amplitude=1.0):
+        flat = projected.float()
+        self._store_latent(flat[:, rank:rank + latent + rot_dim], latent=latent,
+                           norm_weight=norm_weight, eps=eps, rotary=rotary, neighbours=neighbours,
+                           amplitude=amplitude, ctx=ctx, view=view, write=write)
+        return self._normed(flat[:, :rank], query_norm, eps).to(projected.dtype)
 
     def linear_heads(self, a, w, out=None):
         """a [tokens, heads, K] (rows may be slices) with w [heads, N, K] -> [tokens, heads, N]."""
@@ -345,10 +366,10 @@ class PlainOps:
         out.copy_(result)
         return out
 
-    def latent_attention(self, queries, *, heads, latent, scale, ctx, view):
+    def latent_attention(self, queries, *, heads, latent, scale, ctx, view, sinks=None):
         tokens, _, row = queries.shape
         flat = self.paged_attention(queries, heads=heads, kv_heads=1, head_dim=row, scale=scale,
-                                    window=None, ctx=ctx, view=view)
+                                    window=None, ctx=ctx, view=view, sinks=sinks)
         return flat.view(tokens, heads, row)
 
     def sigmoid_gate(self, values, gate):
@@ -367,6 +388,61 @@ class PlainOps:
             x = out.float()
             total += x * torch.rsqrt(x.pow(2).mean(dim=-1, keepdim=True) + eps) * weight
         residual += total / len(outputs)
+
+    # ---- parallel streams
+
+    def read_streams(self, streams, update, read, weight, eps, dtype):
+        if update is not None:
+            streams = update.applied(streams)
+        u = torch.einsum("nsc,s->nc", streams, read)
+        return streams, self._normed(u, weight, eps).to(dtype)
+
+    def sum_streams(self, streams, update, rows):
+        total = (streams if update is None else update.applied(streams)).sum(dim=1)
+        return total if rows is None else total[rows.long()].clone()
+
+    def channel_delta_rule(self, projected, decay_up, gate_up, *, decay_columns, gate_columns, conv,
+                           a_log, dt_bias, norm_weight, eps, unit_eps, ctx, view, write, heads,
+                           kv_heads, key_dim, value_dim, taps):
+        tokens = projected.shape[0]
+        qk, inner = kv_heads * key_dim, heads * value_dim
+        channels, matrices = 2 * qk + inner, heads * key_dim * value_dim
+        flat = projected.float()
+        beta = torch.sigmoid(flat[:, channels:channels + heads])
+        step = flat[:, slice(*decay_columns)] @ decay_up.float().T + dt_bias
+        step = torch.nn.functional.softplus(step, threshold=30.0).view(tokens, heads, key_dim)
+        decay = torch.exp(-torch.exp(a_log)[None, :, None] * step)
+        gate = (flat[:, slice(*gate_columns)] @ gate_up.float().T).to(projected.dtype).float()
+        out = torch.empty(tokens, heads, value_dim)
+        starts, history, slots = ctx.request_start.tolist(), ctx.history.tolist(), view.slots.tolist()
+        unit = lambda x: x / torch.sqrt(x.pow(2).sum(dim=-1, keepdim=True) + unit_eps)
+        share = heads // kv_heads
+        for r in range(ctx.requests):
+            first, last = starts[r], starts[r + 1]
+            n = last - first
+            slot = view.state[slots[r]]
+            state = slot[:matrices].view(heads, key_dim, value_dim).clone()
+            ring = slot[matrices:].view(taps, channels)
+            tail = [ring[p % taps].clone() if p >= 0 else torch.zeros(channels)
+                    for p in range(history[r] - taps + 1, history[r])]
+            padded = torch.cat(([torch.stack(tail)] if tail else []) + [flat[first:last, :channels]])
+            mixed = sum(padded[j:j + n] * conv[:, j] for j in range(taps))
+            mixed = mixed / (1 + torch.exp(-mixed))
+            q = unit(mixed[:, :qk].view(n, kv_heads, key_dim)) * key_dim ** -0.5
+            k = unit(mixed[:, qk:2 * qk].view(n, kv_heads, key_dim))
+            q, k = q.repeat_interleave(share, 1), k.repeat_interleave(share, 1)
+            v = mixed[:, 2 * qk:].view(n, heads, value_dim)
+            for t in range(n):
+                state = decay[first + t][:, :, None] * state
+                u = beta[first + t][:, None] * (v[t] - torch.einsum("hdv,hd->hv", state, k[t]))
+                state = state + k[t][:, :, None] * u[:, None, :]
+                out[first + t] = torch.einsum("hdv,hd->hv", state, q[t])
+            if write:
+                slot[:matrices] = state.reshape(-1)
+                for index in range(max(n - taps, 0), n):
+                    ring[(history[r] + index) % taps] = flat[first + index, :channels]
+        out = self._normed(out, norm_weight, eps).reshape(tokens, inner) * torch.sigmoid(gate)
+        return out.to(projected.dtype)
 
     def gated_delta_rule(self, projected, *, conv, a_log, dt_bias, norm_weight, eps, unit_eps, ctx,
                          view, write, heads, kv_heads, key_dim, value_dim, taps):
@@ -514,7 +590,7 @@ class PlainOps:
         return (v.reshape(tokens, inner) * weight).to(dtype)
 
     def route_general(self, x, router, correction, *, experts, identity, top, scores, normalize,
-                      shared_gate):
+                      shared_gate, groups=1, keep=1, group_score=1, scale=1.0):
         logits = x.float() @ router.T
         outputs = experts + identity
         z = logits[:, :outputs]
@@ -522,11 +598,16 @@ class PlainOps:
         choice = s if correction is None else s + correction
         tokens = s.shape[0]
         weights = torch.zeros(tokens, outputs)
+        per = outputs // groups
         for t in range(tokens):
-            chosen = sorted(range(outputs), key=lambda e: (-float(choice[t, e]), e))[:top]
+            row = choice[t]
+            best = sorted(range(groups), key=lambda g: (
+                -float(row[g * per:(g + 1) * per].topk(min(group_score, per)).values.sum()), g))[:keep]
+            allowed = range(outputs) if groups == 1 else [e for e in range(outputs) if e // per in best]
+            chosen = sorted(allowed, key=lambda e: (-float(choice[t, e]), e))[:top]
             total = sum(float(s[t, e]) for e in chosen) + 1e-20 if normalize else 1.0
             for e in chosen:
-                weights[t, e] = float(s[t, e]) / total
+                weights[t, e] = float(s[t, e]) / total * scale
         others = torch.zeros(2, tokens)
         others[0] = weights[:, experts:].sum(dim=-1)
         if shared_gate:
