@@ -139,6 +139,16 @@ __device__ __forceinline__ void griddep_launch() {
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
 }
 
+// `p`, to be read only after griddep_wait(). What a kernel reads through a `const __restrict__`
+// parameter the compiler may take for unchanging while the kernel runs, and ask for it ahead of
+// the wait, although the kernel before this one has not written it yet; a pointer that comes out
+// of this call, made after the wait, has no such promise.
+template <typename T>
+__device__ __forceinline__ T* settled(T* p) {
+    asm volatile("" : "+l"(p)::"memory");
+    return p;
+}
+
 // Whether launches of the decode path ask for programmatic serialization (mlxone_set_pdl).
 bool mlxone_pdl_enabled();
 

@@ -63,6 +63,7 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ residual, const T* __rest
     __shared__ float scratch[33];
     griddep_launch();
     griddep_wait();
+    delta = settled(delta);
     const size_t base = (size_t)blockIdx.x * hidden;
     float sum = 0.f;
     for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
@@ -126,6 +127,7 @@ __global__ void add_rmsnorm_rows_kernel(float* __restrict__ residual, const T* _
         if (c < hidden) Vec4<float>::load(weight + c, scale[pass]);
     }
     griddep_wait();
+    delta = settled(delta);
     const size_t base = (size_t)blockIdx.x * hidden;
     float values[PASSES][4];
     float sum = 0.f;
@@ -170,6 +172,7 @@ add_rmsnorm_warp_kernel(float* __restrict__ residual, const T* __restrict__ delt
                         int hidden, float eps, float delta_scale) {
     griddep_launch();
     griddep_wait();
+    delta = settled(delta);
     const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     const int lane = threadIdx.x & 31;
     if (row >= rows) return;

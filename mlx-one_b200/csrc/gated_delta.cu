@@ -31,7 +31,7 @@
 // matrix is asked for before the wait for the projection, the convolutions, norms and gates of
 // its own channels are worked out in the block, the recurrence takes one pass, and the output's
 // norm and gate follow after a reduction over the block.
-#include "common.cuh"
+#include "delta_common.cuh"
 
 namespace {
 
@@ -41,44 +41,9 @@ constexpr int CHUNK = 16;            // tokens whose operands are staged in shar
 constexpr int STEP_LANES = 4;        // single-token kernel: lanes that share a column of S
 constexpr int STEP_MAX_COLUMNS = 128;
 
-__device__ __forceinline__ float silu(float z) { return z / (1.f + expf(-z)); }
-__device__ __forceinline__ float softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
-
-__device__ __forceinline__ void copy_async_4(float* dst, const float* src) {
-    const uint32_t to = (uint32_t)__cvta_generic_to_shared(dst);
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(to), "l"(src) : "memory");
-}
-__device__ __forceinline__ void copy_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-__device__ __forceinline__ void copy_async_16(float* dst, const float* src) {
-    const uint32_t to = (uint32_t)__cvta_generic_to_shared(dst);
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(to), "l"(src) : "memory");
-}
-template <int N>
-__device__ __forceinline__ void copy_wait_for() {
-    asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
-}
-
-struct DeltaSizes {
-    int heads, kv_heads, key_dim, value_dim, taps;
-    __host__ __device__ int qk() const { return kv_heads * key_dim; }
-    __host__ __device__ int inner() const { return heads * value_dim; }
-    __host__ __device__ int channels() const { return 2 * qk() + inner(); }
-    __host__ __device__ int width() const { return channels() + inner() + 2 * heads; }
-    __host__ __device__ long long matrices() const { return (long long)heads * key_dim * value_dim; }
-    __host__ __device__ long long state() const {
-        return matrices() + (long long)taps * channels();
-    }
-};
-
-// The input of channel c at `position` - back, for a token at place `index` of its portion:
-// a row of this step, the ring, or zero before the request's start.
-template <typename T>
-__device__ __forceinline__ float conv_input(const T* projected, int ld, const float* ring,
-                                            int channels, int taps, int t, int index, int position,
-                                            int back, int c) {
-    if (index - back >= 0) return to_float<T>(projected[(size_t)(t - back) * ld + c]);
-    if (position - back >= 0) return ring[(size_t)((position - back) % taps) * channels + c];
-    return 0.f;
+// values of a token's row of the projection
+int gated_width(const DeltaSizes& sizes) {
+    return sizes.channels() + sizes.inner() + 2 * sizes.heads;
 }
 
 // ------------------------------------------------------------------ prepare
@@ -642,8 +607,8 @@ MLXONE_API int mlxone_gated_delta(const void* projected, const float* conv, cons
     MLXONE_REQUIRE(value_dim >= 1 && taps >= 1, "gated delta rule: bad value size or taps");
     MLXONE_REQUIRE(requests <= 65535 && heads < 65535, "gated delta rule: too many requests or heads");
     const DeltaSizes sizes = {heads, kv_heads, key_dim, value_dim, taps};
-    MLXONE_REQUIRE(ld >= sizes.width(), "gated delta rule: rows %d apart are shorter than %d", ld,
-                   sizes.width());
+    MLXONE_REQUIRE(ld >= gated_width(sizes), "gated delta rule: rows %d apart are shorter than %d", ld,
+                   gated_width(sizes));
     if (dtype == MLXONE_BF16)
         return launch_delta<__nv_bfloat16>(projected, conv, a_log, dt_bias, norm_weight, eps,
                                            unit_eps, state, slots, token_request, request_start,

@@ -34,7 +34,11 @@ constexpr int THREADS = 192;           // producer warp, mma warp, four epilogue
 constexpr int WAIT_LIMIT = 1 << 24;    // polls before a wait gives up
 constexpr int ERROR_WAIT = 9;
 
-enum : int { STORE_BF16 = 0, SWIGLU = 1, ADD_RESIDUAL = 2, STORE_F32 = 3 };
+// (STORE_RELU2: the square of max(z, 0), stored in bfloat16; grouped products only)
+enum : int { STORE_BF16 = 0, SWIGLU = 1, ADD_RESIDUAL = 2, STORE_F32 = 3, STORE_RELU2 = 4 };
+__host__ __device__ constexpr bool stores_bf16(int epilogue) {
+    return epilogue == STORE_BF16 || epilogue == SWIGLU || epilogue == STORE_RELU2;
+}
 
 __device__ __forceinline__ uint32_t shared_address(const void* p) {
     return static_cast<uint32_t>(__cvta_generic_to_shared(p));
@@ -256,7 +260,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a,
         const int limit = out_limit;
         // whether every row of the output starts on a 16-byte boundary
         const bool whole_rows =
-            (EPILOGUE == STORE_BF16 || EPILOGUE == SWIGLU)
+            stores_bf16(EPILOGUE)
                 ? (ldo % 8 == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0)
                 : (ldo % 4 == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0);
         int round = 0;
@@ -290,6 +294,13 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a,
                     for (int i = 0; i < 32; ++i)
                         if (tile_n + c0 + i < n) value[i] += bias[tile_n + c0 + i];
                 }
+                if (EPILOGUE == STORE_RELU2) {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) {
+                        const float positive = fmaxf(value[i], 0.f);
+                        value[i] = positive * positive;
+                    }
+                }
                 if (c0 + 32 >= OUT_COLUMNS) {
                     // the last piece has left tensor memory: the buffer may be overwritten
                     fence_before_sync();
@@ -306,7 +317,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a,
                     // quarter as many of them as with one value per access.
                     if (row < m) {
                         const size_t at = (size_t)row * ldo + column0;
-                        if (EPILOGUE == STORE_BF16 || EPILOGUE == SWIGLU) {
+                        if (stores_bf16(EPILOGUE)) {
                             uint4* dst = reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(out) + at);
 #pragma unroll
                             for (int piece = 0; piece < 4; ++piece) {
@@ -350,7 +361,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a,
                 const int rows = min(32, m - row0);
                 if (column < limit && rows > 0) {
                     const size_t at = (size_t)row0 * ldo + column;
-                    if (EPILOGUE == STORE_BF16 || EPILOGUE == SWIGLU) {
+                    if (stores_bf16(EPILOGUE)) {
                         bf16* dst = reinterpret_cast<bf16*>(out) + at;
 #pragma unroll 8
                         for (int r = 0; r < rows; ++r)
@@ -519,7 +530,8 @@ MLXONE_API int mlxone_gemm_tcgen05(const void* a, int lda, const void* w, const 
 // tile the first row and the first column of its group's matrix inside the stacked w
 // [w_rows, w_columns] (row stride w_ld), or -1 for a tile without rows. epilogue 0: out bf16
 // [m, n] = a_tile w_group^T with w_group [n, k]; epilogue 1 (SwiGLU): w_group's n gate rows start
-// at the tile's row, its up rows `up_offset` rows further, out bf16 [m, n].
+// at the tile's row, its up rows `up_offset` rows further, out bf16 [m, n]; epilogue 4: as 0, the
+// square of max(z, 0) of every value z.
 MLXONE_API int mlxone_gemm_tcgen05_grouped(const void* a, int lda, const void* w, long long w_rows,
                                            long long w_columns, long long w_ld, void* out, int ldo,
                                            int m, int n, int k, int up_offset, int epilogue,
@@ -534,7 +546,7 @@ MLXONE_API int mlxone_gemm_tcgen05_grouped(const void* a, int lda, const void* w
     MLXONE_REQUIRE((reinterpret_cast<uintptr_t>(a) & 15) == 0 &&
                        (reinterpret_cast<uintptr_t>(w) & 15) == 0 && groups != nullptr,
                    "gemm_tcgen05_grouped: operands must be 16-byte aligned");
-    MLXONE_REQUIRE(epilogue == STORE_BF16 || epilogue == SWIGLU,
+    MLXONE_REQUIRE(stores_bf16(epilogue),
                    "gemm_tcgen05_grouped: epilogue %d is not built", epilogue);
     Grouping grouping;
     grouping.groups = reinterpret_cast<const int2*>(groups);
@@ -544,6 +556,11 @@ MLXONE_API int mlxone_gemm_tcgen05_grouped(const void* a, int lda, const void* w
     if (epilogue == SWIGLU)
         code = launch<256, SWIGLU, WIDE_STAGES>(a, lda, w, nullptr, out, ldo, m, n, k, up_offset,
                                                 error_flag, stream, grouping);
+    else if (epilogue == STORE_RELU2)
+        code = n > 128 ? launch<256, STORE_RELU2, WIDE_STAGES>(a, lda, w, nullptr, out, ldo, m, n, k, 0,
+                                                               error_flag, stream, grouping)
+                       : launch<128, STORE_RELU2, NARROW_STAGES>(a, lda, w, nullptr, out, ldo, m, n,
+                                                                 k, 0, error_flag, stream, grouping);
     else if (n > 128)
         code = launch<256, STORE_BF16, WIDE_STAGES>(a, lda, w, nullptr, out, ldo, m, n, k, 0,
                                                     error_flag, stream, grouping);

@@ -2,26 +2,34 @@
 // steps around the attention kernels.
 //
 // latent_prepare: from the fused input product of a latent-attention mixer to the queries'
-// rotated parts and the token's row [latent | rotated shared key part] in its request's pages.
+// rotated parts and the token's row [latent | rotated shared key part] in its request's pages;
+// also in two steps, for queries that come out of a latent of their own (latent_rows: the page's
+// row and the queries' latent, normed; latent_queries: the rotated parts).
 // sigmoid_gate: values * sigmoid(gate). differential_combine: o = a1 - mix * a2 per head, divided
 // by its root mean square, times a factor.
 #include "common.cuh"
 
 namespace {
 
-// One block per token. `projected` holds, per token, heads * (head_dim + rot_dim) query values
-// (head by head, the rotated part last), then latent + rot_dim values of the down product, then
-// whatever else the mixer projected. queries [tokens, heads, latent + rot_dim]: only the last
-// rot_dim values of every head are written here (the first `latent` are another product's
-// output). The page row [latent + rot_dim] gets the latent divided by its root mean square
+// One block per token; every source has rows of its own stride. q_source (null: this part is left
+// out): heads * (head_dim + rot_dim) query values, head by head, the rotated part last; queries
+// [tokens, heads, latent + rot_dim]: only the last rot_dim values of every head are written here
+// (the first `latent` are another product's output). small_source (null: left out): `rank` values,
+// of which small [tokens, rank] gets the normed ones (times small_weight). down_source (null: left
+// out): latent + rot_dim values of the down product. The page row [latent + rot_dim] gets the latent divided by its root mean square
 // times `norm_weight`, and the rotated shared key part. Rotation: the first `rotary_dim` values
-// of a rotated part; pair i is (2i, 2i + 1) if `neighbours`, else (i, i + rotary_dim / 2).
+// of a rotated part; pair i is (2i, 2i + 1) if `neighbours`, else (i, i + rotary_dim / 2); cosine
+// and sine are multiplied by `amplitude`.
 // Dynamic shared memory: rotary_dim floats (cosines and sines).
 template <typename T>
 __global__ void __launch_bounds__(512)
-latent_prepare_kernel(const T* __restrict__ projected, int ld, T* __restrict__ queries,
+latent_prepare_kernel(const T* __restrict__ q_source, int ld_q, T* __restrict__ queries,
+                      const T* __restrict__ small_source, int ld_small,
+                      const float* __restrict__ small_weight, T* __restrict__ small, int rank,
+                      const T* __restrict__ down_source, int ld_down,
                       const float* __restrict__ norm_weight, float eps,
-                      const float* __restrict__ inv_freq, int rotary_dim, int neighbours,
+                      const float* __restrict__ inv_freq, int rotary_dim, float amplitude,
+                      int neighbours,
                       const int* __restrict__ positions, const int* __restrict__ token_request,
                       T* __restrict__ pages, const int* __restrict__ block_table, int table_width,
                       int page_size, int heads, int head_dim, int rot_dim, int latent, int write,
@@ -30,6 +38,9 @@ latent_prepare_kernel(const T* __restrict__ projected, int ld, T* __restrict__ q
     __shared__ float scratch[33];
     griddep_launch();
     griddep_wait();
+    q_source = settled(q_source);
+    small_source = settled(small_source);
+    down_source = settled(down_source);
     const int t = blockIdx.x;
     const int position = positions[t];
     const int half = rotary_dim / 2;
@@ -38,13 +49,12 @@ latent_prepare_kernel(const T* __restrict__ projected, int ld, T* __restrict__ q
     for (int j = threadIdx.x; j < half; j += blockDim.x) {
         float sine, cosine;
         sincosf((float)position * inv_freq[j], &sine, &cosine);
-        sines[j] = sine;
-        cosines[j] = cosine;
+        sines[j] = sine * amplitude;
+        cosines[j] = cosine * amplitude;
     }
     __syncthreads();
     const int per_head = head_dim + rot_dim;
     const int row = latent + rot_dim;
-    const T* source = projected + (size_t)t * ld;
     // value e of a rotated part that starts at `part`
     auto rotated = [&](const T* part, int e) -> float {
         const float v = to_float<T>(part[e]);
@@ -60,13 +70,28 @@ latent_prepare_kernel(const T* __restrict__ projected, int ld, T* __restrict__ q
         // (u, v) -> (u cos - v sin, v cos + u sin)
         return first ? v * cosines[pair] - w * sines[pair] : v * cosines[pair] + w * sines[pair];
     };
+    if (q_source != nullptr) {
+        const T* source = q_source + (size_t)t * ld_q;
 #pragma unroll 4
-    for (int i = threadIdx.x; i < heads * rot_dim; i += blockDim.x) {
-        const int head = i / rot_dim, e = i % rot_dim;
-        queries[((size_t)t * heads + head) * row + latent + e] =
-            from_float<T>(rotated(source + (size_t)head * per_head + head_dim, e));
+        for (int i = threadIdx.x; i < heads * rot_dim; i += blockDim.x) {
+            const int head = i / rot_dim, e = i % rot_dim;
+            queries[((size_t)t * heads + head) * row + latent + e] =
+                from_float<T>(rotated(source + (size_t)head * per_head + head_dim, e));
+        }
     }
-    if (!write) return;
+    if (small_source != nullptr) {
+        const T* source = small_source + (size_t)t * ld_small;
+        float squares = 0.f;
+        for (int e = threadIdx.x; e < rank; e += blockDim.x) {
+            const float v = to_float<T>(source[e]);
+            squares = fmaf(v, v, squares);
+        }
+        squares = block_sum(squares, scratch);
+        const float inv = rsqrtf(squares / (float)rank + eps);
+        for (int e = threadIdx.x; e < rank; e += blockDim.x)
+            small[(size_t)t * rank + e] = from_float<T>(to_float<T>(source[e]) * inv * small_weight[e]);
+    }
+    if (!write || down_source == nullptr) return;
     const int r = token_request[t];
     const int block = position / page_size;
     const int page = block < table_width ? block_table[(size_t)r * table_width + block] : -1;
@@ -75,7 +100,7 @@ latent_prepare_kernel(const T* __restrict__ projected, int ld, T* __restrict__ q
         return;
     }
     T* dst = pages + ((size_t)page * page_size + position % page_size) * row;
-    const T* down = source + (size_t)heads * per_head;
+    const T* down = down_source + (size_t)t * ld_down;
     float squares = 0.f;
     for (int e = threadIdx.x; e < latent; e += blockDim.x) {
         const float v = to_float<T>(down[e]);
@@ -194,38 +219,43 @@ __global__ void gate_heads_kernel(const T* __restrict__ values, const T* __restr
 
 }  // namespace
 
-MLXONE_API int mlxone_latent_prepare(const void* projected, int ld, void* queries,
+// q_source, small_source, down_source: null leaves a part out (see the kernel).
+MLXONE_API int mlxone_latent_prepare(const void* q_source, int ld_q, void* queries,
+                                     const void* small_source, int ld_small,
+                                     const float* small_weight, void* small, int rank,
+                                     const void* down_source, int ld_down,
                                      const float* norm_weight, float eps, const float* inv_freq,
-                                     int rotary_dim, int neighbours, const int* positions,
-                                     const int* token_request, void* pages, const int* block_table,
-                                     int table_width, int page_size, int tokens, int heads,
-                                     int head_dim, int rot_dim, int latent, int write, int dtype,
-                                     int* error_flag, cudaStream_t stream) {
+                                     int rotary_dim, float amplitude, int neighbours,
+                                     const int* positions, const int* token_request, void* pages,
+                                     const int* block_table, int table_width, int page_size,
+                                     int tokens, int heads, int head_dim, int rot_dim, int latent,
+                                     int write, int dtype, int* error_flag, cudaStream_t stream) {
     if (tokens == 0) return 0;
     MLXONE_REQUIRE(tokens > 0 && heads > 0 && head_dim >= 0 && rot_dim >= 0 && latent > 0,
                    "latent_prepare: bad sizes");
-    MLXONE_REQUIRE(ld >= heads * (head_dim + rot_dim) + latent + rot_dim,
-                   "latent_prepare: rows of %d values are too short", ld);
+    MLXONE_REQUIRE((q_source == nullptr || ld_q >= heads * (head_dim + rot_dim)) &&
+                       (down_source == nullptr || ld_down >= latent + rot_dim) &&
+                       (small_source == nullptr || (rank > 0 && ld_small >= rank)),
+                   "latent_prepare: rows of %d, %d, %d values are too short", ld_q, ld_small, ld_down);
     if (inv_freq == nullptr) rotary_dim = 0;
     MLXONE_REQUIRE(rotary_dim >= 0 && rotary_dim % 2 == 0 && rotary_dim <= rot_dim,
                    "latent_prepare: %d rotated dimensions in a part of %d", rotary_dim, rot_dim);
     const size_t shared = (size_t)rotary_dim * sizeof(float);
     // (the block's size follows the model's sizes alone, so a token's sums never change order)
-    const int most = heads * rot_dim > latent ? heads * rot_dim : latent;
+    int most = latent;
+    if (q_source != nullptr && heads * rot_dim > most) most = heads * rot_dim;
+    if (small_source != nullptr && rank > most) most = rank;
     const int threads = most >= 2048 ? 512 : most >= 512 ? 256 : 128;
-    if (dtype == MLXONE_BF16) {
-        using T = __nv_bfloat16;
-        launch_kernel(latent_prepare_kernel<T>, dim3(tokens), dim3(threads), shared, stream, true,
-                      (const T*)projected, ld, (T*)queries, norm_weight, eps, inv_freq, rotary_dim,
-                      neighbours, positions, token_request, (T*)pages, block_table, table_width,
-                      page_size, heads, head_dim, rot_dim, latent, write, error_flag);
-    } else {
-        using T = float;
-        launch_kernel(latent_prepare_kernel<T>, dim3(tokens), dim3(threads), shared, stream, true,
-                      (const T*)projected, ld, (T*)queries, norm_weight, eps, inv_freq, rotary_dim,
-                      neighbours, positions, token_request, (T*)pages, block_table, table_width,
-                      page_size, heads, head_dim, rot_dim, latent, write, error_flag);
-    }
+#define PREPARE(T)                                                                              \
+    launch_kernel(latent_prepare_kernel<T>, dim3(tokens), dim3(threads), shared, stream, true,  \
+                  (const T*)q_source, ld_q, (T*)queries, (const T*)small_source, ld_small,      \
+                  small_weight, (T*)small, rank, (const T*)down_source, ld_down, norm_weight, eps, \
+                  inv_freq, rotary_dim, amplitude, neighbours, positions, token_request, (T*)pages, \
+                  block_table, table_width, page_size, heads, head_dim, rot_dim, latent, write, \
+                  error_flag)
+    if (dtype == MLXONE_BF16) PREPARE(__nv_bfloat16);
+    else PREPARE(float);
+#undef PREPARE
     MLXONE_LAUNCH_CHECK("latent_prepare");
     return 0;
 }

@@ -18,6 +18,10 @@
 // side; each leaves (unnormalised output, maximum, sum) per row in scratch memory and a second
 // kernel merges them.
 //
+// `sinks` (float32 [heads] or null): exp(sink) of a row's head is one more term of its softmax's
+// denominator that has no key and no value: the row starts from (maximum = sink, sum = 1, output =
+// 0) instead of from nothing, in the first of several runs of keys only.
+//
 // Sizes: R a multiple of 8 up to 576 (padded with zeros to a multiple of 16 in shared memory),
 // latent a multiple of 8 up to 512. Anything else runs the general kernel.
 #include "common.cuh"
@@ -127,7 +131,7 @@ latent_attention_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pag
                         bf16* __restrict__ out, float* __restrict__ partial,
                         float* __restrict__ stats, int total_rows, int heads, int row_size,
                         int latent, float scale, int splits, int row_limit,
-                        int* __restrict__ error_flag) {
+                        const float* __restrict__ sinks, int* __restrict__ error_flag) {
     constexpr int ROWS = 16 * MT;
     extern __shared__ __align__(16) unsigned char raw[];
     const int request = blockIdx.y, split = blockIdx.z;
@@ -191,6 +195,11 @@ latent_attention_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pag
     for (int m = 0; m < MT; ++m) {
         peak[m][0] = peak[m][1] = -INFINITY;
         total[m][0] = total[m][1] = 0.f;
+        if (sinks != nullptr && split == 0) {
+            peak[m][0] = sinks[(row0 + m * 16 + g) % heads] * LOG2E;
+            peak[m][1] = sinks[(row0 + m * 16 + g + 8) % heads] * LOG2E;
+            total[m][0] = total[m][1] = 1.f;
+        }
 #pragma unroll
         for (int j = 0; j < GROUPS; ++j) o[m][j][0] = o[m][j][1] = o[m][j][2] = o[m][j][3] = 0.f;
     }
@@ -380,7 +389,7 @@ latent_attention_long_kernel(const bf16* __restrict__ q, const bf16* __restrict_
                              const int* __restrict__ positions,
                              const int* __restrict__ request_start, bf16* __restrict__ out,
                              int heads, int row_size, int latent, float scale,
-                             int* __restrict__ error_flag) {
+                             const float* __restrict__ sinks, int* __restrict__ error_flag) {
     constexpr int ROWS = 16 * (WARPS / C);
     extern __shared__ __align__(16) unsigned char raw[];
     const int request = blockIdx.y;
@@ -430,6 +439,11 @@ latent_attention_long_kernel(const bf16* __restrict__ q, const bf16* __restrict_
 #pragma unroll
     for (int j = 0; j < LONG_TILES; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
     float peak[2] = {-INFINITY, -INFINITY}, total[2] = {0.f, 0.f};
+    if (sinks != nullptr) {
+        peak[0] = sinks[(row0 + group * 16 + g) % heads] * LOG2E;
+        peak[1] = sinks[(row0 + group * 16 + g + 8) % heads] * LOG2E;
+        total[0] = total[1] = 1.f;
+    }
     const float factor = scale * LOG2E;
     const bf16* query_rows = q_tile + (group * 16 + (lane & 15)) * stride + (lane >> 4) * 8;
 
@@ -579,7 +593,7 @@ template <int C>
 int launch_latent_long(const bf16* q, const bf16* pages, const int* block_table, int table_width,
                        int page_size, const int* positions, const int* request_start, bf16* out,
                        int requests, int max_rows, int heads, int row_size, int latent, float scale,
-                       int* error_flag, cudaStream_t stream) {
+                       const float* sinks, int* error_flag, cudaStream_t stream) {
     constexpr int ROWS = 16 * (WARPS / C);
     static bool prepared = false;
     if (!prepared) {
@@ -592,7 +606,7 @@ int launch_latent_long(const bf16* q, const bf16* pages, const int* block_table,
     const dim3 grid((max_rows + ROWS - 1) / ROWS, requests);
     latent_attention_long_kernel<C><<<grid, WARPS * 32, long_shared_bytes<C>(row_size), stream>>>(
         q, pages, block_table, table_width, page_size, positions, request_start, out, heads,
-        row_size, latent, scale, error_flag);
+        row_size, latent, scale, sinks, error_flag);
     MLXONE_LAUNCH_CHECK("latent_attention_long");
     return 0;
 }
@@ -607,6 +621,8 @@ latent_merge_kernel(const float* __restrict__ partial, const float* __restrict__
     __shared__ float factors[MAX_SPLITS];
     const int row = blockIdx.x;
     griddep_wait();
+    partial = settled(partial);
+    stats = settled(stats);
     if (threadIdx.x < 32) {
         const int s = threadIdx.x;
         float peak = -INFINITY, sum = 0.f;
@@ -639,7 +655,7 @@ int launch_latent(const bf16* q, const bf16* pages, const int* block_table, int 
                   int page_size, const int* positions, const int* request_start, bf16* out,
                   float* partial, float* stats, int total_rows, int requests, int max_rows,
                   int heads, int row_size, int latent, float scale, int splits, int row_limit,
-                  int* error_flag, cudaStream_t stream) {
+                  const float* sinks, int* error_flag, cudaStream_t stream) {
     constexpr int ROWS = 16 * MT;
     const int stride = ((row_size + 15) & ~15) + 8;
     const size_t shared = (size_t)(ROWS + 2 * KEYS) * stride * sizeof(bf16) +
@@ -657,7 +673,7 @@ int launch_latent(const bf16* q, const bf16* pages, const int* block_table, int 
     cudaError_t launched = launch_kernel(
         latent_attention_kernel<MT>, grid, dim3(WARPS * 32), shared, stream, true, q, pages,
         block_table, table_width, page_size, positions, request_start, out, partial, stats,
-        total_rows, heads, row_size, latent, scale, splits, row_limit, error_flag);
+        total_rows, heads, row_size, latent, scale, splits, row_limit, sinks, error_flag);
     MLXONE_REQUIRE(launched == cudaSuccess, "latent attention: %s", cudaGetErrorString(launched));
     MLXONE_LAUNCH_CHECK("latent_attention_mma");
     return 0;
@@ -679,7 +695,8 @@ MLXONE_API int mlxone_latent_attention_mma(const void* q, const void* pages, con
                                            const int* request_start, void* out, float* scratch,
                                            int tokens, int requests, int max_portion, int heads,
                                            int row_size, int latent, float scale, int splits,
-                                           int* error_flag, cudaStream_t stream) {
+                                           const float* sinks, int* error_flag,
+                                           cudaStream_t stream) {
     if (tokens == 0) return 0;
     MLXONE_REQUIRE(mlxone_latent_attention_mma_fits(row_size, latent),
                    "latent attention: rows of %d with %d latent values do not fit", row_size, latent);
@@ -701,10 +718,10 @@ MLXONE_API int mlxone_latent_attention_mma(const void* q, const void* pages, con
         status = halves
             ? launch_latent_long<2>((const bf16*)q, (const bf16*)pages, block_table, table_width,
                                     page_size, positions, request_start, (bf16*)out, requests,
-                                    (int)max_rows, heads, row_size, latent, scale, error_flag, stream)
+                                    (int)max_rows, heads, row_size, latent, scale, sinks, error_flag, stream)
             : launch_latent_long<1>((const bf16*)q, (const bf16*)pages, block_table, table_width,
                                     page_size, positions, request_start, (bf16*)out, requests,
-                                    (int)max_rows, heads, row_size, latent, scale, error_flag, stream);
+                                    (int)max_rows, heads, row_size, latent, scale, sinks, error_flag, stream);
         if (status || requests == 1) return status;
         row_limit = LONG_ROWS;
     }
@@ -713,12 +730,12 @@ MLXONE_API int mlxone_latent_attention_mma(const void* q, const void* pages, con
         status = launch_latent<2>((const bf16*)q, (const bf16*)pages, block_table, table_width,
                                   page_size, positions, request_start, (bf16*)out, partial, stats,
                                   total_rows, requests, short_rows, heads, row_size, latent,
-                                  scale, splits, row_limit, error_flag, stream);
+                                  scale, splits, row_limit, sinks, error_flag, stream);
     else
         status = launch_latent<1>((const bf16*)q, (const bf16*)pages, block_table, table_width,
                                   page_size, positions, request_start, (bf16*)out, partial, stats,
                                   total_rows, requests, short_rows, heads, row_size, latent,
-                                  scale, splits, row_limit, error_flag, stream);
+                                  scale, splits, row_limit, sinks, error_flag, stream);
     if (status) return status;
     if (splits > 1) {
         cudaError_t launched = launch_kernel(latent_merge_kernel, dim3(total_rows), dim3(128), 0,

@@ -23,6 +23,7 @@ route_experts_kernel(const T* __restrict__ x, int ld, const float* __restrict__ 
     __shared__ unsigned char allowed[MAX_EXPERTS];
     griddep_launch();
     griddep_wait();
+    x = settled(x);
     const int t = blockIdx.x;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const T* row = x + (size_t)t * ld;
@@ -96,7 +97,9 @@ route_experts_kernel(const T* __restrict__ x, int ld, const float* __restrict__ 
 // The second routing kernel: scores over all `outputs` of the router (sigmoid, or softmax over all
 // of them), an optional correction per output that is added where the `top` best are chosen
 // (ties: the lower index) and nowhere else, weights = the chosen outputs' scores, divided by their
-// sum only with `normalize`. The first `experts` outputs are experts with tensors: their weights
+// sum only with `normalize`, and multiplied by `scale`. With `groups` > 1 the outputs form that
+// many equal runs of neighbours, a run's value is the sum of its `group_score` largest, and only
+// outputs of the `keep` best runs (ties: the lower run) can be chosen. The first `experts` outputs are experts with tensors: their weights
 // go to weights[t, experts]. The outputs behind them hand the token on as it is: the sum of their
 // chosen weights goes to others[0][t]. With `shared_gate` the router has one more row behind its
 // outputs, and others[1][t] = sigmoid of that row's product with the token.
@@ -105,16 +108,36 @@ route_experts_kernel(const T* __restrict__ x, int ld, const float* __restrict__ 
 // that a row's loads are on their way together; the sums are added in a fixed order.
 constexpr int GENERAL_THREADS = 512;
 
+// The place of the largest of values[0 .. count) (ties: the lower place; -1: all are minus
+// infinity), the same in all lanes of a warp.
+__device__ __forceinline__ int warp_best(const float* values, int count, int lane) {
+    float best = -INFINITY;
+    int at = count;
+    for (int e = lane; e < count; e += 32)
+        if (values[e] > best) { best = values[e]; at = e; }
+#pragma unroll
+    for (int across = 16; across > 0; across >>= 1) {
+        const float other = __shfl_xor_sync(0xffffffffu, best, across);
+        const int other_at = __shfl_xor_sync(0xffffffffu, at, across);
+        if (other > best || (other == best && other_at < at)) { best = other; at = other_at; }
+    }
+    return best == -INFINITY ? -1 : at;
+}
+
 template <typename T>
 __global__ void __launch_bounds__(GENERAL_THREADS)
 route_general_kernel(const T* __restrict__ x, int ld, const float* __restrict__ router,
                      const float* __restrict__ correction, float* __restrict__ weights,
                      float* __restrict__ others, int tokens, int hidden, int experts, int outputs,
-                     int top, int softmax, int normalize, int shared_gate, int wide) {
+                     int top, int softmax, int normalize, int shared_gate, int groups, int keep,
+                     int group_score, float scale, int wide) {
     __shared__ float score[MAX_EXPERTS + 1];
     __shared__ float choice[MAX_EXPERTS];
+    __shared__ float group_value[MAX_EXPERTS];
+    __shared__ int chosen[64];
     griddep_launch();
     griddep_wait();
+    x = settled(x);
     const int t = blockIdx.x;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const T* row = x + (size_t)t * ld;
@@ -152,40 +175,77 @@ route_general_kernel(const T* __restrict__ x, int ld, const float* __restrict__ 
     for (int e = threadIdx.x; e < experts; e += GENERAL_THREADS)
         weights[(size_t)t * experts + e] = 0.f;
     __syncthreads();
-    if (threadIdx.x != 0) return;
+    if (warp != 0) return;
+    // ---- one warp: a lane holds every 32nd output; sums over the lanes have a fixed order
     if (softmax) {
         float most = -INFINITY, total = 0.f;
-        for (int e = 0; e < outputs; ++e) most = fmaxf(most, score[e]);
-        for (int e = 0; e < outputs; ++e) { score[e] = expf(score[e] - most); total += score[e]; }
-        for (int e = 0; e < outputs; ++e) score[e] /= total;
+        for (int e = lane; e < outputs; e += 32) most = fmaxf(most, score[e]);
+        most = warp_max(most);
+        for (int e = lane; e < outputs; e += 32) { score[e] = expf(score[e] - most); total += score[e]; }
+        total = warp_sum(total);
+        for (int e = lane; e < outputs; e += 32) score[e] /= total;
     } else {
-        for (int e = 0; e < outputs; ++e) score[e] = 1.f / (1.f + expf(-score[e]));
+        for (int e = lane; e < outputs; e += 32) score[e] = 1.f / (1.f + expf(-score[e]));
     }
-    for (int e = 0; e < outputs; ++e)
+    for (int e = lane; e < outputs; e += 32)
         choice[e] = correction != nullptr ? score[e] + correction[e] : score[e];
-    int chosen[64];
+    __syncwarp();
+    if (groups > 1) {
+        // a group's value: the sum of its `group_score` largest, found one below the other
+        const int per = outputs / groups;
+        for (int group = lane; group < groups; group += 32) {
+            float value = 0.f, last = INFINITY;
+            int last_at = -1;
+            for (int pick = 0; pick < group_score && pick < per; ++pick) {
+                float best = -INFINITY;
+                int at = -1;
+                for (int i = 0; i < per; ++i) {
+                    const float v = choice[group * per + i];
+                    if ((v < last || (v == last && i > last_at)) && (at < 0 || v > best)) { best = v; at = i; }
+                }
+                if (at < 0) break;
+                value += best;
+                last = best;
+                last_at = at;
+            }
+            group_value[group] = value;
+        }
+        __syncwarp();
+        for (int pick = 0; pick < keep; ++pick) {
+            const int best = warp_best(group_value, groups, lane);
+            if (best < 0) break;
+            if (lane == 0) group_value[best] = -INFINITY;
+            __syncwarp();
+        }
+        // (the kept groups are those whose value was taken away)
+        for (int e = lane; e < outputs; e += 32)
+            if (group_value[e / per] != -INFINITY) choice[e] = -INFINITY;
+        __syncwarp();
+    }
     int count = 0;
     float total = 0.f;
-    for (int pick = 0; pick < top; ++pick) {
-        int best = -1;
-        float best_value = -INFINITY;
-        for (int e = 0; e < outputs; ++e)
-            if (choice[e] > best_value) { best_value = choice[e]; best = e; }
+    for (; count < top; ++count) {
+        const int best = warp_best(choice, outputs, lane);
         if (best < 0) break;
-        choice[best] = -INFINITY;
-        chosen[count++] = best;
         total += score[best];
+        if (lane == 0) {
+            choice[best] = -INFINITY;
+            chosen[count] = best;
+        }
+        __syncwarp();
     }
-    const float factor = normalize ? 1.f / (total + 1e-20f) : 1.f;
+    const float factor = normalize ? scale / (total + 1e-20f) : scale;
     float handed_on = 0.f;
     // (in ascending order of the outputs, so that the sum does not depend on the ranking)
     for (int e = experts; e < outputs; ++e)
         for (int i = 0; i < count; ++i)
             if (chosen[i] == e) handed_on += score[e] * factor;
-    for (int i = 0; i < count; ++i)
+    for (int i = lane; i < count; i += 32)
         if (chosen[i] < experts) weights[(size_t)t * experts + chosen[i]] = score[chosen[i]] * factor;
-    others[t] = handed_on;
-    others[(size_t)tokens + t] = shared_gate ? 1.f / (1.f + expf(-score[outputs])) : 1.f;
+    if (lane == 0) {
+        others[t] = handed_on;
+        others[(size_t)tokens + t] = shared_gate ? 1.f / (1.f + expf(-score[outputs])) : 1.f;
+    }
 }
 
 // out[t, c] += factors[t] * x[t, c], taken in 32-bit
@@ -209,6 +269,8 @@ __global__ void scale_expert_columns_kernel(T* __restrict__ x, int ld, const flo
                                             const float* __restrict__ tail, int tail_width) {
     griddep_launch();
     griddep_wait();
+    weights = settled(weights);
+    tail = settled(tail);
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= total) return;
     const int across = experts * width + tail_width;
@@ -237,6 +299,7 @@ sort_by_expert_kernel(const float* __restrict__ weights, int* __restrict__ pair_
     __shared__ int start[MAX_EXPERTS];
     griddep_launch();
     griddep_wait();
+    weights = settled(weights);
     for (int e = threadIdx.x; e < experts; e += SORT_THREADS) count[e] = 0;
     __syncthreads();
     const long long pairs = (long long)tokens * experts;
@@ -260,13 +323,15 @@ sort_by_expert_kernel(const float* __restrict__ weights, int* __restrict__ pair_
         if (pair_row[i] >= 0) pair_row[i] += start[i % experts];
 }
 
-// sorted[pair_row[t, e], :] = x[t, :] for every chosen pair. One block per token; 16 bytes a
+// sorted[pair_row[t, e], :] = x[t, :] for every chosen pair (`limit` rows). One block per token; 16 bytes a
 // copy where the rows allow it.
 template <typename T>
 __global__ void gather_by_expert_kernel(const T* __restrict__ x, int ld, const int* __restrict__ pair_row,
-                                        T* __restrict__ sorted, int hidden, int experts) {
+                                        T* __restrict__ sorted, int hidden, int experts, int limit) {
     griddep_launch();
     griddep_wait();
+    x = settled(x);
+    pair_row = settled(pair_row);
     const int t = blockIdx.x;
     constexpr int PER = 16 / sizeof(T);
     const bool wide = hidden % PER == 0 && ld % PER == 0 &&
@@ -274,7 +339,7 @@ __global__ void gather_by_expert_kernel(const T* __restrict__ x, int ld, const i
                       (reinterpret_cast<uintptr_t>(sorted) & 15) == 0;
     for (int e = 0; e < experts; ++e) {
         const int row = pair_row[(size_t)t * experts + e];
-        if (row < 0) continue;
+        if (row < 0 || row >= limit) continue;
         const T* from = x + (size_t)t * ld;
         T* to = sorted + (size_t)row * hidden;
         if (wide) {
@@ -293,18 +358,22 @@ constexpr int MAX_TOP = 64;
 template <typename T>
 __global__ void combine_experts_kernel(const T* __restrict__ y, const int* __restrict__ pair_row,
                                        const float* __restrict__ weights, const T* __restrict__ shared_out,
-                                       T* __restrict__ out, int hidden, int experts) {
+                                       T* __restrict__ out, int hidden, int experts, int limit) {
     __shared__ int rows[MAX_TOP];
     __shared__ float factors[MAX_TOP];
     __shared__ int chosen;
     griddep_launch();
     griddep_wait();
+    y = settled(y);
+    pair_row = settled(pair_row);
+    weights = settled(weights);
+    shared_out = settled(shared_out);
     const int t = blockIdx.x;
     if (threadIdx.x == 0) {
         int count = 0;
         for (int e = 0; e < experts && count < MAX_TOP; ++e) {
             const int row = pair_row[(size_t)t * experts + e];
-            if (row >= 0) {
+            if (row >= 0 && row < limit) {
                 rows[count] = row;
                 factors[count++] = weights[(size_t)t * experts + e];
             }
@@ -363,7 +432,7 @@ MLXONE_API int mlxone_sort_by_expert(const float* weights, int* pair_row, int* g
 }
 
 MLXONE_API int mlxone_gather_by_expert(const void* x, int ld, const int* pair_row, void* sorted,
-                                       int tokens, int hidden, int experts, int dtype,
+                                       int tokens, int hidden, int experts, int limit, int dtype,
                                        cudaStream_t stream) {
     if (tokens == 0) return 0;
     MLXONE_REQUIRE(tokens > 0 && hidden > 0 && experts > 0, "gather_by_expert: bad sizes");
@@ -371,28 +440,28 @@ MLXONE_API int mlxone_gather_by_expert(const void* x, int ld, const int* pair_ro
     if (dtype == MLXONE_BF16)
         launch_kernel(gather_by_expert_kernel<__nv_bfloat16>, dim3(tokens), dim3(threads), 0, stream,
                       true, (const __nv_bfloat16*)x, ld, pair_row, (__nv_bfloat16*)sorted, hidden,
-                      experts);
+                      experts, limit);
     else
         launch_kernel(gather_by_expert_kernel<float>, dim3(tokens), dim3(threads), 0, stream, true,
-                      (const float*)x, ld, pair_row, (float*)sorted, hidden, experts);
+                      (const float*)x, ld, pair_row, (float*)sorted, hidden, experts, limit);
     MLXONE_LAUNCH_CHECK("gather_by_expert");
     return 0;
 }
 
 MLXONE_API int mlxone_combine_experts(const void* y, const int* pair_row, const float* weights,
                                       const void* shared_out, void* out, int tokens, int hidden,
-                                      int experts, int dtype, cudaStream_t stream) {
+                                      int experts, int limit, int dtype, cudaStream_t stream) {
     if (tokens == 0) return 0;
     MLXONE_REQUIRE(tokens > 0 && hidden > 0 && experts > 0, "combine_experts: bad sizes");
     const int threads = hidden >= 1024 ? 256 : 128;
     if (dtype == MLXONE_BF16)
         launch_kernel(combine_experts_kernel<__nv_bfloat16>, dim3(tokens), dim3(threads), 0, stream,
                       true, (const __nv_bfloat16*)y, pair_row, weights,
-                      (const __nv_bfloat16*)shared_out, (__nv_bfloat16*)out, hidden, experts);
+                      (const __nv_bfloat16*)shared_out, (__nv_bfloat16*)out, hidden, experts, limit);
     else
         launch_kernel(combine_experts_kernel<float>, dim3(tokens), dim3(threads), 0, stream, true,
                       (const float*)y, pair_row, weights, (const float*)shared_out, (float*)out,
-                      hidden, experts);
+                      hidden, experts, limit);
     MLXONE_LAUNCH_CHECK("combine_experts");
     return 0;
 }
@@ -455,7 +524,8 @@ MLXONE_API int mlxone_scale_expert_columns_tail(void* x, int ld, const float* we
 MLXONE_API int mlxone_route_general(const void* x, int ld, const float* router,
                                     const float* correction, float* weights, float* others,
                                     int tokens, int hidden, int experts, int identity, int top,
-                                    int softmax, int normalize, int shared_gate, int dtype,
+                                    int softmax, int normalize, int shared_gate, int groups,
+                                    int keep, int group_score, float scale, int dtype,
                                     cudaStream_t stream) {
     if (tokens == 0) return 0;
     const int outputs = experts + identity;
@@ -463,6 +533,10 @@ MLXONE_API int mlxone_route_general(const void* x, int ld, const float* router,
                    "route_general: 1 to %d outputs of the router", MAX_EXPERTS);
     MLXONE_REQUIRE(top > 0 && top <= 64 && top <= outputs, "route_general: top %d of %d outputs", top,
                    outputs);
+    MLXONE_REQUIRE(groups >= 1 && outputs % groups == 0 && keep >= 1 && keep <= groups &&
+                       group_score >= 1 && top <= keep * (outputs / groups),
+                   "route_general: %d outputs do not form %d groups of which %d are kept for the top "
+                   "%d", outputs, groups, keep, top);
     // four values a load where rows start on 16 bytes (the router's) and on 4 values (the tokens')
     const size_t value = dtype == MLXONE_BF16 ? 2 : 4;
     const int wide = hidden % 4 == 0 && ld % 4 == 0 && (uintptr_t)x % (4 * value) == 0 &&
@@ -470,11 +544,13 @@ MLXONE_API int mlxone_route_general(const void* x, int ld, const float* router,
     if (dtype == MLXONE_BF16)
         launch_kernel(route_general_kernel<__nv_bfloat16>, dim3(tokens), dim3(GENERAL_THREADS), 0,
                       stream, true, (const __nv_bfloat16*)x, ld, router, correction, weights, others,
-                      tokens, hidden, experts, outputs, top, softmax, normalize, shared_gate, wide);
+                      tokens, hidden, experts, outputs, top, softmax, normalize, shared_gate, groups,
+                      keep, group_score, scale, wide);
     else
         launch_kernel(route_general_kernel<float>, dim3(tokens), dim3(GENERAL_THREADS), 0, stream,
                       true, (const float*)x, ld, router, correction, weights, others, tokens, hidden,
-                      experts, outputs, top, softmax, normalize, shared_gate, wide);
+                      experts, outputs, top, softmax, normalize, shared_gate, groups, keep, group_score,
+                      scale, wide);
     MLXONE_LAUNCH_CHECK("route_general");
     return 0;
 }

@@ -57,6 +57,7 @@ class CudaOps:
         self.lib.mlxone_last_error.restype = ctypes.c_char_p
         self.lib.mlxone_gated_delta_scratch.restype = ctypes.c_longlong
         self.lib.mlxone_gated_delta_state.restype = ctypes.c_longlong
+        self.lib.mlxone_channel_delta_scratch.restype = ctypes.c_longlong
         self.lib.mlxone_lightning_scratch.restype = ctypes.c_longlong
         self.lib.mlxone_state_space_scratch.restype = ctypes.c_longlong
         if self.lib.mlxone_abi_version() != 1:
@@ -217,6 +218,7 @@ class CudaOps:
     # epilogues of the skinny product
     _STORE, _SWIGLU, _ADD, _STORE_F32 = 0, 1, 2, 3
     _ACTIVATE = 16          # + the activation's code: a bfloat16 store of the activated product
+    _GROUPED_RELU2 = 4      # (grouped products only) a bfloat16 store of max(z, 0)^2
     _GATED = 32             # + the activation's code: as _SWIGLU with that gate
 
     def _skinny(self, a, w, fused=False) -> bool:
@@ -324,10 +326,10 @@ class CudaOps:
         m, k = a.shape
         n = w.shape[0]
         if a.dtype == torch.float32:
-            self._need(a, torch.float32, "a")
+            self._need_rows(a, torch.float32, "a")
             self._need(w, torch.float32, "w")
             out = torch.empty((m, n), dtype=torch.float32, device=self.device)
-            self._call("mlxone_gemm_f32", _c_void_p(_ptr(a)), _c_int(k), _c_void_p(_ptr(w)),
+            self._call("mlxone_gemm_f32", _c_void_p(_ptr(a)), _c_int(max(a.stride(0), k)), _c_void_p(_ptr(w)),
                        _c_int(k), _c_void_p(_ptr(bias)), _c_void_p(_ptr(out)), _c_int(n),
                        _c_int(m), _c_int(n), _c_int(k))
             return out
@@ -560,29 +562,76 @@ class CudaOps:
 
     # ---- attention over one latent row per token; two score maps per head
 
-    def latent_prepare(self, projected, queries, *, heads, head_dim, rot_dim, latent, norm_weight,
-                       eps, rotary, neighbours, ctx, view, write):
-        """The rotated parts of the queries into ``queries[:, :, latent:]``; the token's row
-        [normed latent | rotated shared key part] into its request's pages."""
-        self._need_rows(projected, queries.dtype, "projected")
-        self._need(queries, queries.dtype, "queries")
-        self._need(norm_weight, torch.float32, "norm weight")
-        self._need(view.kv, queries.dtype, "pages")
+    def _latent_prepare(self, dtype, tokens, *, q=None, queries=None, small_source=None, small=None,
+                        small_weight=None, down=None, norm_weight=None, eps=0.0, heads=1, head_dim=0,
+                        rot_dim, latent, rotary, amplitude, neighbours, ctx, view=None, write=False):
         row = latent + rot_dim
-        if queries.shape[1:] != (heads, row) or view.kv.shape[0] != 1 or \
-                view.kv.shape[2] != 1 or view.kv.shape[-1] != row:
-            raise KernelError("queries and pages hold rows of latent + rot_dim values")
+        for rows, what in ((q, "queries' projection"), (small_source, "queries' latent"),
+                           (down, "down projection")):
+            if rows is not None:
+                self._need_rows(rows, dtype, what)
+        if queries is not None:
+            self._need(queries, dtype, "queries")
+            if queries.shape[1:] != (heads, row):
+                raise KernelError("queries are rows of latent + rot_dim values")
+        table = pages = None
+        width = page_size = 1
+        if down is not None:
+            self._need(norm_weight, torch.float32, "norm weight")
+            self._need(view.kv, dtype, "pages")
+            if view.kv.shape[0] != 1 or view.kv.shape[2] != 1 or view.kv.shape[-1] != row:
+                raise KernelError("pages hold rows of latent + rot_dim values")
+            pages, table = view.kv, view.block_table
+            width, page_size = table.shape[1], view.page_size
         inv_freq, rotary_dim = (None, 0) if rotary is None else rotary
-        self._call("mlxone_latent_prepare", _c_void_p(_ptr(projected)),
-                   _c_int(projected.stride(0)), _c_void_p(_ptr(queries)),
-                   _c_void_p(_ptr(norm_weight)), _c_float(eps), _c_void_p(_ptr(inv_freq)),
-                   _c_int(rotary_dim), _c_int(1 if neighbours else 0),
+        stride = lambda rows: 0 if rows is None else rows.stride(0)
+        self._call("mlxone_latent_prepare", _c_void_p(_ptr(q)), _c_int(stride(q)),
+                   _c_void_p(_ptr(queries)), _c_void_p(_ptr(small_source)),
+                   _c_int(stride(small_source)), _c_void_p(_ptr(small_weight)),
+                   _c_void_p(_ptr(small)), _c_int(0 if small is None else small.shape[1]),
+                   _c_void_p(_ptr(down)), _c_int(stride(down)), _c_void_p(_ptr(norm_weight)),
+                   _c_float(eps), _c_void_p(_ptr(inv_freq)), _c_int(rotary_dim),
+                   _c_float(amplitude), _c_int(1 if neighbours else 0),
                    _c_void_p(_ptr(ctx.positions)), _c_void_p(_ptr(ctx.token_request)),
-                   _c_void_p(_ptr(view.kv)), _c_void_p(_ptr(view.block_table)),
-                   _c_int(view.block_table.shape[1]), _c_int(view.page_size),
-                   _c_int(projected.shape[0]), _c_int(heads), _c_int(head_dim), _c_int(rot_dim),
-                   _c_int(latent), _c_int(1 if write else 0), _c_int(_dtype_code(queries.dtype)),
-                   _c_void_p(_ptr(self.error_flag)))
+                   _c_void_p(_ptr(pages)), _c_void_p(_ptr(table)), _c_int(width),
+                   _c_int(page_size), _c_int(tokens), _c_int(heads), _c_int(head_dim),
+                   _c_int(rot_dim), _c_int(latent), _c_int(1 if write else 0),
+                   _c_int(_dtype_code(dtype)), _c_void_p(_ptr(self.error_flag)))
+
+    def latent_prepare(self, projected, queries, *, heads, head_dim, rot_dim, latent, norm_weight,
+                       eps, rotary, neighbours, ctx, view, write, amplitude=1.0):
+        """projected [tokens, queries | latent | shared key part | ...]: the rotated parts of the
+        queries into ``queries[:, :, latent:]``; the token's row [normed latent | rotated shared
+        key part] into its request's pages. ``amplitude``: a factor on cosine and sine."""
+        width = heads * (head_dim + rot_dim)
+        self._latent_prepare(queries.dtype, projected.shape[0], q=projected[:, :width],
+                             queries=queries, down=projected[:, width:width + latent + rot_dim],
+                             norm_weight=norm_weight, eps=eps, heads=heads, head_dim=head_dim,
+                             rot_dim=rot_dim, latent=latent, rotary=rotary, amplitude=amplitude,
+                             neighbours=neighbours, ctx=ctx, view=view, write=write)
+
+    def latent_rows(self, projected, *, rank, query_norm, norm_weight, eps, rot_dim, latent, rotary,
+                    neighbours, ctx, view, write, amplitude=1.0):
+        """projected [tokens, queries' latent | latent | shared key part]: the token's row into its
+        request's pages as ``latent_prepare`` does; returns the queries' latent [tokens, rank],
+        normed with ``query_norm``."""
+        self._need(query_norm, torch.float32, "query norm")
+        small = torch.empty((projected.shape[0], rank), dtype=projected.dtype, device=self.device)
+        self._latent_prepare(projected.dtype, projected.shape[0], small_source=projected[:, :rank],
+                             small=small, small_weight=query_norm,
+                             down=projected[:, rank:rank + latent + rot_dim],
+                             norm_weight=norm_weight, eps=eps, rot_dim=rot_dim, latent=latent,
+                             rotary=rotary, amplitude=amplitude, neighbours=neighbours, ctx=ctx,
+                             view=view, write=write)
+        return small
+
+    def latent_queries(self, q, queries, *, heads, head_dim, rot_dim, latent, rotary, neighbours,
+                       ctx, amplitude=1.0):
+        """q [tokens, heads * (head_dim + rot_dim)]: the rotated parts of the queries into
+        ``queries[:, :, latent:]``."""
+        self._latent_prepare(queries.dtype, q.shape[0], q=q, queries=queries, heads=heads,
+                             head_dim=head_dim, rot_dim=rot_dim, latent=latent, rotary=rotary,
+                             amplitude=amplitude, neighbours=neighbours, ctx=ctx)
 
     def linear_heads(self, a, w, out=None):
         """a [tokens, heads, K] with w [heads, N, K] -> [tokens, heads, N], one product per head.
@@ -607,16 +656,22 @@ class CudaOps:
             torch.bmm(a.transpose(0, 1), w.transpose(1, 2), out=out.transpose(0, 1))
         return out
 
-    def latent_attention(self, queries, *, heads, latent, scale, ctx, view):
+    def latent_attention(self, queries, *, heads, latent, scale, ctx, view, sinks=None):
         """Causal softmax attention of queries [tokens, heads, row] over the one row per token in
         the request's single-plane pages, which is key and value at once. Returns [tokens, heads,
         row]; the first ``latent`` values of a row are the weights' average of the latents.
+        ``sinks`` (float32 [heads]): exp(sink) of a query's head stands in its softmax's
+        denominator.
 
         The bfloat16 kernel is launched as a programmatic dependent of the kernel ahead of it in
         the stream; before it waits for that kernel it reads ``ctx.positions``, the block table
         and rows of positions before the step's first (rows that earlier steps wrote)."""
         tokens, _, row = queries.shape
         self._need(queries, view.kv.dtype, "queries")
+        if sinks is not None:
+            self._need(sinks, torch.float32, "sinks")
+            if sinks.numel() != heads:
+                raise KernelError("one sink per query head")
         out = torch.empty((tokens, heads, row), dtype=queries.dtype, device=self.device)
         if queries.dtype == torch.bfloat16 and \
                 self.lib.mlxone_latent_attention_mma_fits(_c_int(row), _c_int(latent)):
@@ -640,7 +695,7 @@ class CudaOps:
                        _c_void_p(_ptr(ctx.positions)), _c_void_p(_ptr(ctx.request_start)),
                        _c_void_p(_ptr(out)), _c_void_p(_ptr(scratch)), _c_int(tokens),
                        _c_int(ctx.requests), _c_int(ctx.max_portion), _c_int(heads), _c_int(row),
-                       _c_int(latent), _c_float(scale), _c_int(splits),
+                       _c_int(latent), _c_float(scale), _c_int(splits), _c_void_p(_ptr(sinks)),
                        _c_void_p(_ptr(self.error_flag)))
             return out
         self._call("mlxone_attention_generic_planes", _c_void_p(_ptr(queries)),
@@ -649,7 +704,7 @@ class CudaOps:
                    _c_int(view.kv.shape[1]), _c_void_p(_ptr(ctx.positions)),
                    _c_void_p(_ptr(ctx.token_request)), _c_void_p(_ptr(out)), _c_int(tokens),
                    _c_int(heads), _c_int(1), _c_int(row), _c_float(scale), _c_int(0),
-                   _c_int(_dtype_code(queries.dtype)), _c_void_p(None), _c_int(1),
+                   _c_int(_dtype_code(queries.dtype)), _c_void_p(_ptr(sinks)), _c_int(1),
                    _c_void_p(_ptr(self.error_flag)))
         return out
 
@@ -769,12 +824,14 @@ class CudaOps:
                    _c_int(width), _c_int(_dtype_code(gated.dtype)))
 
     def route_general(self, x, router, correction, *, experts, identity, top, scores, normalize,
-                      shared_gate):
+                      shared_gate, groups=1, keep=1, group_score=1, scale=1.0):
         """The second routing kernel. ``router`` float32 [experts + identity (+ 1 with
         ``shared_gate``), hidden]; scores are the sigmoid of the 32-bit logits or their softmax
         over the experts + identity outputs; ``correction`` (float32 per output, or None) is
         added where the ``top`` best are chosen; the weights are the chosen scores, divided by
-        their sum with ``normalize``. Returns (weights float32 [tokens, experts], zero where an
+        their sum with ``normalize``, times ``scale``. With ``groups`` the outputs form that many
+        equal runs of neighbours, of which the ``keep`` best by the sum of their ``group_score``
+        largest scores may be chosen from. Returns (weights float32 [tokens, experts], zero where an
         expert was not chosen; others float32 [2, tokens]: the sum of the chosen identity
         outputs' weights, and the sigmoid of the router's last row's logit, 1 without
         ``shared_gate``)."""
@@ -796,7 +853,8 @@ class CudaOps:
                    _c_void_p(_ptr(router)), _c_void_p(_ptr(correction)), _c_void_p(_ptr(weights)),
                    _c_void_p(_ptr(others)), _c_int(tokens), _c_int(x.shape[1]), _c_int(experts),
                    _c_int(identity), _c_int(top), _c_int(1 if scores == "softmax" else 0),
-                   _c_int(1 if normalize else 0), _c_int(1 if shared_gate else 0),
+                   _c_int(1 if normalize else 0), _c_int(1 if shared_gate else 0), _c_int(groups),
+                   _c_int(keep), _c_int(group_score), _c_float(scale),
                    _c_int(_dtype_code(x.dtype)))
         return weights, others
 
@@ -940,13 +998,17 @@ class CudaOps:
                 and x.stride(1) == 1 and x.stride(0) % 8 == 0)
 
     def routed_experts_sorted(self, x, weights, gate_up, down, *, experts, width, top,
-                              shared_gate_up=None, shared_down=None, shared_scale=None):
+                              shared_gate_up=None, shared_down=None, shared_scale=None,
+                              activation=None):
         """The weighted sum of every token's chosen experts (+ the shared expert's output), with
         the tokens sorted by expert: gate_up [2 stack, hidden] holds the experts' gate rows, then
         (``stack`` rows further) their up rows; down [hidden, stack] their down matrices side by
-        side. weights [tokens, experts] float32, zero where an expert was not chosen."""
+        side. ``activation`` (relu2): experts without a gate, gate_up [stack, hidden] holds their
+        up rows alone. weights [tokens, experts] float32, zero where an expert was not chosen."""
         tokens, hidden = x.shape
-        stack = gate_up.shape[0] // 2
+        if activation not in (None, "relu2"):
+            raise KernelError(f"no grouped product with the activation {activation!r}")
+        stack = gate_up.shape[0] if activation else gate_up.shape[0] // 2
         tiles = -(-(tokens * top + experts * 127) // 128)
         rows = tiles * 128
         pair_row = torch.empty((tokens, experts), dtype=torch.int32, device=self.device)
@@ -959,12 +1021,13 @@ class CudaOps:
         sorted_x = torch.empty((rows, hidden), dtype=x.dtype, device=self.device)
         self._call("mlxone_gather_by_expert", _c_void_p(_ptr(x)), _c_int(x.stride(0)),
                    _c_void_p(_ptr(pair_row)), _c_void_p(_ptr(sorted_x)), _c_int(tokens),
-                   _c_int(hidden), _c_int(experts), _c_int(_dtype_code(x.dtype)))
+                   _c_int(hidden), _c_int(experts), _c_int(rows), _c_int(_dtype_code(x.dtype)))
         gated = torch.empty((rows, width), dtype=x.dtype, device=self.device)
         self._call("mlxone_gemm_tcgen05_grouped", _c_void_p(_ptr(sorted_x)), _c_int(hidden),
                    _c_void_p(_ptr(gate_up)), _c_ll(gate_up.shape[0]), _c_ll(hidden), _c_ll(hidden),
                    _c_void_p(_ptr(gated)), _c_int(width), _c_int(rows), _c_int(width),
-                   _c_int(hidden), _c_int(stack), _c_int(self._SWIGLU),
+                   _c_int(hidden), _c_int(0 if activation else stack),
+                   _c_int(self._GROUPED_RELU2 if activation else self._SWIGLU),
                    _c_void_p(_ptr(groups[0])), _c_void_p(_ptr(self.error_flag)))
         y = torch.empty((rows, hidden), dtype=x.dtype, device=self.device)
         self._call("mlxone_gemm_tcgen05_grouped", _c_void_p(_ptr(gated)), _c_int(width),
@@ -984,7 +1047,8 @@ class CudaOps:
         out = torch.empty((tokens, hidden), dtype=x.dtype, device=self.device)
         self._call("mlxone_combine_experts", _c_void_p(_ptr(y)), _c_void_p(_ptr(pair_row)),
                    _c_void_p(_ptr(weights)), _c_void_p(_ptr(shared_out)), _c_void_p(_ptr(out)),
-                   _c_int(tokens), _c_int(hidden), _c_int(experts), _c_int(_dtype_code(x.dtype)))
+                   _c_int(tokens), _c_int(hidden), _c_int(experts), _c_int(rows),
+                   _c_int(_dtype_code(x.dtype)))
         return out
 
     # ---- lightning attention
@@ -1076,6 +1140,112 @@ class CudaOps:
         if not (single and value_dim <= 128):
             self.launches += 2
         return out
+
+    def channel_delta_rule(self, projected, decay_up, gate_up, *, decay_columns, gate_columns, conv,
+                           a_log, dt_bias, norm_weight, eps, unit_eps, ctx, view, write, heads,
+                           kv_heads, key_dim, value_dim, taps):
+        """From the fused projection [tokens, q | k | v | beta | ...] to the mixer's gated output
+        [tokens, heads * value_dim]: convolutions with silu, unit-length queries and keys, the
+        recurrence with one decay per head and key channel over each request's tokens on its
+        32-bit state, the output's norm and sigmoid gate. The inner rows of the decay and of the
+        gate are the columns ``decay_columns`` and ``gate_columns`` (first, end) of the
+        projection, ``decay_up`` and ``gate_up`` the matrices applied to them. A step of single
+        tokens is one kernel; else the two products, preparation, scan and finish."""
+        tokens = projected.shape[0]
+        dtype = projected.dtype
+        self._need_rows(projected, dtype, "projected")
+        inner = heads * value_dim
+        for tensor, what in ((conv, "conv"), (a_log, "A_log"), (dt_bias, "dt_bias"),
+                             (norm_weight, "norm weight"), (view.state, "state")):
+            self._need(tensor, torch.float32, what)
+        self._need(decay_up, dtype, "decay_up")
+        self._need(gate_up, dtype, "gate_up")
+        size = self.lib.mlxone_gated_delta_state(heads, kv_heads, key_dim, value_dim, taps)
+        if view.state[0].numel() != size:
+            raise KernelError(f"a state slot has {view.state[0].numel()} values, the mixer needs {size}")
+        ranks = (decay_columns[1] - decay_columns[0], gate_columns[1] - gate_columns[0])
+        if decay_up.shape != (heads * key_dim, ranks[0]) or gate_up.shape != (inner, ranks[1]) or                 max(decay_columns[1], gate_columns[1]) > projected.shape[1]:
+            raise KernelError("the inner rows do not match the matrices applied to them")
+        out = torch.empty((tokens, inner), dtype=dtype, device=self.device)
+        constants = (_c_void_p(_ptr(conv)), _c_void_p(_ptr(a_log)), _c_void_p(_ptr(dt_bias)),
+                     _c_void_p(_ptr(norm_weight)), _c_float(eps), _c_float(unit_eps),
+                     _c_void_p(_ptr(view.state)), _c_void_p(_ptr(view.slots)))
+        sizes = (_c_int(heads), _c_int(kv_heads), _c_int(key_dim), _c_int(value_dim), _c_int(taps),
+                 _c_int(1 if write else 0), _c_int(_dtype_code(dtype)))
+        if (ctx.max_portion == 1 and tokens == ctx.requests and max(ranks) <= 1024
+                and value_dim <= self.lib.mlxone_channel_delta_step_columns()):
+            self._call("mlxone_channel_delta_step", _c_void_p(_ptr(projected)),
+                       _c_int(projected.stride(0)), _c_void_p(_ptr(decay_up)),
+                       _c_int(decay_columns[0]), _c_int(ranks[0]), _c_void_p(_ptr(gate_up)),
+                       _c_int(gate_columns[0]), _c_int(ranks[1]), *constants,
+                       _c_void_p(_ptr(ctx.history)), _c_void_p(_ptr(out)), _c_int(tokens), *sizes)
+            return out
+        # (what enters the recurrence stays in 32-bit behind its product)
+        steps = self.linear(projected[:, slice(*decay_columns)], decay_up, out_dtype=torch.float32)
+        gate = self.linear(projected[:, slice(*gate_columns)], gate_up)
+        scratch = torch.empty(self.lib.mlxone_channel_delta_scratch(tokens, heads, key_dim, value_dim),
+                              dtype=torch.float32, device=self.device)
+        self._call("mlxone_channel_delta", _c_void_p(_ptr(projected)), _c_int(projected.stride(0)),
+                   _c_void_p(_ptr(steps)), _c_void_p(_ptr(gate)), *constants,
+                   _c_void_p(_ptr(ctx.request_start)), _c_void_p(_ptr(ctx.history)),
+                   _c_void_p(_ptr(scratch)), _c_void_p(_ptr(out)), _c_int(tokens),
+                   _c_int(ctx.requests), *sizes)
+        self.launches += 2
+        return out
+
+    # ---- parallel streams
+
+    def read_streams(self, streams, update, read, weight, eps, dtype):
+        """streams float32 [tokens, n, hidden]: applies the pending ``update`` (StreamUpdate:
+        X_t <- sum_s mix[s, t] X_s + out[t] y; None: nothing is pending) in place (into new streams
+        where their number changes), and norms u = sum_t read[t] X_t. Returns (streams, the normed
+        u [tokens, hidden] in ``dtype``). One kernel."""
+        self._need(streams, torch.float32, "streams")
+        self._need(weight, torch.float32, "norm weight")
+        self._need(read, torch.float32, "reading weights")
+        tokens, before, hidden = streams.shape
+        after, y, mix, out = streams, None, None, None
+        if update is not None:
+            y, mix, out = update.output, update.mix, update.out
+            self._need(y, dtype, "a sublayer's output")
+            self._need(mix, torch.float32, "mix")
+            self._need(out, torch.float32, "out")
+            if y.shape != (tokens, hidden) or mix.shape != (before, out.numel()):
+                raise KernelError("an update does not match the streams")
+            if out.numel() != before:
+                after = torch.empty((tokens, out.numel(), hidden), dtype=torch.float32,
+                                    device=self.device)
+        count = after.shape[1]
+        if read.numel() != count or weight.numel() != hidden:
+            raise KernelError("one reading weight per stream, one norm weight per value")
+        normed = torch.empty((tokens, hidden), dtype=dtype, device=self.device)
+        self._call("mlxone_read_streams", _c_void_p(_ptr(streams)), _c_void_p(_ptr(after)),
+                   _c_void_p(_ptr(y)), _c_void_p(_ptr(mix)), _c_void_p(_ptr(out)),
+                   _c_void_p(_ptr(read)), _c_void_p(_ptr(weight)), _c_void_p(_ptr(normed)),
+                   _c_int(tokens), _c_int(before), _c_int(count), _c_int(hidden), _c_float(eps),
+                   _c_int(_dtype_code(dtype)))
+        return after, normed
+
+    def sum_streams(self, streams, update, rows):
+        """float32 [len(rows), hidden]: the streams of the wanted tokens (``rows`` int32; None:
+        all, in order) added up, as they are after the pending ``update``."""
+        self._need(streams, torch.float32, "streams")
+        tokens, before, hidden = streams.shape
+        y = mix = out = None
+        after, code = before, _F32
+        if update is not None:
+            y, mix, out = update.output, update.mix, update.out
+            after, code = out.numel(), _dtype_code(y.dtype)
+            self._need(y, y.dtype, "a sublayer's output")
+        if rows is not None:
+            self._need(rows, torch.int32, "rows")
+        count = tokens if rows is None else rows.numel()
+        total = torch.empty((count, hidden), dtype=torch.float32, device=self.device)
+        self._call("mlxone_sum_streams", _c_void_p(_ptr(streams)), _c_void_p(_ptr(y)),
+                   _c_void_p(_ptr(mix)), _c_void_p(_ptr(out)), _c_void_p(_ptr(rows)),
+                   _c_void_p(_ptr(total)), _c_int(count), _c_int(tokens), _c_int(before),
+                   _c_int(after), _c_int(hidden), _c_int(code))
+        return total
 
     def swiglu(self, gate_up):
         rows, twice = gate_up.shape
