@@ -17,6 +17,8 @@ Two more workloads, each printing one JSON line of its own (the default line is 
 
     python bench.py --case batching     continuous batching of 128 requests at the LFM2-700M shape
     python bench.py --case long         4 x 32,768-token prompts at the LFM2-350M shape, then decoding
+    python bench.py --case susalorn     Susalorn beside Lamisun and Galarax at equal width, depth and
+                                        vocabulary: decode and prefill, and the new kernels alone
     python bench.py --case lamisun      Lamisun beside LFM2 at equal width, depth and vocabulary:
                                         decode and prefill tokens/s, and the new kernels alone
     python bench.py --case tirudra      Tirudra beside Farorax at equal width, depth and vocabulary:
@@ -247,6 +249,9 @@ def model_flops(spec, tokens):
             elif part.kind == "lightning":
                 # 32-bit multiply-adds of the recurrence (not tensor-core work, but work)
                 flops += 4 * tokens * part["heads"] * part["key_dim"] * part["value_dim"]
+            elif part.kind == "channel_delta":
+                # 32-bit multiply-adds of the recurrence (not tensor-core work, but work)
+                flops += 6 * tokens * part["heads"] * part["key_dim"] * part["value_dim"]
             elif part.kind == "mamba2":
                 flops += 4 * tokens * part["heads"] * part["state"] * part["value_dim"]
     return flops
@@ -1662,6 +1667,258 @@ def case_lamisun(args) -> int:
     return 0
 
 
+# --------------------------------------------------------------------------- Susalorn beside Lamisun and Galarax
+
+
+def susalorn_shape(width: int, layers: int, vocab: int = 65536) -> dict:
+    """A Susalorn of the sizes that a model of this width has: layers in turn with attention over
+    latent rows (heads of 64 unrotated + a rotated part shared by the heads, a latent of a quarter
+    of the width, queries through a latent of half the width) and the channel-wise delta rule
+    (heads of 128 x 128, inner width = model width, inner sizes of 128), four streams, 16 experts
+    of half the width of which a token uses 4 (four groups, two kept)."""
+    rot_dim, latent = (32, 256) if width <= 1024 else (64, 512)
+    first = {"heads": width // 64, "dim": 64, "rot_dim": rot_dim, "vdim": 64, "kv_rank": latent,
+             "q_rank": width // 2, "scale": (64 + rot_dim) ** -0.5,
+             "rot": {"base": 10000.0, "dims": rot_dim,
+                     "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    second = {"heads": width // 128, "kv_heads": width // 256, "dim": 128, "vdim": 128, "conv": 4,
+              "decay_rank": 128, "gate_rank": 128}
+    moe = {"kind": "moe", "expert": {"ff": width // 2},
+           "router": {"experts": 16, "top": 4, "groups": {"count": 4, "keep": 2}, "scale": 2.0}}
+    entries = [{"type": "channel_delta", "mixer": second, "mlp": moe} if index % 2 else
+               {"type": "latent_attention", "mixer": first, "mlp": moe} for index in range(layers)]
+    return {"architecture": "Susalorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "streams": 4, "layers": entries}
+
+
+def susalorn_kernels(width, batch, peak):
+    """The kernels that Susalorn adds, alone, beside the like kernels of Lamisun, Galarax and
+    Farorax, for a decode step of ``batch`` tokens over 2,048 earlier ones and a prompt of
+    PREFILL_TOKENS tokens: algorithmic bytes (or flops) / time against the measured peaks.
+    Arguments rotate over copies that together exceed L2."""
+    import torch
+
+    from mlx_one_b200.kernels import default_ops
+    from mlx_one_b200.parts import (FixedState, PagedKeyValues, PagedView, StateView,
+                                    StepContext, StreamUpdate)
+    from mlx_one_b200.parts.mixers import GatedDeltaRule
+
+    ops, device = default_ops("cuda:0"), "cuda:0"
+    ints = lambda values: torch.tensor(values, dtype=torch.int32, device=device)
+    bf16 = lambda *shape: torch.randn(*shape, device=device).bfloat16()
+
+    def ctx_of(portions, histories):
+        positions, owner, starts = [], [], [0]
+        for r, (n, before) in enumerate(zip(portions, histories)):
+            positions += list(range(before, before + n))
+            owner += [r] * n
+            starts.append(starts[-1] + n)
+        return StepContext(tokens=len(positions), requests=len(portions),
+                           token_ids=ints([0] * len(positions)), positions=ints(positions),
+                           token_request=ints(owner), request_start=ints(starts),
+                           history=ints(histories), max_portion=max(portions),
+                           max_context=max(p + h for p, h in zip(portions, histories)))
+
+    def entry(seconds, moved=None, flops=None):
+        out = {"us": round(seconds * 1e6, 2)}
+        if moved is not None:
+            out["gbs"] = round(moved / seconds / 1e9, 1)
+            out["hbm_frac"] = round(moved / seconds / 1e9 / peak["hbm_gbs"], 4)
+        if flops is not None:
+            out["tflops"] = round(flops / seconds / 1e12, 2)
+            out["tensor_frac"] = round(flops / seconds / 1e12 / peak["bf16_tflops"], 4)
+        return out
+
+    shape = susalorn_shape(width, 2)
+    first, second = shape["layers"][0]["mixer"], shape["layers"][1]["mixer"]
+    streams = shape["streams"]
+    out = {}
+    for label, portions, histories in (("decode", [1] * batch, [2048] * batch),
+                                       ("prefill", [PREFILL_TOKENS], [0])):
+        ctx = ctx_of(portions, histories)
+        tokens, requests = ctx.tokens, ctx.requests
+        # ---- between two sublayers: four streams written and read, beside add + norm of one
+        copies = 4
+        many = [torch.zeros(tokens, streams, width, device=device) for _ in range(copies)]
+        delta = [bf16(tokens, width) for _ in range(copies)]
+        vector, ones = torch.ones(width, device=device), torch.ones(streams, device=device)
+        mix = torch.eye(streams, device=device)
+        seconds = graph_seconds(lambda i: ops.read_streams(
+            many[i], StreamUpdate(delta[i], mix, ones), ones, vector, 1e-6, torch.bfloat16), copies, 2 * copies)
+        out[f"{label}_read_streams_4"] = entry(seconds, tokens * width * (8 * streams + 2 + 2))
+        seconds = graph_seconds(lambda i: ops.add_rmsnorm(
+            many[i].view(-1, width)[:tokens], delta[i], vector, 1e-6, torch.bfloat16), copies, 2 * copies)
+        out[f"{label}_add_rmsnorm"] = entry(seconds, tokens * width * (4 + 4 + 2 + 2))
+        del many, delta
+        # ---- the delta rule: a decay per key channel beside one per head (Galarax)
+        H, G, D, V, taps = second["heads"], second["kv_heads"], 128, 128, second["conv"]
+        rank = second["decay_rank"]
+        sizes = dict(heads=H, kv_heads=G, key_dim=D, value_dim=V, taps=taps)
+        state_size = GatedDeltaRule.state_size({"heads": H, "kv_heads": G, "key_dim": D,
+                                                "value_dim": V, "taps": taps})
+        channels = 2 * G * D + H * V
+        base = channels + H + -H % 8
+        copies = max(2, min(24, int(200e6 // (requests * state_size * 4))))
+        state = torch.zeros(copies * requests, state_size, device=device)
+        views = [StateView(state, ints(list(range(c * requests, (c + 1) * requests))),
+                           FixedState((state_size,), "float32")) for c in range(copies)]
+        projected = [bf16(tokens, base + 2 * rank) for _ in range(copies)]
+        common = dict(conv=torch.randn(channels, taps, device=device) * 0.5,
+                      a_log=torch.zeros(H, device=device), norm_weight=torch.ones(V, device=device),
+                      eps=1e-6, unit_eps=1e-6, ctx=ctx, write=True, **sizes)
+        ups = [(bf16(H * D, rank) * 0.1, bf16(H * V, rank) * 0.1) for _ in range(copies)]
+        dt_bias = torch.zeros(H * D, device=device)
+        seconds = graph_seconds(lambda i: ops.channel_delta_rule(
+            projected[i], *ups[i], decay_columns=(base, base + rank),
+            gate_columns=(base + rank, base + 2 * rank), dt_bias=dt_bias, view=views[i], **common),
+            copies, 2 * copies)
+        moved = tokens * (base + 2 * rank + H * V) * 2 + 2 * requests * state_size * 4 + 2 * H * D * rank * 2
+        out[f"{label}_channel_delta"] = entry(seconds, moved)
+        out[f"{label}_channel_delta"]["gflops"] = round(6.0 * tokens * H * D * V / seconds / 1e9, 1)
+        wide = [bf16(tokens, channels + H * V + 2 * H) for _ in range(copies)]
+        step_bias = torch.zeros(H, device=device)
+        seconds = graph_seconds(lambda i: ops.gated_delta_rule(
+            wide[i], dt_bias=step_bias, view=views[i], **common), copies, 2 * copies)
+        moved = tokens * (channels + 2 * H * V + 2 * H) * 2 + 2 * requests * state_size * 4
+        out[f"{label}_gated_delta_galarax"] = entry(seconds, moved)
+        out[f"{label}_gated_delta_galarax"]["gflops"] = round(6.0 * tokens * H * D * V / seconds / 1e9, 1)
+        del state, views, projected, wide, ups
+        # ---- attention over latent rows: preparation in two steps beside Lamisun's one, then
+        # attention with and without sinks
+        heads, nope, rot, latent = first["heads"], first["dim"], first["rot_dim"], first["kv_rank"]
+        row, query_rank, copies = latent + rot, first["q_rank"], 8
+        span = histories[0] + portions[0]
+        pages = -(-span // PAGE_SIZE)
+        blocks = ints([[r * pages + b for b in range(pages)] for r in range(requests)])
+        rows = (torch.randn(1, requests * pages + 1, 1, PAGE_SIZE, row, device=device) * 0.3).bfloat16()
+        view = PagedView(rows, blocks, PAGE_SIZE, PagedKeyValues(1, row, planes=1))
+        rotary = (torch.rand(rot // 2, device=device), rot)
+        small = [bf16(tokens, query_rank + row) for _ in range(copies)]
+        q = [bf16(tokens, heads * (nope + rot)) for _ in range(copies)]
+        queries = [bf16(tokens, heads, row) * 0.3 for _ in range(copies)]
+        both = [bf16(tokens, heads * (nope + rot) + row) for _ in range(copies)]
+        norm_q, norm_c = torch.ones(query_rank, device=device), torch.ones(latent, device=device)
+        turn = dict(rot_dim=rot, latent=latent, rotary=rotary, neighbours=False, ctx=ctx)
+
+        def two_steps(i):
+            ops.latent_rows(small[i], rank=query_rank, query_norm=norm_q, norm_weight=norm_c, eps=1e-6,
+                            view=view, write=True, amplitude=1.2, **turn)
+            ops.latent_queries(q[i], queries[i], heads=heads, head_dim=nope, amplitude=1.2, **turn)
+
+        seconds = graph_seconds(two_steps, copies, 2 * copies)
+        out[f"{label}_latent_rows_queries"] = entry(
+            seconds, tokens * (query_rank + heads * rot + row) * 2 * 2)
+        seconds = graph_seconds(lambda i: ops.latent_prepare(
+            both[i], queries[i], heads=heads, head_dim=nope, norm_weight=norm_c, eps=1e-6, view=view,
+            write=True, **turn), copies, 2 * copies)
+        out[f"{label}_latent_prepare_lamisun"] = entry(seconds, tokens * (heads * rot + row) * 2 * 2)
+        seen = sum(h + i + 1 for n, h in zip(portions, histories) for i in range(n))
+        sinks = torch.zeros(heads, device=device)
+        for name, extra in (("latent_attention_sinks", dict(sinks=sinks)), ("latent_attention_lamisun", {})):
+            seconds = graph_seconds(lambda i: ops.latent_attention(
+                queries[i], heads=heads, latent=latent, scale=first["scale"], ctx=ctx, view=view, **extra),
+                copies, 2 * copies)
+            out[f"{label}_{name}"] = entry(
+                seconds, requests * span * row * 2 + tokens * heads * row * 2 * 2,
+                2.0 * heads * (row + latent) * seen)
+        del rows, small, q, queries, both
+        # ---- routed experts without gates beside gated ones (Farorax), equal experts and top
+        mlp = shape["layers"][0]["mlp"]
+        experts, top, ff = mlp["router"]["experts"], mlp["router"]["top"], mlp["expert"]["ff"]
+        stack = experts * ff
+        copies = max(2, min(8, int(300e6 // (stack * width * 6))))
+        gate_up = [bf16(2 * stack, width) * 0.02 for _ in range(copies)]
+        down = [bf16(width, stack) * 0.02 for _ in range(copies)]
+        x, router = bf16(tokens, width), torch.randn(experts, width, device=device)
+
+        def plain_experts(i):
+            weights, _ = ops.route_general(x, router, None, experts=experts, identity=0, top=top,
+                                           scores="softmax", normalize=True, shared_gate=False, groups=4,
+                                           keep=2, group_score=1, scale=2.0)
+            up = gate_up[i][:stack]
+            if ops.sorts_experts(x, experts=experts, width=ff, top=top, stack=stack):
+                return ops.routed_experts_sorted(x, weights, up, down[i], experts=experts, width=ff,
+                                                 top=top, activation="relu2")
+            hidden = ops.linear_act(x, up, "relu2")
+            ops.scale_expert_columns(hidden, weights, ff)
+            return ops.linear(hidden, down[i])
+
+        def gated_experts(i):
+            weights = ops.route_experts(x, router, experts=experts, top=top, groups=4, keep=2, group_score=2)
+            if ops.sorts_experts(x, experts=experts, width=ff, top=top, stack=stack):
+                return ops.routed_experts_sorted(x, weights, gate_up[i], down[i], experts=experts,
+                                                 width=ff, top=top)
+            hidden = ops.linear_swiglu(x, gate_up[i])
+            ops.scale_expert_columns(hidden, weights, ff)
+            return ops.linear(hidden, down[i])
+
+        touched = min(experts, tokens * top) * ff
+        for name, fn, matrices in (("routed_ff", plain_experts, 2), ("routed_ff_farorax", gated_experts, 3)):
+            seconds = graph_seconds(fn, copies, 2 * copies)
+            out[f"{label}_{name}"] = entry(
+                seconds, touched * width * 2 * matrices if label == "decode" else None,
+                2.0 * matrices * tokens * top * ff * width if label == "prefill" else None)
+        for name, fn in (("route_general", lambda i: ops.route_general(
+                x, router, None, experts=experts, identity=0, top=top, scores="softmax", normalize=True,
+                shared_gate=False, groups=4, keep=2, group_score=1, scale=2.0)),
+                         ("route_experts_farorax", lambda i: ops.route_experts(
+                             x, router, experts=experts, top=top, groups=4, keep=2, group_score=2))):
+            out[f"{label}_{name}"] = entry(graph_seconds(fn, copies, 2 * copies), tokens * width * 2)
+        del gate_up, down
+        torch.cuda.empty_cache()
+    return out
+
+
+def case_susalorn(args) -> int:
+    """Susalorn beside Lamisun (attention over latent rows) and Galarax (the delta rule), the
+    closest of the engine's models, at equal width, depth and vocabulary, random weights: decode
+    tokens/s at ``--batch`` and ``--context`` (device-timed graph replays of the engine's step),
+    prefill tokens/s of one 2,048-token prompt, each against its bound, and the new kernels alone."""
+    import gc
+
+    import torch
+
+    peak = peaks()
+    warmup, steps = max(args.warmup, 3), min(args.steps, 128)
+    context = args.context or 2048
+    layers = min(args.layers, 8)
+    results = {}
+    for width in (1024, 2048):
+        for label, data in ((f"susalorn_w{width}", susalorn_shape(width, layers)),
+                            (f"lamisun_w{width}", lamisun_shape(width, layers)),
+                            (f"galarax_w{width}", galarax_shape(width, layers))):
+            engine = engine_of(data, args.batch, context, warmup + steps, f"random-{label}")
+            model, spec = engine.model, engine.model.spec
+            weight_bytes = model.weight_bytes()
+            kv_per_token = engine.cache_bytes_per_token()
+            state_bytes = sum(g.storage[:, 0].numel() * g.storage.element_size()
+                              for g in engine.cache.states)
+            seconds, _, mean_context, launches = time_decode(engine, args.batch, context, warmup,
+                                                             steps, seed=3)
+            step_bytes = weight_bytes + args.batch * (mean_context * kv_per_token + 2 * state_bytes)
+            prefill_seconds = time_prefill(engine, PREFILL_TOKENS, 2, 3, seed=5)
+            flops = model_flops(spec, PREFILL_TOKENS)
+            results[label] = {
+                "layers": layers, "weight_mb": round(weight_bytes / 1e6, 1),
+                "state_mb_per_request": round(state_bytes / 1e6, 2),
+                "decode_tokens_per_s": round(args.batch * steps / seconds, 1),
+                "decode_ms_per_step": round(seconds / steps * 1e3, 4),
+                "decode_hbm_frac": round(step_bytes / (seconds / steps) / 1e9 / peak["hbm_gbs"], 4),
+                "launches_per_step": launches,
+                "prefill_tokens_per_s": round(PREFILL_TOKENS / prefill_seconds, 1),
+                "prefill_ms": round(prefill_seconds * 1e3, 3),
+                "prefill_tensor_frac": round(flops / prefill_seconds / (peak["bf16_tflops"] * 1e12), 4)}
+            del engine, model
+            gc.collect()
+            torch.cuda.empty_cache()
+        results[f"kernels_w{width}"] = susalorn_kernels(width, args.batch, peak)
+    print(json.dumps({"case": "susalorn", "batch": args.batch, "context": context, "steps": steps,
+                      "warmup": warmup, "dtype": "bf16", "peaks": peak["source"],
+                      "data": "synthetic: random weights, seeded uniform-random token ids",
+                      "results": results}))
+    return 0
+
+
 def decode_step_case(batch: int, context: int) -> int:
     """A few eager decode steps of the whole model at the benchmark's sizes, for a list of the
     step's launches (`ncu --metrics gpu__time_duration.sum`): the prompts are fed first, the last
@@ -2070,7 +2327,8 @@ def main() -> int:
     parser.add_argument("--batch", type=int, default=8)
     parser.add_argument("--context", type=int, default=None,
                         help="context length (default 4096; --case long: prompt tokens, 32768)")
-    parser.add_argument("--case", default="decode", choices=["decode", "batching", "long", "galarax", "farorax", "lamisun", "tirudra"],
+    parser.add_argument("--case", default="decode", choices=["decode", "batching", "long", "galarax", "farorax", "lamisun",
+                                                               "tirudra", "susalorn"],
                         help="decode: the default line; batching: 128 requests batched "
                              "continuously (LFM2-700M shape); long: 4 x 32,768 tokens "
                              "(LFM2-350M shape)")
@@ -2106,6 +2364,8 @@ def main() -> int:
         return case_farorax(args)
     if args.case == "lamisun":
         return case_lamisun(args)
+    if args.case == "susalorn":
+        return case_susalorn(args)
     if args.case == "tirudra":
         return case_tirudra(args)
     args.context = args.context or 4096

@@ -22,9 +22,9 @@
 //   prepare  per (eight tokens, query/key head): convolutions + silu, unit lengths (q also times
 //            D^-1/2), decays; c_j * k_j, c_j * q_j, g_(j+1) ... g_8 * k_j, c_8, M and Q.
 //   scan     per (request, value head, tile of columns of S): a column of S depends on no other
-//            column. A thread keeps PER rows of four columns, LANES threads share the rows; the
-//            sums over the rows of all eight tokens and four columns are taken together (each
-//            exchange of the butterfly halves what a lane carries), u, o and the update follow.
+//            column. A thread keeps PER rows of two columns, LANES threads share the rows
+//            (products on pairs of rows, two multiply-adds an instruction); the sums over the rows
+//            of all eight tokens and both columns are taken together (each exchange of the butterfly halves what a lane carries), u, o and the update follow.
 //            The operands of the next 16 tokens travel to shared memory (cp.async) while the
 //            current 16 are worked on. Extra blocks write the convolution's inputs into the ring.
 //   finish   per (token, head): o / rms(o) * weight * sigmoid(gate), in the compute type.
@@ -37,14 +37,35 @@ namespace {
 
 constexpr int GROUP = 8;             // tokens worked on together
 constexpr int PREP_THREADS = 128;
-constexpr int SCAN_THREADS = 128;
+constexpr int SCAN_THREADS = 256;
 constexpr int CHUNK = 16;            // tokens whose operands are staged in shared memory together
-constexpr int COLS = 4;              // columns of S per thread of the scan
+constexpr int COLS = 2;              // columns of S per thread of the scan
 constexpr int PAIRS = GROUP * COLS;
 constexpr int SOLVE = 2 * GROUP * GROUP;    // M, then Q, both [GROUP][GROUP]
 constexpr int STEP_LANES = 4;        // single-token kernel: lanes that share a column of S
 constexpr int STEP_MAX_COLUMNS = 128;
 constexpr int STEP_ROWS = 16;        // rows of the second matrices that a warp holds in registers
+
+// Two 32-bit numbers in one register pair.
+using Pair = unsigned long long;
+__device__ __forceinline__ Pair pair_of(float lo, float hi) {
+    Pair p;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(p) : "f"(lo), "f"(hi));
+    return p;
+}
+__device__ __forceinline__ void halves(Pair p, float& lo, float& hi) {
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(p));
+}
+__device__ __forceinline__ Pair pair_fma(Pair a, Pair b, Pair c) {
+    Pair d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ Pair pair_mul(Pair a, Pair b) {
+    Pair d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
 
 __device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
 
@@ -110,12 +131,19 @@ __device__ __forceinline__ void convolve(const T* projected, int ld, const float
         float in[GROUP + TAPS - 1], w[TAPS > 0 ? TAPS : 1];
 #pragma unroll
         for (int j = 0; j < TAPS; ++j) w[j] = conv[(size_t)c * TAPS + j];
+        if (index >= TAPS - 1 && count == GROUP) {
+            // all inputs are rows of this step: one round trip for all of them
+            const T* row = projected + (size_t)(t0 - (TAPS - 1)) * ld + c;
 #pragma unroll
-        for (int i = 0; i < GROUP + TAPS - 1; ++i) {
-            const int place = i - (TAPS - 1);
-            in[i] = place < count
-                ? conv_input<T>(projected, ld, ring, channels, TAPS, t0, index, position, -place, c)
-                : 0.f;
+            for (int i = 0; i < GROUP + TAPS - 1; ++i) in[i] = to_float<T>(row[(size_t)i * ld]);
+        } else {
+#pragma unroll
+            for (int i = 0; i < GROUP + TAPS - 1; ++i) {
+                const int place = i - (TAPS - 1);
+                in[i] = place < count
+                    ? conv_input<T>(projected, ld, ring, channels, TAPS, t0, index, position, -place, c)
+                    : 0.f;
+            }
         }
 #pragma unroll
         for (int j = 0; j < GROUP; ++j) {
@@ -144,7 +172,7 @@ __device__ __forceinline__ void convolve(const T* projected, int ld, const float
 // group's first token: cum [tokens, H, D] (c_8) and solve [tokens, H, SOLVE] (M and Q, row j: what
 // token j takes of token i). Dynamic shared memory: q and k [GROUP][D].
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(PREP_THREADS)
+__global__ void __launch_bounds__(PREP_THREADS, 4)
 channel_prepare_kernel(const T* __restrict__ projected, const float* __restrict__ steps,
                        const float* __restrict__ conv, const float* __restrict__ a_log,
                        const float* __restrict__ dt_bias, const float* __restrict__ state,
@@ -207,12 +235,13 @@ channel_prepare_kernel(const T* __restrict__ projected, const float* __restrict_
             float decay[GROUP], k[GROUP], q[GROUP];
             const float bias = dt_bias[h * D + d];
 #pragma unroll
+            for (int j = 0; j < GROUP; ++j)
+                decay[j] = steps[((size_t)(t0 + min(j, count - 1)) * H + h) * D + d];
+#pragma unroll
             for (int j = 0; j < GROUP; ++j) {
                 k[j] = keys[j * D + d];
                 q[j] = qs[j * D + d];
-                decay[j] = 1.f;
-                if (j < count)
-                    decay[j] = expf(rate * softplus(steps[((size_t)(t0 + j) * H + h) * D + d] + bias));
+                decay[j] = j < count ? expf(rate * softplus(decay[j] + bias)) : 1.f;
             }
             float before = 1.f;
 #pragma unroll
@@ -312,7 +341,7 @@ struct ScanShape {
 };
 
 template <typename T, int PER, int LANES>
-__global__ void __launch_bounds__(SCAN_THREADS)
+__global__ void __launch_bounds__(SCAN_THREADS, 1)
 channel_scan_kernel(const float* __restrict__ kc, const float* __restrict__ qc,
                     const float* __restrict__ ks, const float* __restrict__ v_in,
                     const float* __restrict__ cum, const float* __restrict__ solve,
@@ -322,7 +351,11 @@ channel_scan_kernel(const float* __restrict__ kc, const float* __restrict__ qc,
                     int write, int ld) {
     using Shape = ScanShape<PER, LANES>;
     constexpr int ROWS = Shape::ROWS, COLUMNS = Shape::COLUMNS, BUFFER = Shape::BUFFER;
-    constexpr int OWN = PAIRS / LANES;                // (column, token) pairs a lane finishes
+    // What a lane holds after the sums: with 32 lanes one of the 32 values, a of (column, token)
+    // pair l in the lower half of the warp and b of pair l - 16 in the upper; with fewer lanes a and
+    // b of OWN pairs.
+    constexpr bool SPLIT = LANES == 2 * PAIRS;
+    constexpr int OWN = SPLIT ? 1 : PAIRS / LANES;
     extern __shared__ __align__(16) float staged[];
     griddep_wait();
     kc = settled(kc);
@@ -355,14 +388,15 @@ channel_scan_kernel(const float* __restrict__ kc, const float* __restrict__ qc,
     const int lane = threadIdx.x & (LANES - 1), team = threadIdx.x / LANES;
     const int column0 = blockIdx.x * COLUMNS + team * COLS;
     float* matrix = slot + (size_t)h * D * V;
-    float S[COLS][PER];
+    Pair S[COLS][PER / 2];                            // rows 2 e and 2 e + 1 of this lane's
+    auto stored = [&](int c, int e) {
+        const int row = lane * PER + e;
+        return column0 + c < V && row < D ? matrix[(size_t)row * V + column0 + c] : 0.f;
+    };
 #pragma unroll
-    for (int e = 0; e < PER; ++e)
+    for (int e = 0; e < PER; e += 2)
 #pragma unroll
-        for (int c = 0; c < COLS; ++c) {
-            const int row = lane * PER + e;
-            S[c][e] = column0 + c < V && row < D ? matrix[(size_t)row * V + column0 + c] : 0.f;
-        }
+        for (int c = 0; c < COLS; ++c) S[c][e / 2] = pair_of(stored(c, e), stored(c, e + 1));
     const bool quads = D % 4 == 0 && ((reinterpret_cast<uintptr_t>(kc) | reinterpret_cast<uintptr_t>(qc) |
                                        reinterpret_cast<uintptr_t>(ks) | reinterpret_cast<uintptr_t>(cum)) & 15) == 0;
     const bool value_quads = V % 4 == 0 && (reinterpret_cast<uintptr_t>(v_in) & 15) == 0;
@@ -420,39 +454,46 @@ channel_scan_kernel(const float* __restrict__ kc, const float* __restrict__ qc,
         const float* solves = cums + (CHUNK / GROUP) * ROWS;
         const float* vs = solves + (CHUNK / GROUP) * SOLVE;
         for (int t0 = 0; t0 < count; t0 += GROUP) {
-            // a and b of every (column, token): value (c * GROUP + j) * 2 (+ 1 for b)
+            // a and b of every (column, token) pair c * GROUP + j
             float sum[2 * PAIRS];
 #pragma unroll
-            for (int i = 0; i < 2 * PAIRS; ++i) sum[i] = 0.f;
-#pragma unroll
             for (int j = 0; j < GROUP; ++j) {
+                Pair a[COLS], b[COLS];
 #pragma unroll
                 for (int e = 0; e < PER; e += 4) {
-                    const float4 k4 = *reinterpret_cast<const float4*>(kcs + (t0 + j) * ROWS + lane * PER + e);
-                    const float4 q4 = *reinterpret_cast<const float4*>(qcs + (t0 + j) * ROWS + lane * PER + e);
+                    const ulonglong2 k4 = *reinterpret_cast<const ulonglong2*>(kcs + (t0 + j) * ROWS + lane * PER + e);
+                    const ulonglong2 q4 = *reinterpret_cast<const ulonglong2*>(qcs + (t0 + j) * ROWS + lane * PER + e);
 #pragma unroll
                     for (int c = 0; c < COLS; ++c) {
-                        float& a = sum[(c * GROUP + j) * 2];
-                        float& b = sum[(c * GROUP + j) * 2 + 1];
-                        a = fmaf(S[c][e], k4.x, a); b = fmaf(S[c][e], q4.x, b);
-                        a = fmaf(S[c][e + 1], k4.y, a); b = fmaf(S[c][e + 1], q4.y, b);
-                        a = fmaf(S[c][e + 2], k4.z, a); b = fmaf(S[c][e + 2], q4.z, b);
-                        a = fmaf(S[c][e + 3], k4.w, a); b = fmaf(S[c][e + 3], q4.w, b);
+                        a[c] = e == 0 ? pair_mul(S[c][0], k4.x) : pair_fma(S[c][e / 2], k4.x, a[c]);
+                        b[c] = e == 0 ? pair_mul(S[c][0], q4.x) : pair_fma(S[c][e / 2], q4.x, b[c]);
+                        a[c] = pair_fma(S[c][e / 2 + 1], k4.y, a[c]);
+                        b[c] = pair_fma(S[c][e / 2 + 1], q4.y, b[c]);
                     }
+                }
+#pragma unroll
+                for (int c = 0; c < COLS; ++c) {
+                    const int pair = c * GROUP + j;
+                    float lo, hi;
+                    halves(a[c], lo, hi);
+                    sum[SPLIT ? pair : 2 * pair] = lo + hi;
+                    halves(b[c], lo, hi);
+                    sum[SPLIT ? PAIRS + pair : 2 * pair + 1] = lo + hi;
                 }
             }
             reduce_many<2 * PAIRS, LANES>(sum, lane);
-            // this lane's pairs: lane * OWN + i, pair = c * GROUP + j
             const float* solve_group = solves + (t0 / GROUP) * SOLVE;
+            const int first_pair = SPLIT ? lane % PAIRS : lane * OWN;
 #pragma unroll
             for (int i = 0; i < OWN; ++i) {
-                const int pair = lane * OWN + i, c = pair / GROUP, j = pair % GROUP;
-                own[pair] = vs[(t0 + j) * COLUMNS + team * COLS + c] - sum[2 * i];
+                const int pair = first_pair + i, c = pair / GROUP, j = pair % GROUP;
+                if (!SPLIT || lane < PAIRS)
+                    own[pair] = vs[(t0 + j) * COLUMNS + team * COLS + c] - sum[2 * i];
             }
             __syncwarp();
 #pragma unroll
             for (int i = 0; i < OWN; ++i) {
-                const int pair = lane * OWN + i, c = pair / GROUP, j = pair % GROUP;
+                const int pair = first_pair + i, c = pair / GROUP, j = pair % GROUP;
                 float u = 0.f;
 #pragma unroll
                 for (int l = 0; l < GROUP; l += 4) {
@@ -461,13 +502,13 @@ channel_scan_kernel(const float* __restrict__ kc, const float* __restrict__ qc,
                     u = fmaf(m.x, w.x, u); u = fmaf(m.y, w.y, u);
                     u = fmaf(m.z, w.z, u); u = fmaf(m.w, w.w, u);
                 }
-                own[PAIRS + pair] = u;
+                if (!SPLIT || lane < PAIRS) own[PAIRS + pair] = u;
             }
             __syncwarp();
 #pragma unroll
             for (int i = 0; i < OWN; ++i) {
-                const int pair = lane * OWN + i, c = pair / GROUP, j = pair % GROUP;
-                float o = sum[2 * i + 1];
+                const int pair = first_pair + i, c = pair / GROUP, j = pair % GROUP;
+                float o = sum[SPLIT ? 0 : 2 * i + 1];
 #pragma unroll
                 for (int l = 0; l < GROUP; l += 4) {
                     const float4 m = *reinterpret_cast<const float4*>(solve_group + GROUP * GROUP + j * GROUP + l);
@@ -475,37 +516,37 @@ channel_scan_kernel(const float* __restrict__ kc, const float* __restrict__ qc,
                     o = fmaf(m.x, w.x, o); o = fmaf(m.y, w.y, o);
                     o = fmaf(m.z, w.z, o); o = fmaf(m.w, w.w, o);
                 }
-                if (t0 + j < count && column0 + c < V)
+                if ((!SPLIT || lane >= PAIRS) && t0 + j < count && column0 + c < V)
                     out[((size_t)(base + t0 + j) * H + h) * V + column0 + c] = o;
             }
             // S = c_8 * S + sum_j (g_(j+1) ... g_8 * k_j) u_j
 #pragma unroll
             for (int e = 0; e < PER; e += 4) {
-                const float4 c4 = *reinterpret_cast<const float4*>(cums + (t0 / GROUP) * ROWS + lane * PER + e);
+                const ulonglong2 c4 = *reinterpret_cast<const ulonglong2*>(cums + (t0 / GROUP) * ROWS + lane * PER + e);
 #pragma unroll
                 for (int c = 0; c < COLS; ++c) {
-                    S[c][e] *= c4.x; S[c][e + 1] *= c4.y; S[c][e + 2] *= c4.z; S[c][e + 3] *= c4.w;
+                    S[c][e / 2] = pair_mul(S[c][e / 2], c4.x);
+                    S[c][e / 2 + 1] = pair_mul(S[c][e / 2 + 1], c4.y);
                 }
             }
 #pragma unroll
             for (int j = 0; j < GROUP; j += 4) {
-                float u[COLS][4];
+                Pair u[COLS][4];
 #pragma unroll
                 for (int c = 0; c < COLS; ++c) {
                     const float4 w = *reinterpret_cast<const float4*>(own + PAIRS + c * GROUP + j);
-                    u[c][0] = w.x; u[c][1] = w.y; u[c][2] = w.z; u[c][3] = w.w;
+                    u[c][0] = pair_of(w.x, w.x); u[c][1] = pair_of(w.y, w.y);
+                    u[c][2] = pair_of(w.z, w.z); u[c][3] = pair_of(w.w, w.w);
                 }
 #pragma unroll
                 for (int step = 0; step < 4; ++step) {
 #pragma unroll
                     for (int e = 0; e < PER; e += 4) {
-                        const float4 k4 = *reinterpret_cast<const float4*>(kss + (t0 + j + step) * ROWS + lane * PER + e);
+                        const ulonglong2 k4 = *reinterpret_cast<const ulonglong2*>(kss + (t0 + j + step) * ROWS + lane * PER + e);
 #pragma unroll
                         for (int c = 0; c < COLS; ++c) {
-                            S[c][e] = fmaf(k4.x, u[c][step], S[c][e]);
-                            S[c][e + 1] = fmaf(k4.y, u[c][step], S[c][e + 1]);
-                            S[c][e + 2] = fmaf(k4.z, u[c][step], S[c][e + 2]);
-                            S[c][e + 3] = fmaf(k4.w, u[c][step], S[c][e + 3]);
+                            S[c][e / 2] = pair_fma(k4.x, u[c][step], S[c][e / 2]);
+                            S[c][e / 2 + 1] = pair_fma(k4.y, u[c][step], S[c][e / 2 + 1]);
                         }
                     }
                 }
@@ -517,11 +558,14 @@ channel_scan_kernel(const float* __restrict__ kc, const float* __restrict__ qc,
     griddep_launch();
     if (write) {
 #pragma unroll
-        for (int e = 0; e < PER; ++e)
+        for (int e = 0; e < PER; e += 2)
 #pragma unroll
             for (int c = 0; c < COLS; ++c) {
                 const int row = lane * PER + e;
-                if (column0 + c < V && row < D) matrix[(size_t)row * V + column0 + c] = S[c][e];
+                float lo, hi;
+                halves(S[c][e / 2], lo, hi);
+                if (column0 + c < V && row < D) matrix[(size_t)row * V + column0 + c] = lo;
+                if (column0 + c < V && row + 1 < D) matrix[(size_t)(row + 1) * V + column0 + c] = hi;
             }
     }
 }
