@@ -160,11 +160,10 @@ def delta_recurrence(q, k, v, beta, decay):
     out = torch.zeros_like(v)
     S = torch.zeros(H, D, v.shape[2], dtype=v.dtype)
     for t in range(T):
-        for n in range(H):
-            s = S[n] * decay[t, n][:, None]
-            u = beta[t, n] * (v[t, n] - s.T @ k[t, n])
-            S[n] = s + torch.outer(k[t, n], u)
-            out[t, n] = S[n].T @ q[t, n]
+        S = S * decay[t][:, :, None]
+        u = beta[t][:, None] * (v[t] - (S * k[t][:, :, None]).sum(1))
+        S = S + k[t][:, :, None] * u[:, None, :]
+        out[t] = (S * q[t][:, :, None]).sum(1)
     return out
 
 
@@ -189,18 +188,20 @@ MIXERS = {"latent_attention": latent_attention, "channel_delta": channel_delta}
 # --------------------------------------------------------------------------- feed-forwards
 
 
-def dense(h, w, m, prefix):
+def dense(h, w, m, prefix, margins=None):
     return (silu(h @ w[prefix + "gate"].T) * (h @ w[prefix + "up"].T)) @ w[prefix + "down"].T
 
 
-def route(logits, router):
+def route(logits, router, margins=None):
     """Weights [T, experts]: softmax over all experts, the best groups by their largest score, the
-    best experts among theirs, normalised and scaled."""
+    best experts among theirs, normalised and scaled. ``margins``: a list that receives, per
+    token, by how much (in logits) the choice of groups and experts was made."""
     T, E = logits.shape
     scores = torch.softmax(logits, -1)
     groups = router.get("groups") or {"count": 1, "keep": 1}
     size = E // groups["count"]
     out = torch.zeros_like(scores)
+    margin = torch.full((T,), float("inf"), dtype=torch.float64)
     for t in range(T):
         best = [max(float(scores[t, g * size + i]) for i in range(size)) for g in range(groups["count"])]
         kept = sorted(range(groups["count"]), key=lambda g: (-best[g], g))[:groups["keep"]]
@@ -209,11 +210,21 @@ def route(logits, router):
         total = sum(scores[t, e] for e in chosen) + 1e-20
         for e in chosen:
             out[t, e] = scores[t, e] / total * router.get("scale", 1.0)
+        worst = min(math.log(best[g] + 1e-300) for g in kept)
+        for g in range(len(best)):
+            if g not in kept:
+                margin[t] = min(float(margin[t]), worst - math.log(best[g] + 1e-300))
+        worst = min(float(logits[t, e]) for e in chosen)
+        for e in allowed:
+            if e not in chosen:
+                margin[t] = min(float(margin[t]), worst - float(logits[t, e]))
+    if margins is not None:
+        margins.append(margin)
     return out
 
 
-def experts(h, w, m, prefix):
-    weights = route(h @ w[prefix + "router"].T, m["router"])
+def experts(h, w, m, prefix, margins=None):
+    weights = route(h @ w[prefix + "router"].T, m["router"], margins)
     out = torch.zeros_like(h)
     for e in range(m["router"]["experts"]):
         hidden = torch.clamp(h @ w[f"{prefix}e{e}.up"].T, min=0) ** 2
@@ -235,9 +246,9 @@ def layer_order(config):
     return list(range(loop["start"])) + looped * loop["times"] + list(range(loop["stop"], count))
 
 
-def forward(config, weights, tokens, kind=torch.float64, streams=None):
+def forward(config, weights, tokens, kind=torch.float64, streams=None, margins=None):
     """Logits [T, vocab] of one sequence. ``streams``: a list that receives the sum of the
-    streams after the embedding and after every layer run."""
+    streams after the embedding and after every layer run; ``margins``: see ``route``."""
     w = {name: t.to(kind) for name, t in weights.items()}
     eps = config["norm"]["eps"]
     x = w["embed"][torch.as_tensor(tokens, dtype=torch.long)]
@@ -251,7 +262,7 @@ def forward(config, weights, tokens, kind=torch.float64, streams=None):
         X = write_streams(X, w[p + "hc1.mix"], w[p + "hc1.out"], y)
         if layer.get("mlp") is not None:
             h = rms_norm(read_streams(X, w[p + "hc2.in"]), w[p + "norm2"], eps)
-            y = FEED_FORWARDS[layer["mlp"]["kind"]](h, w, layer["mlp"], p + "mlp.")
+            y = FEED_FORWARDS[layer["mlp"]["kind"]](h, w, layer["mlp"], p + "mlp.", margins)
             X = write_streams(X, w[p + "hc2.mix"], w[p + "hc2.out"], y)
         if streams is not None:
             streams.append(X.sum(0))
