@@ -115,13 +115,13 @@ __device__ __forceinline__ int warp_best(const float* values, int count, int lan
     int at = count;
     for (int e = lane; e < count; e += 32)
         if (values[e] > best) { best = values[e]; at = e; }
-#pragma unroll
-    for (int across = 16; across > 0; across >>= 1) {
-        const float other = __shfl_xor_sync(0xffffffffu, best, across);
-        const int other_at = __shfl_xor_sync(0xffffffffu, at, across);
-        if (other > best || (other == best && other_at < at)) { best = other; at = other_at; }
-    }
-    return best == -INFINITY ? -1 : at;
+    // floats as integers of the same order: the warp's maximum and, among its lanes, the lowest
+    // place are one reduction each
+    const unsigned bits = __float_as_uint(best + 0.f);
+    const unsigned key = bits ^ ((bits >> 31) ? 0xffffffffu : 0x80000000u);
+    const unsigned most = __reduce_max_sync(0xffffffffu, key);
+    at = __reduce_min_sync(0xffffffffu, key == most ? at : count);
+    return at == count ? -1 : at;
 }
 
 template <typename T>
