@@ -195,7 +195,7 @@ __global__ void __launch_bounds__(256)
 sum_streams_kernel(const float* __restrict__ streams, const T* __restrict__ y,
                    const float* __restrict__ mix, const float* __restrict__ out,
                    const int* __restrict__ rows, float* __restrict__ total, int n_in, int n_out,
-                   int hidden, int tokens) {
+                   int hidden, int tokens, int wide) {
     __shared__ float factor[MAX_STREAMS + 1];
     griddep_launch();
     if (threadIdx.x <= n_in) {
@@ -213,6 +213,26 @@ sum_streams_kernel(const float* __restrict__ streams, const T* __restrict__ y,
     const int i = blockIdx.x;
     const int t = rows != nullptr ? rows[i] : i;
     if (t < 0 || t >= tokens) return;
+    if (wide) {
+        // four values a load, the streams' loads on their way together
+        for (int c = threadIdx.x * 4; c < hidden; c += blockDim.x * 4) {
+            float sum[4] = {0.f, 0.f, 0.f, 0.f};
+            if (y != nullptr) {
+                Four<T>::load(y + (size_t)t * hidden + c, sum);
+#pragma unroll
+                for (int k = 0; k < 4; ++k) sum[k] *= factor[n_in];
+            }
+#pragma unroll 4
+            for (int s = 0; s < n_in; ++s) {
+                float x[4];
+                Four<float>::load(streams + ((size_t)t * n_in + s) * hidden + c, x);
+#pragma unroll
+                for (int k = 0; k < 4; ++k) sum[k] = fmaf(factor[s], x[k], sum[k]);
+            }
+            Four<float>::store(total + (size_t)i * hidden + c, sum);
+        }
+        return;
+    }
     for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
         float sum = y != nullptr ? factor[n_in] * to_float<T>(y[(size_t)t * hidden + c]) : 0.f;
         for (int s = 0; s < n_in; ++s)
@@ -295,13 +315,15 @@ MLXONE_API int mlxone_sum_streams(const float* streams, const void* y, const flo
     if (count == 0) return 0;
     MLXONE_REQUIRE(count > 0 && tokens > 0 && hidden > 0 && n_in >= 1 && n_in <= MAX_STREAMS &&
                        n_out >= 1 && n_out <= MAX_STREAMS, "sum_streams: 1 to %d streams", MAX_STREAMS);
+    const auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    const int wide = hidden % 4 == 0 && aligned(streams) && aligned(y) && aligned(total);
     if (dtype == MLXONE_BF16)
         launch_kernel(sum_streams_kernel<__nv_bfloat16>, dim3(count), dim3(256), 0, stream, true,
                       streams, (const __nv_bfloat16*)y, mix, out, rows, total, n_in, n_out, hidden,
-                      tokens);
+                      tokens, wide);
     else
         launch_kernel(sum_streams_kernel<float>, dim3(count), dim3(256), 0, stream, true, streams,
-                      (const float*)y, mix, out, rows, total, n_in, n_out, hidden, tokens);
+                      (const float*)y, mix, out, rows, total, n_in, n_out, hidden, tokens, wide);
     MLXONE_LAUNCH_CHECK("sum_streams");
     return 0;
 }

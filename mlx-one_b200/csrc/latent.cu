@@ -42,6 +42,13 @@ latent_prepare_kernel(const T* __restrict__ q_source, int ld_q, T* __restrict__ 
     small_source = settled(small_source);
     down_source = settled(down_source);
     const int t = blockIdx.x;
+    // (two blocks a token: the second has the queries' latent, the first the rest)
+    if (gridDim.y == 2 && blockIdx.y == 0) small_source = nullptr;
+    if (gridDim.y == 2 && blockIdx.y == 1) {
+        q_source = nullptr;
+        down_source = nullptr;
+        rotary_dim = 0;
+    }
     const int position = positions[t];
     const int half = rotary_dim / 2;
     float* cosines = shared;
@@ -112,6 +119,92 @@ latent_prepare_kernel(const T* __restrict__ q_source, int ld_q, T* __restrict__ 
         dst[e] = from_float<T>(to_float<T>(down[e]) * inv * norm_weight[e]);
     for (int e = threadIdx.x; e < rot_dim; e += blockDim.x)
         dst[latent + e] = from_float<T>(rotated(down + latent, e));
+}
+
+// Few tokens: the queries against the latents in one kernel. Grid (heads, tiles of 64 latent columns
+// + 1): queries[t, h, n] = up_k[h, n, :] . q[t, h, :head_dim] for the tile's columns n, two threads
+// a column with half of the products each, the matrix's rows asked for before the wait; the last
+// block of a head rotates its queries' rotated parts. head_dim a multiple of 16 up to 128, at most
+// TOKENS tokens.
+constexpr int ABSORB_COLUMNS = 64, ABSORB_PIECES = 8;
+
+template <int TOKENS>
+__global__ void __launch_bounds__(2 * ABSORB_COLUMNS)
+latent_absorb_kernel(const __nv_bfloat16* __restrict__ q, int ld, const __nv_bfloat16* __restrict__ up_k,
+                     __nv_bfloat16* __restrict__ queries, const float* __restrict__ inv_freq,
+                     int rotary_dim, float amplitude, int neighbours, const int* __restrict__ positions,
+                     int tokens, int heads, int head_dim, int rot_dim, int latent) {
+    using T = __nv_bfloat16;
+    __shared__ __align__(16) float staged[TOKENS * (128 + 8)];
+    griddep_launch();
+    const int h = blockIdx.x, row = latent + rot_dim;
+    const T* source = q + (size_t)h * (head_dim + rot_dim);
+    if (blockIdx.y == gridDim.y - 1) {
+        griddep_wait();
+        source = settled(source);
+        const int half = rotary_dim / 2, rest = rot_dim - rotary_dim;
+        for (int i = threadIdx.x; i < tokens * (half + rest); i += blockDim.x) {
+            const int t = i / (half + rest), pair = i - t * (half + rest);
+            const T* part = source + (size_t)t * ld + head_dim;
+            T* to = queries + ((size_t)t * heads + h) * row + latent;
+            if (pair >= half) {
+                to[half + pair] = part[half + pair];              // = rotary_dim + (pair - half)
+                continue;
+            }
+            float sine, cosine;
+            sincosf((float)positions[t] * inv_freq[pair], &sine, &cosine);
+            sine *= amplitude;
+            cosine *= amplitude;
+            const int first = neighbours ? 2 * pair : pair, second = neighbours ? first + 1 : pair + half;
+            const float u = to_float<T>(part[first]), v = to_float<T>(part[second]);
+            to[first] = from_float<T>(u * cosine - v * sine);
+            to[second] = from_float<T>(v * cosine + u * sine);
+        }
+        return;
+    }
+    const int side = threadIdx.x & 1, n = blockIdx.y * ABSORB_COLUMNS + (threadIdx.x >> 1);
+    const int halved = head_dim / 2, pieces = halved / 8, stride = halved + 4;
+    uint4 held[ABSORB_PIECES];
+#pragma unroll
+    for (int i = 0; i < ABSORB_PIECES; ++i) {
+        held[i] = make_uint4(0u, 0u, 0u, 0u);
+        if (i < pieces && n < latent)
+            held[i] = *reinterpret_cast<const uint4*>(up_k + ((size_t)h * latent + n) * head_dim +
+                                                      side * halved + i * 8);
+    }
+    griddep_wait();
+    source = settled(source);
+    for (int i = threadIdx.x; i < TOKENS * head_dim; i += blockDim.x) {
+        const int t = i / head_dim, e = i - t * head_dim;
+        staged[t * 2 * stride + (e < halved ? e : e + 4)] = t < tokens ? to_float<T>(source[(size_t)t * ld + e]) : 0.f;
+    }
+    __syncthreads();
+    float sum[TOKENS];
+#pragma unroll
+    for (int t = 0; t < TOKENS; ++t) sum[t] = 0.f;
+#pragma unroll
+    for (int i = 0; i < ABSORB_PIECES; ++i) {
+        if (i >= pieces) break;
+        const T* w = reinterpret_cast<const T*>(&held[i]);
+        float weight[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) weight[k] = to_float<T>(w[k]);
+#pragma unroll
+        for (int t = 0; t < TOKENS; ++t) {
+            const float* x = staged + t * 2 * stride + side * stride + i * 8;
+            const float4 lo = *reinterpret_cast<const float4*>(x), hi = *reinterpret_cast<const float4*>(x + 4);
+            sum[t] = fmaf(weight[0], lo.x, sum[t]); sum[t] = fmaf(weight[1], lo.y, sum[t]);
+            sum[t] = fmaf(weight[2], lo.z, sum[t]); sum[t] = fmaf(weight[3], lo.w, sum[t]);
+            sum[t] = fmaf(weight[4], hi.x, sum[t]); sum[t] = fmaf(weight[5], hi.y, sum[t]);
+            sum[t] = fmaf(weight[6], hi.z, sum[t]); sum[t] = fmaf(weight[7], hi.w, sum[t]);
+        }
+    }
+#pragma unroll
+    for (int t = 0; t < TOKENS; ++t) {
+        sum[t] += __shfl_xor_sync(0xffffffffu, sum[t], 1);
+        if (t < tokens && n < latent && (t & 1) == side)
+            queries[((size_t)t * heads + h) * row + n] = from_float<T>(sum[t]);
+    }
 }
 
 // out[t, c] = values[t, c] * sigmoid(gate[t * ld_gate + c])
@@ -247,7 +340,8 @@ MLXONE_API int mlxone_latent_prepare(const void* q_source, int ld_q, void* queri
     if (small_source != nullptr && rank > most) most = rank;
     const int threads = most >= 2048 ? 512 : most >= 512 ? 256 : 128;
 #define PREPARE(T)                                                                              \
-    launch_kernel(latent_prepare_kernel<T>, dim3(tokens), dim3(threads), shared, stream, true,  \
+    launch_kernel(latent_prepare_kernel<T>, dim3(tokens, small_source != nullptr ? 2 : 1),      \
+                  dim3(threads), shared, stream, true,                                          \
                   (const T*)q_source, ld_q, (T*)queries, (const T*)small_source, ld_small,      \
                   small_weight, (T*)small, rank, (const T*)down_source, ld_down, norm_weight, eps, \
                   inv_freq, rotary_dim, amplitude, neighbours, positions, token_request, (T*)pages, \
@@ -257,6 +351,39 @@ MLXONE_API int mlxone_latent_prepare(const void* q_source, int ld_q, void* queri
     else PREPARE(float);
 #undef PREPARE
     MLXONE_LAUNCH_CHECK("latent_prepare");
+    return 0;
+}
+
+// 1 if latent_absorb takes `tokens` tokens of heads with head_dim unrotated values.
+MLXONE_API int mlxone_latent_absorb_fits(int tokens, int head_dim) {
+    return tokens >= 1 && tokens <= 16 && head_dim % 16 == 0 && head_dim >= 16 &&
+           head_dim <= 16 * ABSORB_PIECES;
+}
+
+// q [tokens, heads * (head_dim + rot_dim)] bfloat16 with rows `ld` apart; up_k [heads, latent,
+// head_dim]; queries [tokens, heads, latent + rot_dim].
+MLXONE_API int mlxone_latent_absorb(const void* q, int ld, const void* up_k, void* queries,
+                                    const float* inv_freq, int rotary_dim, float amplitude,
+                                    int neighbours, const int* positions, int tokens, int heads,
+                                    int head_dim, int rot_dim, int latent, cudaStream_t stream) {
+    if (tokens == 0) return 0;
+    if (inv_freq == nullptr) rotary_dim = 0;
+    MLXONE_REQUIRE(mlxone_latent_absorb_fits(tokens, head_dim) && heads > 0 && latent > 0 && rot_dim >= 0 &&
+                       ld >= heads * (head_dim + rot_dim), "latent_absorb: bad sizes");
+    MLXONE_REQUIRE((reinterpret_cast<uintptr_t>(up_k) & 15) == 0, "latent_absorb: up_k is not aligned");
+    MLXONE_REQUIRE(rotary_dim >= 0 && rotary_dim % 2 == 0 && rotary_dim <= rot_dim,
+                   "latent_absorb: %d rotated dimensions in a part of %d", rotary_dim, rot_dim);
+    const dim3 grid(heads, (latent + ABSORB_COLUMNS - 1) / ABSORB_COLUMNS + 1);
+#define ABSORB(TOKENS)                                                                              \
+    launch_kernel(latent_absorb_kernel<TOKENS>, grid, dim3(2 * ABSORB_COLUMNS), 0, stream, true,    \
+                  (const __nv_bfloat16*)q, ld, (const __nv_bfloat16*)up_k, (__nv_bfloat16*)queries, \
+                  inv_freq, rotary_dim, amplitude, neighbours, positions, tokens, heads, head_dim,  \
+                  rot_dim, latent)
+    if (tokens <= 4) ABSORB(4);
+    else if (tokens <= 8) ABSORB(8);
+    else ABSORB(16);
+#undef ABSORB
+    MLXONE_LAUNCH_CHECK("latent_absorb");
     return 0;
 }
 

@@ -114,6 +114,8 @@ class CudaOps:
         # one up to 16 rows: out_proj 4.3 us against 5.7 us, w2 10.5 us against 13.0 us, w13 with
         # its gate 14.6 us against 12.9 us plus a gate kernel
         self.skinny_fused_max_rows = 16
+        # latent attention of few tokens: the key up-projection with the queries' rotation in one kernel
+        self.fused_latent = True
         self._sample_scratch: torch.Tensor | None = None
         self._device_index = self.device.index if self.device.index is not None else torch.cuda.current_device()
 
@@ -632,6 +634,33 @@ class CudaOps:
         self._latent_prepare(queries.dtype, q.shape[0], q=q, queries=queries, heads=heads,
                              head_dim=head_dim, rot_dim=rot_dim, latent=latent, rotary=rotary,
                              amplitude=amplitude, neighbours=neighbours, ctx=ctx)
+
+    def latent_absorb(self, q, up_k, queries, *, heads, head_dim, rot_dim, latent, rotary, neighbours,
+                      ctx, amplitude=1.0):
+        """The finished query rows [tokens, heads, latent + rot_dim] from q [tokens, heads * (head_dim +
+        rot_dim)] and the transposed key up-projections [heads, latent, head_dim]: up_k q of the
+        unrotated parts in front, the rotated parts behind. Up to 16 tokens in bfloat16 one kernel,
+        else ``latent_queries`` and ``linear_heads``."""
+        tokens = q.shape[0]
+        self._need_rows(q, queries.dtype, "q")
+        self._need(queries, queries.dtype, "queries")
+        self._need(up_k, queries.dtype, "up_k")
+        if queries.shape != (tokens, heads, latent + rot_dim) or up_k.shape != (heads, latent, head_dim) or \
+                q.shape[1] != heads * (head_dim + rot_dim):
+            raise KernelError("queries are rows of latent + rot_dim values")
+        if queries.dtype == torch.bfloat16 and self.fused_latent and \
+                self.lib.mlxone_latent_absorb_fits(_c_int(tokens), _c_int(head_dim)):
+            inv_freq, rotary_dim = (None, 0) if rotary is None else rotary
+            self._call("mlxone_latent_absorb", _c_void_p(_ptr(q)), _c_int(q.stride(0)),
+                       _c_void_p(_ptr(up_k)), _c_void_p(_ptr(queries)), _c_void_p(_ptr(inv_freq)),
+                       _c_int(rotary_dim), _c_float(amplitude), _c_int(1 if neighbours else 0),
+                       _c_void_p(_ptr(ctx.positions)), _c_int(tokens), _c_int(heads),
+                       _c_int(head_dim), _c_int(rot_dim), _c_int(latent))
+            return
+        self.latent_queries(q, queries, heads=heads, head_dim=head_dim, rot_dim=rot_dim, latent=latent,
+                            rotary=rotary, neighbours=neighbours, ctx=ctx, amplitude=amplitude)
+        self.linear_heads(q.unflatten(1, (heads, -1))[:, :, :head_dim], up_k,
+                          out=queries[:, :, :latent])
 
     def linear_heads(self, a, w, out=None):
         """a [tokens, heads, K] with w [heads, N, K] -> [tokens, heads, N], one product per head.

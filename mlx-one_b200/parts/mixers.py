@@ -720,16 +720,15 @@ class LatentAttention(Mixer):
                                          norm_weight=self.down_norm, eps=self.eps, view=cache,
                                          write=write, **common)
             q = self.ops.linear(small, self.query_up)
-            self.ops.latent_queries(q, queries, heads=heads, head_dim=self.head_dim, **common)
+            self.ops.latent_absorb(q, self.up_k, queries, heads=heads, head_dim=self.head_dim, **common)
         else:
             # the latent's norm, the rotation of the shared key part and of the queries' rotated
             # parts, the row [c | r] appended to the request's pages
             self.ops.latent_prepare(projected, queries, heads=heads, head_dim=self.head_dim,
                                     norm_weight=self.down_norm, eps=self.eps, view=cache,
                                     write=write, **common)
-            q = projected[:, :heads * (self.head_dim + rot)]
-        plain = q.unflatten(1, (heads, -1))
-        self.ops.linear_heads(plain[:, :, :self.head_dim], self.up_k, out=queries[:, :, :latent])
+            plain = projected[:, :heads * (self.head_dim + rot)].unflatten(1, (heads, -1))
+            self.ops.linear_heads(plain[:, :, :self.head_dim], self.up_k, out=queries[:, :, :latent])
         return projected, queries
 
     def forward(self, x, ctx, cache, write):

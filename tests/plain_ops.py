@@ -366,6 +366,12 @@ class PlainOps:
         out.copy_(result)
         return out
 
+    def latent_absorb(self, q, up_k, queries, *, heads, head_dim, rot_dim, latent, rotary, neighbours,
+                      ctx, amplitude=1.0):
+        self.latent_queries(q, queries, heads=heads, head_dim=head_dim, rot_dim=rot_dim, latent=latent,
+                            rotary=rotary, neighbours=neighbours, ctx=ctx, amplitude=amplitude)
+        self.linear_heads(q.unflatten(1, (heads, -1))[:, :, :head_dim], up_k, out=queries[:, :, :latent])
+
     def latent_attention(self, queries, *, heads, latent, scale, ctx, view, sinks=None):
         tokens, _, row = queries.shape
         flat = self.paged_attention(queries, heads=heads, kv_heads=1, head_dim=row, scale=scale,

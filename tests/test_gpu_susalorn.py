@@ -330,6 +330,37 @@ def test_sinks_and_a_far_row(ops, dtype, heads, latent_size, rot_dim):
     ops.check_errors()
 
 
+@pytest.mark.parametrize("tokens, heads, head_dim, rot_dim, dims, latent_size", [
+    (1, 3, 16, 4, 4, 40), (4, 5, 48, 24, 16, 72), (7, 16, 64, 32, 32, 256), (8, 2, 128, 64, 64, 512),
+    (16, 20, 32, 8, 8, 200), (13, 1, 96, 2, 2, 8), (17, 2, 64, 16, 16, 64), (3, 2, 24, 8, 8, 32)])
+@pytest.mark.parametrize("neighbours", [False, True])
+def test_queries_of_few_tokens_in_one_kernel(ops, tokens, heads, head_dim, rot_dim, dims, latent_size, neighbours):
+    """The key up-projection and the rotation of up to 16 tokens in one kernel (more tokens and other
+    sizes in two) against the plain products; the queries' rows may be a slice of wider rows."""
+    generator = torch.Generator().manual_seed(tokens)
+    width = heads * (head_dim + rot_dim)
+    q = torch.randn(tokens, width + 24, generator=generator).bfloat16()
+    up_k = (torch.randn(heads, latent_size, head_dim, generator=generator) / head_dim ** 0.5).bfloat16()
+    inv_freq = torch.rand(dims // 2, generator=generator)
+    ctx = context([1] * tokens, [7 * i * i + i for i in range(tokens)])
+    queries = torch.full((tokens, heads, latent_size + rot_dim), 9.0, dtype=torch.bfloat16, device=DEVICE)
+    ops.latent_absorb(on(q)[:, :width], on(up_k), queries, heads=heads, head_dim=head_dim, rot_dim=rot_dim,
+                      latent=latent_size, rotary=(on(inv_freq), dims), neighbours=neighbours, ctx=ctx,
+                      amplitude=1.3)
+    rows = q[:, :width].double().view(tokens, heads, -1)
+    front = torch.einsum("thk,hnk->thn", rows[:, :, :head_dim], up_k.double())
+    parts = rows[:, :, head_dim:].clone()
+    angle = (ctx.positions.cpu().float()[:, None] * inv_freq[None, :]).double()[:, None, :]
+    first = slice(0, dims, 2) if neighbours else slice(0, dims // 2)
+    second = slice(1, dims, 2) if neighbours else slice(dims // 2, dims)
+    u, v = parts[..., first].clone(), parts[..., second].clone()
+    parts[..., first] = 1.3 * (u * torch.cos(angle) - v * torch.sin(angle))
+    parts[..., second] = 1.3 * (v * torch.cos(angle) + u * torch.sin(angle))
+    got = queries.cpu().double()
+    assert (got[:, :, :latent_size] - front).abs().max() < 0.02 * max(1.0, float(front.abs().max()))
+    assert (got[:, :, latent_size:] - parts).abs().max() < 0.03
+
+
 # ------------------------------------------------------------------ the delta rule
 
 
