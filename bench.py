@@ -2216,6 +2216,30 @@ def kernel_case(name: str, batch: int, context: int) -> int:
             run = lambda i: ops.state_space_scan(rows[i % 4], raw[i % 4], view=views[i % 4], **constants)
             work = (f"{ctx.tokens} tokens of {len(portions)} requests, {heads} heads of {state_dim} x "
                     f"{value_dim}, state {slot * 4 / 1e6:.1f} MB a request")
+    elif name in ("channel_delta_prefill", "channel_delta_decode"):
+        # the delta rule with a decay per key channel at the shape of a 2048-wide model: one prompt
+        # of 2,048 tokens (two inner products, prepare, scan, finish) or `batch` single tokens
+        from mlx_one_b200.parts import FixedState, StateView
+        from mlx_one_b200.parts.mixers import GatedDeltaRule
+
+        sizes = dict(heads=16, kv_heads=8, key_dim=128, value_dim=128, taps=4)
+        slot, rank = GatedDeltaRule.state_size(sizes), 128
+        channels = 2 * 8 * 128 + 16 * 128
+        portions = [1] * batch if name == "channel_delta_decode" else [PREFILL_TOKENS]
+        ctx, _ = batch_context(portions, [context if name == "channel_delta_decode" else 0] * len(portions))
+        state = torch.zeros(4 * len(portions), slot, device=device)
+        views = [StateView(state, torch.arange(c * len(portions), (c + 1) * len(portions), dtype=torch.int32,
+                                               device=device), FixedState((slot,), "float32")) for c in range(4)]
+        rows = [torch.randn(ctx.tokens, channels + 16 + 2 * rank, device=device).bfloat16() for _ in range(4)]
+        ups = [(torch.randn(2048, rank, device=device) * 0.1).bfloat16() for _ in range(2)]
+        constants = dict(decay_columns=(channels + 16, channels + 16 + rank),
+                         gate_columns=(channels + 16 + rank, channels + 16 + 2 * rank),
+                         conv=torch.randn(channels, 4, device=device) * 0.5, a_log=torch.zeros(16, device=device),
+                         dt_bias=torch.zeros(2048, device=device), norm_weight=torch.ones(128, device=device),
+                         eps=1e-6, unit_eps=1e-6, ctx=ctx, write=True, **sizes)
+        run = lambda i: ops.channel_delta_rule(rows[i % 4], *ups, view=views[i % 4], **constants)
+        work = (f"{ctx.tokens} tokens of {len(portions)} requests, 16 heads of 128 x 128 on 8 key heads, "
+                f"state {slot * 4 / 1e6:.1f} MB a request")
     elif name in ("latent_prefill", "latent_decode"):
         # attention over latent rows at the sizes of a Lamisun 1024 wide: one 2,048-token prompt
         # (the kernel whose warps own 16 rows) or `batch` single tokens (key runs and their merge)
@@ -2343,7 +2367,8 @@ def main() -> int:
                              "skinny_in_proj, skinny_down, decode_attention, prefill_attention, tcgen05_swiglu, "
                              "swapped_swiglu, mixed_attention, sampling, delta_prefill, delta_decode, lightning_prefill, "
                              "lightning_decode, experts_sorted, latent_prefill, latent_decode, state_space_prefill, "
-                             "state_space_decode, channel_conv_prefill, decode_step (the "
+                             "state_space_decode, channel_conv_prefill, channel_delta_prefill, "
+                             "channel_delta_decode, decode_step (the "
                              "whole step, eager, for a launch list), decode_timeline (where "
                              "the graph-replayed step's time goes, kernel by kernel)")
     parser.add_argument("--dependent-launches", type=int, default=1,
