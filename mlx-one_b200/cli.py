@@ -10,7 +10,7 @@ from dataclasses import asdict
 import click
 
 
-@click.group(help="B200-native inference engine (LFM2, Galarax, Farorax, Lamisun, Tirudra and Susalorn models).")
+@click.group(help="B200-native inference engine (LFM2, Galarax, Farorax, Lamisun, Tirudra, Susalorn and Zinizen models).")
 def main() -> None:
     pass
 

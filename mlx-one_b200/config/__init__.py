@@ -5,10 +5,11 @@ from .lamisun import LamisunConfig
 from .lfm2 import Lfm2Config
 from .susalorn import SusalornConfig
 from .tirudra import TirudraConfig
+from .zinizen import ZinizenConfig
 from .registry import (Architecture, architecture_key, architecture_names, get_architecture, read_config,
                        register_architecture, unregister_architecture)
 
 __all__ = ["ConfigError", "FaroraxConfig", "GalaraxConfig", "LamisunConfig", "Lfm2Config",
-           "SusalornConfig", "TirudraConfig", "Architecture", "architecture_key", "architecture_names",
-           "get_architecture", "read_config", "register_architecture",
+           "SusalornConfig", "TirudraConfig", "ZinizenConfig", "Architecture", "architecture_key",
+           "architecture_names", "get_architecture", "read_config", "register_architecture",
            "unregister_architecture"]

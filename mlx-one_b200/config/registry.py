@@ -34,6 +34,7 @@ _BUILTIN = {
     "lamisun": "mlx_one_b200.architectures.lamisun:ARCHITECTURE",
     "tirudra": "mlx_one_b200.architectures.tirudra:ARCHITECTURE",
     "susalorn": "mlx_one_b200.architectures.susalorn:ARCHITECTURE",
+    "zinizen": "mlx_one_b200.architectures.zinizen:ARCHITECTURE",
 }
 _REGISTERED: dict[str, Architecture] = {}
 

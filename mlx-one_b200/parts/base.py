@@ -112,6 +112,9 @@ class StepContext:
     # shape, so it holds for every replay. A mixer may give these tokens to a kernel made for
     # single tokens and the rest to another.
     leading_single: int = 0
+    # What a layer leaves for later layers of the same step, by name (a tensor of the step's tokens:
+    # the values that later layers mix theirs with). Nothing of it outlives the step.
+    shared: dict = field(default_factory=dict)
 
 
 class NoHostValues(Mapping):
@@ -228,15 +231,38 @@ class FeedForward(Part):
         raise NotImplementedError
 
 
+class NormedUpdate:
+    """The output of a sublayer that is still to be normed and added to the stream: residual +
+    norm(output), the norm taken over the output's row in 32-bit; ``bias`` None: x / rms(x) * weight,
+    else (x - mean) / sqrt(variance + eps) * weight + bias."""
+
+    def __init__(self, output: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None,
+                 eps: float) -> None:
+        self.output, self.weight, self.bias, self.eps = output, weight, bias, eps
+
+    def of(self, output: torch.Tensor) -> "NormedUpdate":
+        """The same norm of other rows (the rows of a step whose logits are wanted)."""
+        return NormedUpdate(output, self.weight, self.bias, self.eps)
+
+    def applied(self, residual: torch.Tensor) -> torch.Tensor:
+        """The stream after the update, computed plainly (for observers)."""
+        x = self.output.float()
+        if self.bias is not None:
+            x = x - x.mean(dim=-1, keepdim=True)
+        x = x * torch.rsqrt(x.pow(2).mean(dim=-1, keepdim=True) + self.eps) * self.weight
+        return residual + (x if self.bias is None else x + self.bias)
+
+
 class Norm(Part):
     # True: forward takes ``lazy=`` (see below); a norm that leaves it False is always computed
     supports_lazy = False
 
     def forward(self, residual: torch.Tensor, delta: torch.Tensor | None,
                 lazy: bool = False, delta_scale: float = 1.0) -> torch.Tensor:
-        """Adds ``delta_scale * delta`` (compute dtype, or None) into the 32-bit ``residual`` in
-        place and returns the normed residual in the compute dtype. With ``lazy`` a norm may
-        return a ``NormedInput`` instead, for a consumer that ``accepts_normed_input``."""
+        """Adds ``delta_scale * delta`` (compute dtype, or None; where a block hands on
+        ``NormedUpdate``s, such a one) into the 32-bit ``residual`` in place and returns the normed
+        residual in the compute dtype. With ``lazy`` a norm may return a ``NormedInput`` instead,
+        for a consumer that ``accepts_normed_input``."""
         raise NotImplementedError
 
 
@@ -302,6 +328,8 @@ class Block(Part):
     # embedding's output, ahead of the first block): ``residual`` has that shape, ``delta`` is a
     # ``StreamUpdate`` or None, and ``forward`` returns (streams, StreamUpdate).
     parallel_streams = False
+    # True: the block is given, and returns, a ``NormedUpdate`` (or None) instead of a plain output
+    normed_updates = False
 
     @classmethod
     def cache_need(cls, spec: PartSpec):

@@ -2,7 +2,7 @@
 
 from __future__ import annotations
 
-from .base import Block, FixedState, StreamUpdate
+from .base import Block, FixedState, NormedUpdate, StreamUpdate
 from .registry import BLOCKS
 from .spec import TensorSpec
 
@@ -130,15 +130,28 @@ class SandwichBlock(Block):
     the block's own: v / rms(v) * (offset + weight) over the model width, with the stored weights
     ``post_mixer`` and ``post_feed_forward``, taken and added in 32-bit. A layer without a
     feed-forward ends after the mixer. Parameters: ``size``, ``eps``, ``offset`` (0; 1 for
-    weights stored around zero), ``feed_forward`` (True: the layer has one)."""
+    weights stored around zero), ``feed_forward`` (True: the layer has one), ``norm``
+    (``rmsnorm``; ``layernorm``: the norms behind the parts are (v - mean) / sqrt(variance + eps) *
+    weight + bias, with the stored ``post_mixer.bias`` and ``post_feed_forward.bias``).
+
+    With layer norms a part's output is handed on as a ``NormedUpdate``: one kernel norms it, adds it
+    to the stream and applies the norm ahead of the next part (of the next layer, at the end)."""
 
     @classmethod
     def tensors(cls, spec):
         init = "norm0" if spec.get("offset") else "norm"
-        out = {"post_mixer": TensorSpec((spec["size"],), init)}
-        if spec.get("feed_forward", True):
-            out["post_feed_forward"] = TensorSpec((spec["size"],), init)
+        names = ["post_mixer"] + (["post_feed_forward"] if spec.get("feed_forward", True) else [])
+        out = {name: TensorSpec((spec["size"],), init) for name in names}
+        if cls._layer_norms(spec):
+            out.update({name + ".bias": TensorSpec((spec["size"],), "bias") for name in names})
         return out
+
+    @staticmethod
+    def _layer_norms(spec):
+        kind = spec.get("norm") or "rmsnorm"
+        if kind not in ("rmsnorm", "layernorm"):
+            raise ValueError(f"unknown norm {kind!r}")
+        return kind == "layernorm"
 
     def __init__(self, spec, tensors, runtime, **roles):
         super().__init__(spec, tensors, runtime, **roles)
@@ -149,6 +162,11 @@ class SandwichBlock(Block):
         self.post_feed_forward = weight("post_feed_forward") if "post_feed_forward" in tensors else None
         if (self.feed_forward is None) != (self.post_feed_forward is None):
             raise ValueError("a feed-forward and the norm behind it come together")
+        self.normed_updates = self._layer_norms(spec)
+        self.biases = {}
+        if self.normed_updates:
+            self.biases = {name[:-len(".bias")]: self.vector(tensors[name])
+                           for name in tensors if name.endswith(".bias")}
 
     def _read(self, norm, residual, delta, consumer, scale=1.0):
         extra = {} if scale == 1.0 else {"delta_scale": scale}
@@ -156,7 +174,18 @@ class SandwichBlock(Block):
             return norm.forward(residual, delta, lazy=True, **extra)
         return norm.forward(residual, delta, **extra)
 
+    def _forward_updates(self, residual, delta, ctx, cache, write):
+        normed = self.mixer_norm.forward(residual, delta)
+        out = self.mixer.forward(normed, ctx, cache, write)
+        delta = NormedUpdate(out, self.post_mixer, self.biases["post_mixer"], self.eps)
+        if self.feed_forward is not None:
+            out = self.feed_forward.forward(self.feed_forward_norm.forward(residual, delta), ctx)
+            delta = NormedUpdate(out, self.post_feed_forward, self.biases["post_feed_forward"], self.eps)
+        return delta
+
     def forward(self, residual, delta, ctx, cache, write, delta_scale=1.0):
+        if self.normed_updates:
+            return self._forward_updates(residual, delta, ctx, cache, write)
         normed = self._read(self.mixer_norm, residual, delta, self.mixer, delta_scale)
         mixed = self.mixer.forward(normed, ctx, cache, write)
         self.ops.normed_mean_add(residual, [mixed], [self.post_mixer], self.eps)

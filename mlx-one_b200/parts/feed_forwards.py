@@ -105,7 +105,9 @@ class RoutedExperts(FeedForward):
     (0: that many further outputs of the router, behind the experts', stand for experts without
     tensors whose output is the input itself), ``shared_gate`` (True: the shared expert's output
     is multiplied by sigmoid(w x), one number per token, with the stored ``shared.sg`` [1,
-    hidden]).
+    hidden]), ``limit`` and ``shared_limit`` (with ``activation`` ``clamped``: the experts' and the
+    shared expert's gate g and up value u are cut, g to at most the limit, u to at most the limit
+    on both sides, and the hidden value is g sigmoid(1.702 g) (u + 1)).
 
     Router logits W_r x are 32-bit, scores s = sigmoid of them; the ``top`` allowed experts
     with the largest scores are chosen and weighted with s / (sum of the chosen s + 1e-20). The
@@ -153,6 +155,15 @@ class RoutedExperts(FeedForward):
         self.experts, self.width = spec["experts"], spec["width"]
         self.shared_width = spec.get("shared_width") or 0
         self.activation = spec.get("activation") or "silu"
+        self.limits, self.shared_limits = {}, {}
+        if self.activation == "clamped":
+            if not spec.get("gated", True):
+                raise ValueError("clamped hidden values need a gate")
+            # (the stacked product's columns from ``boundary`` on are the shared expert's)
+            limit = float(spec["limit"])
+            second = float(spec["shared_limit"]) if self.shared_width else limit
+            self.limits = dict(limits=(limit, second, self.experts * self.width))
+            self.shared_limits = dict(limits=(second, second, 0))
         scores = spec.get("scores") or "sigmoid"
         if scores not in ("sigmoid", "softmax"):
             raise ValueError(f"unknown routing scores {scores!r}")
@@ -195,10 +206,12 @@ class RoutedExperts(FeedForward):
                                      .reshape(1, -1)], dim=0).contiguous()
         # the shared expert once more on its own, for steps that sort their tokens by expert
         self.shared = {}
-        sorted_kinds = ("silu",) if self.gated else ("relu2",)
+        sorted_kinds = ("silu", "clamped") if self.gated else ("relu2",)
         self.sortable = (self.activation in sorted_kinds and hasattr(self.ops, "sorts_experts")
                          and runtime.dtype == torch.bfloat16)
-        self.sorted_form = {} if self.gated else dict(activation=self.activation)
+        self.sorted_form = {} if self.activation == "silu" else dict(activation=self.activation)
+        if self.activation == "clamped":
+            self.sorted_form.update(limit=float(spec["limit"]), shared_limits=self.shared_limits["limits"])
         if self.sortable and self.shared_width:
             self.shared = dict(
                 shared_gate_up=self.matrix(torch.cat([tensors["shared.gate"], tensors["shared.up"]], dim=0)),
@@ -213,7 +226,7 @@ class RoutedExperts(FeedForward):
             return self.ops.linear_act(x, self.gate_up, self.activation)
         if self.activation == "silu":
             return self.ops.linear_swiglu(x, self.gate_up)
-        return self.ops.linear_gated(x, self.gate_up, self.activation)
+        return self.ops.linear_gated(x, self.gate_up, self.activation, **self.limits)
 
     def _sorts(self, x):
         return self.sortable and self.ops.sorts_experts(

@@ -1,7 +1,7 @@
 """Sequence mixers: grouped-query attention over paged keys and values, the gated short
 convolution with a fixed-size state, the gated delta rule with a matrix state per head (one
-decay per head, or one per key channel), several mixers side by side on one input, attention over one latent row per token, and
-attention with two score maps per head."""
+decay per head, or one per key channel), several mixers side by side on one input, attention over one latent row per token,
+attention with two score maps per head, and a gated linear recurrence per channel."""
 
 from __future__ import annotations
 
@@ -17,8 +17,10 @@ class Attention(Mixer):
     """Grouped-query attention. Parameters: ``hidden``, ``heads``, ``kv_heads``,
     ``head_dim`` (size of a query and key head), ``value_dim`` (size of a value head; None =
     head_dim), ``bias`` (the three input projections have biases), ``qk_norm_eps`` (None = no
-    per-head RMSNorm of queries and keys), ``qk_norm`` (``weighted_before``: with a stored
-    weight, before the rotation; ``plain_after``: without a weight, after the rotation),
+    RMSNorm of queries and keys), ``qk_norm`` (``weighted_before``: per head, with a stored
+    weight, before the rotation; ``plain_after``: per head, without a weight, after the rotation;
+    ``weighted_rows``: over all heads of the queries, and of the keys, at once, with weights of
+    those sizes, before the rotation),
     ``position`` (a position-encoding PartSpec), ``window`` (None = all keys), ``scale`` (None =
     head_dim^-0.5), ``sink`` (a stored number per query head, ``sink`` [heads], that stands in
     the softmax's denominator as exp(sink) beside the keys' terms: it has no key and no value
@@ -32,7 +34,14 @@ class Attention(Mixer):
     token's; the last taps - 1 projected rows of a request are kept in a state slot), ``gate``
     (None; ``values``: the heads' outputs are multiplied value by value with sigmoid(W_g x),
     ``gate.weight`` [heads * value_dim, hidden]; ``heads``: one number per head, ``gate.weight``
-    [heads, hidden]; the gate reads the mixer's input and is applied before the output matrix).
+    [heads, hidden]; the gate reads the mixer's input and is applied before the output matrix),
+    ``temperature`` (None; (coef, every): queries at position p are multiplied by 1 + coef *
+    ln(floor((p + 1) / every) + 1)), ``score_cap`` (None; c: a score s = scale q.k becomes c tanh(s /
+    c)), ``distance_slopes`` (None; a number per query head: slope * (i - j) is taken off the score
+    of query i and key j, after the cap), ``value_mix`` (None; ``first``: the projected values are
+    left for later layers of the step; ``later``: the values are (1 - m) v + m v_first, m the stored
+    number ``value_mix`` and v_first what the ``first`` layer left for the same token; the mixed
+    values are what the pages hold).
 
     q, k, v projections (one fused matrix product), per-head RMSNorm of q and k, rotation,
     keys and values appended to the request's pages, causal softmax(q k^T scale) v where
@@ -54,7 +63,7 @@ class Attention(Mixer):
         if spec.get("qk_norm_eps") is None:
             return None
         kind = spec.get("qk_norm") or "weighted_before"
-        if kind not in ("weighted_before", "plain_after"):
+        if kind not in ("weighted_before", "plain_after", "weighted_rows"):
             raise ValueError(f"unknown qk_norm {kind!r}")
         return kind
 
@@ -87,6 +96,11 @@ class Attention(Mixer):
         if cls._norm_kind(spec) == "weighted_before":
             out["q_layernorm.weight"] = TensorSpec((hd,), "norm")
             out["k_layernorm.weight"] = TensorSpec((hd,), "norm")
+        elif cls._norm_kind(spec) == "weighted_rows":
+            out["q_layernorm.weight"] = TensorSpec((q_dim,), "norm")
+            out["k_layernorm.weight"] = TensorSpec((k_dim,), "norm")
+        if cls._value_mix(spec) is not None:
+            out["value_mix"] = TensorSpec((), "wide")
         if spec.get("sink"):
             out["sink"] = TensorSpec((spec["heads"],), "wide")
         return out
@@ -99,6 +113,13 @@ class Attention(Mixer):
         if kind == "keys" and (spec.get("value_dim") or spec["head_dim"]) != spec["head_dim"]:
             raise ValueError("values that are the keys have the keys' size")
         return kind == "projected"
+
+    @staticmethod
+    def _value_mix(spec):
+        kind = spec.get("value_mix")
+        if kind not in (None, "first", "later"):
+            raise ValueError(f"unknown value_mix {kind!r}")
+        return kind
 
     @staticmethod
     def _gate_kind(spec):
@@ -160,8 +181,7 @@ class Attention(Mixer):
             biases = [reorder("q_proj.bias", self.heads), reorder("k_proj.bias", self.kv_heads),
                       tensors[values + ".bias"]]
         if self.gate_kind is not None:
-            general = (self.value_dim != self.head_dim or self._norm_kind(spec) == "plain_after"
-                       or self.position.amplitude() != 1.0)
+            general = self._general(spec)
             if self.taps or general:
                 stacked.append(tensors["gate.weight"])
                 if biases:
@@ -186,31 +206,61 @@ class Attention(Mixer):
         self.norm_kind = self._norm_kind(spec)
         self.eps = spec.get("qk_norm_eps")
         self.q_norm = self.k_norm = None
-        if self.norm_kind == "weighted_before":
+        if self.norm_kind in ("weighted_before", "weighted_rows"):
             self.q_norm = self.vector(tensors["q_layernorm.weight"])
             self.k_norm = self.vector(tensors["k_layernorm.weight"])
-            if order is not None:
+            if order is not None and self.norm_kind == "weighted_rows":
+                self.q_norm = self._reordered(self.q_norm, self.heads, order).contiguous()
+                self.k_norm = self._reordered(self.k_norm, self.kv_heads, order).contiguous()
+            elif order is not None:
                 self.q_norm = self.q_norm[order.to(self.q_norm.device)].contiguous()
                 self.k_norm = self.k_norm[order.to(self.k_norm.device)].contiguous()
         self.ops.check_attention_sizes(self.heads, self.kv_heads, self.row_dim)
         # what the plain form of the operation (one head size, weighted norm before a pure
         # rotation) does not cover goes to the kernels as extra arguments
         self.extra = {}
-        if (self.value_dim != self.head_dim or self.norm_kind == "plain_after"
-                or self.position.amplitude() != 1.0):
+        if self._general(spec):
             self.extra = dict(value_dim=self.value_dim, amplitude=self.position.amplitude(),
                               norm_after=self.norm_kind == "plain_after")
+            if self.norm_kind == "weighted_rows":
+                self.extra["norm_rows"] = True
+            if spec.get("temperature"):
+                self.extra["temperature"] = tuple(float(value) for value in spec["temperature"])
+        self.value_mix = self._value_mix(spec)
+        self.mix_factor = 0.0
+        if self.value_mix == "later":
+            self.mix_factor = float(tensors["value_mix"].to(torch.float32))
         self.sinks = {}
         if spec.get("sink"):
             self.sinks = dict(sinks=self.vector(tensors["sink"]))
         if self.keep_first:
             self.sinks["keep_first"] = self.keep_first
+        # what happens to a score between the product and the softmax
+        slopes = spec.get("distance_slopes")
+        if spec.get("score_cap") or slopes is not None:
+            if self.sinks or self.window:
+                raise ValueError("capped or distance-biased scores go without sinks and windows")
+            self.sinks["score_cap"] = float(spec.get("score_cap") or 0.0)
+            if slopes is not None:
+                slopes = torch.tensor([float(value) for value in slopes], dtype=torch.float64)
+                if slopes.numel() != self.heads:
+                    raise ValueError("one slope per query head")
+                self.sinks["slopes"] = slopes.to(torch.float32).to(runtime.device)
+                # the smallest slope of the query heads that share a key head, on the host: it bounds
+                # how far back their queries can see anything
+                self.sinks["least_slope"] = float(slopes.min())
         # (with a second product for the gate the input is read twice: it is normed once, ahead)
         self.accepts_normed_input = self.gate is None
 
     fuses_residual = True
     scales_residual = True
     accepts_normed_input = True
+
+    def _general(self, spec):
+        """Whether the preparation of queries, keys and values needs its general kernel."""
+        return (self.value_dim != self.head_dim or self._norm_kind(spec) in ("plain_after", "weighted_rows")
+                or self.position.amplitude() != 1.0 or bool(spec.get("temperature"))
+                or self._value_mix(spec) is not None)
 
     def inner_parts(self):
         return (self.position,)
@@ -234,11 +284,18 @@ class Attention(Mixer):
             qkv = self.ops.channel_conv(qkv, self.conv, None, taps=self.taps, activation=None,
                                         ctx=ctx, view=None if self.taps < 2 else cache["inputs"],
                                         write=write)
+        extra = self.extra
+        if self.value_mix is not None:
+            inner = self.kv_heads * self.value_dim
+            if self.value_mix == "first":
+                ctx.shared["values"] = qkv[:, qkv.shape[1] - inner:]
+            else:
+                extra = dict(extra, value_mix=(self.mix_factor, ctx.shared["values"]))
         mixed = self.ops.qkv_attention(
             qkv, heads=self.heads, kv_heads=self.kv_heads, head_dim=self.head_dim,
             q_weight=self.q_norm, k_weight=self.k_norm, eps=self.eps,
             rotary=self.position.rotary_table(), scale=self.scale, window=self.window, ctx=ctx,
-            view=pages, write=write, **self.sinks, **self.extra)
+            view=pages, write=write, **self.sinks, **extra)
         if self.gate_kind is not None:
             # (the heads' outputs may have rows of the pages' size: the gate leaves the values)
             mixed = self.ops.gate_heads(mixed, gate, heads=self.heads, row_dim=self.row_dim,
@@ -628,7 +685,7 @@ class LatentAttention(Mixer):
     ``query_latent`` (None: queries come straight from the mixer's input; else the size of a
     latent of their own), ``eps`` (of the latents' norms), ``position`` (a position-encoding
     PartSpec for the rotated part), ``scale``, ``gate`` (a sigmoid gate on the heads' outputs,
-    computed from the mixer's input), ``sink`` (a stored number per head, ``sink`` [heads], that
+    computed from the mixer's input: True, one number per value; ``heads``, one per head), ``sink`` (a stored number per head, ``sink`` [heads], that
     stands in the softmax's denominator as exp(sink): no key, no value, not scaled).
 
     q = W_q x, or with a query latent W_uq c_q with c_q = rms_norm(W_dq x) (``query_down``,
@@ -661,8 +718,9 @@ class LatentAttention(Mixer):
                     "up_k": TensorSpec((heads * spec["head_dim"], latent)),
                     "up_v": TensorSpec((inner, latent)),
                     "out": TensorSpec((hidden, inner))})
-        if spec.get("gate", True):
-            out["gate"] = TensorSpec((inner, hidden))
+        gate = spec.get("gate", True)
+        if gate:
+            out["gate"] = TensorSpec((heads if gate == "heads" else inner, hidden))
         if spec.get("sink"):
             out["sink"] = TensorSpec((heads,), "wide")
         return out
@@ -679,7 +737,10 @@ class LatentAttention(Mixer):
         position: PartSpec = spec.get("position") or PartSpec("none")
         self.position = POSITIONS.get(position.kind)(position, {}, runtime)
         self.neighbours = getattr(self.position, "layout", "halves") == "neighbours"
-        self.gated = bool(spec.get("gate", True))
+        gate = spec.get("gate", True)
+        if gate not in (True, False, None, "heads"):
+            raise ValueError(f"unknown gate {gate!r}")
+        self.gated, self.gate_per_head = bool(gate), gate == "heads"
         self.query_latent = int(spec.get("query_latent") or 0)
         # one product for everything that reads x: queries (or their latent) | latent and shared
         # key part | gate
@@ -739,7 +800,10 @@ class LatentAttention(Mixer):
                                           ctx=ctx, view=cache, **self.sinks)
         values = self.ops.linear_heads(mixed[:, :, :latent], self.up_v)
         values = values.view(tokens, heads * self.value_dim)
-        if self.gated:
+        if self.gate_per_head:
+            values = self.ops.gate_heads(values, projected[:, projected.shape[1] - heads:], heads=heads,
+                                         row_dim=self.value_dim, value_dim=self.value_dim, per_head=True)
+        elif self.gated:
             values = self.ops.sigmoid_gate(values, projected[:, projected.shape[1] - values.shape[1]:])
         return self.ops.linear(values, self.out)
 
@@ -907,3 +971,81 @@ class SelectiveStateSpace(Mixer):
         if residual is not None:
             raise ValueError("this mixer hands its output back")
         return out
+
+
+@MIXERS.register("rglru")
+class GatedLinearRecurrence(Mixer):
+    """Two branches of the mixer's input, one through a convolution over time and a linear recurrence
+    per channel with gated decay (the real-gated linear recurrent unit of Griffin). Parameters:
+    ``hidden``, ``width`` (channels), ``blocks`` (equal parts of the channels that the gates'
+    matrices work on), ``taps``.
+
+    y = gelu_tanh(W_y x + b_y) and u = the causal convolution over the last ``taps`` tokens of
+    W_x x + b_x (``conv`` [width, taps], last column the current token's, and ``conv.b``). Per part
+    of u: r = sigmoid(R u + b_r) and i = sigmoid(I u + b_i), with the parts' matrices ``ra``, ``ri``
+    [blocks, n, n] (out, in). Per channel: log a = -8 r softplus(lam), S = a S + sqrt(1 - a^2) i u,
+    and the output is W_o (S * y). The gates, the decay and S are 32-bit; S is zero at a request's
+    start. A request keeps S in a 32-bit slot and the convolution's last taps - 1 inputs in a slot
+    of the compute dtype."""
+
+    DECAY = 8.0
+
+    @classmethod
+    def tensors(cls, spec):
+        hidden, width, blocks = spec["hidden"], spec["width"], spec["blocks"]
+        part = width // blocks
+        return {"y": TensorSpec((width, hidden)), "y.b": TensorSpec((width,), "bias"),
+                "x": TensorSpec((width, hidden)), "x.b": TensorSpec((width,), "bias"),
+                "conv": TensorSpec((width, spec["taps"]), "wide"), "conv.b": TensorSpec((width,), "bias"),
+                "ra": TensorSpec((blocks, part, part)), "ra.b": TensorSpec((blocks, part), "bias"),
+                "ri": TensorSpec((blocks, part, part)), "ri.b": TensorSpec((blocks, part), "bias"),
+                "lam": TensorSpec((width,), "wide"), "o": TensorSpec((hidden, width))}
+
+    @classmethod
+    def cache_need(cls, spec):
+        need = {"state": FixedState((spec["width"],), "float32")}
+        if spec["taps"] > 1:
+            need["inputs"] = FixedState((spec["taps"] - 1, spec["width"]))
+        return need
+
+    def __init__(self, spec, tensors, runtime):
+        super().__init__(spec, tensors, runtime)
+        self.width, self.blocks, self.taps = spec["width"], spec["blocks"], int(spec["taps"])
+        if self.width % self.blocks:
+            raise ValueError("the channels must split into equal parts for the gates")
+        # one product for both branches: x | y
+        self.project = self.matrix(torch.cat([tensors["x"], tensors["y"]], dim=0))
+        self.project_bias = self.vector(torch.cat([tensors["x.b"], tensors["y.b"]], dim=0))
+        self.conv = self.vector(tensors["conv"])
+        self.conv_bias = self.vector(tensors["conv.b"])
+        # per part the rows of both gates: r's, then i's
+        self.gates = self.matrix(torch.cat([tensors["ra"], tensors["ri"]], dim=1))
+        self.gate_bias = self.vector(torch.cat([tensors["ra.b"], tensors["ri.b"]], dim=1))
+        # log a = rate * r, the rate worked out once
+        lam = tensors["lam"].to(torch.float64)
+        self.rate = (-self.DECAY * torch.nn.functional.softplus(lam, threshold=40.0)) \
+            .to(torch.float32).contiguous()
+        self.out = self.matrix(tensors["o"])
+
+    fuses_residual = True
+    scales_residual = True
+    accepts_normed_input = True
+
+    def input_projection(self):
+        return self.project, self.project_bias
+
+    def forward(self, x, ctx, cache, write, residual=None):
+        return self.forward_projected(self.ops.linear(x, self.project, self.project_bias), ctx, cache,
+                                      write, residual)
+
+    def forward_projected(self, projected, ctx, cache, write, residual=None):
+        u = self.ops.channel_conv(projected[:, :self.width], self.conv, self.conv_bias, taps=self.taps,
+                                  activation=None, ctx=ctx, view=cache.get("inputs"), write=write)
+        mixed = self.ops.gated_recurrence(u, projected[:, self.width:], gates=self.gates,
+                                          gate_bias=self.gate_bias, rate=self.rate, ctx=ctx,
+                                          view=cache["state"], write=write)
+        if residual is None:
+            return self.ops.linear(mixed, self.out)
+        if self.residual_scale != 1.0:
+            return self.ops.linear_add(mixed, self.out, None, residual, scale=self.residual_scale)
+        return self.ops.linear_add(mixed, self.out, None, residual)

@@ -6,7 +6,7 @@ from typing import Any, Mapping
 
 import torch
 
-from .base import Runtime, StepContext
+from .base import NormedUpdate, Runtime, StepContext
 from .registry import BLOCKS, EMBEDDINGS, FEED_FORWARDS, MIXERS, NORMS
 from .spec import LayerCall, ModelSpec, PartSpec, TensorSpec
 
@@ -191,12 +191,19 @@ class Model:
                 all(block.parallel_streams for block in self.layers)
                 and all(call.inject is None for call in self.order)):
             raise ValueError("parallel streams run through all layers, and nothing is injected into them")
+        # blocks that hand on outputs that are still to be normed (see Block.normed_updates)
+        if any(block.normed_updates for block in self.layers) and not (
+                all(block.normed_updates for block in self.layers)
+                and all(call.inject is None for call in self.order)):
+            raise ValueError("blocks that hand on normed updates come together, and nothing is injected "
+                             "between them")
         self.own_caches = [bool(type(block).cache_need(block.spec)) for block in self.layers]
         # For debugging: called as observer(place, residual, delta) after the embedding
         # (place -1) and after every call of a layer (place = its number in the order); the
         # hidden state there is residual + s * delta, s the block's ``pending_scale`` (1 unless the
         # architecture gives its parts' outputs a factor); with parallel streams it is the sum over
-        # the streams of delta.applied(residual) (of ``residual`` while delta is None). It sees
+        # the streams of delta.applied(residual) (of ``residual`` while delta is None), and where the
+        # blocks hand on normed updates it is delta.applied(residual). It sees
         # the step's own tensors (a step's rows may be followed by fillers): copy what is to be
         # kept. Steps that are replayed from a CUDA graph do not call it.
         self.observer = None
@@ -220,6 +227,7 @@ class Model:
         if self.parallel_streams:
             residual = residual.unsqueeze(1)            # one stream as yet: they are all equal
         delta, scale = None, 1.0
+        ctx.shared.clear()
         if self.observer is not None:
             self.observer(-1, residual, delta)
         for place, call in enumerate(self.order):
@@ -269,6 +277,9 @@ class Model:
             picked, picked_delta = self.ops.sum_streams(residual, delta, rows), None
         elif rows is None:
             picked, picked_delta = residual, delta
+        elif isinstance(delta, NormedUpdate):
+            picked, output = self.ops.gather_rows(residual, delta.output, rows)
+            picked_delta = delta.of(output)
         else:
             picked, picked_delta = self.ops.gather_rows(residual, delta, rows)
         # the output product may apply the norm itself where the kernels can do that

@@ -2,7 +2,7 @@
 
 from __future__ import annotations
 
-from .base import Norm, NormedInput
+from .base import Norm, NormedInput, NormedUpdate
 from .registry import NORMS
 from .spec import TensorSpec
 
@@ -47,3 +47,27 @@ class RMSNorm(Norm):
         """In place: residual += x * rsqrt(mean(x^2) + eps) * weight, the norm taken over a part's
         output ``x`` (compute dtype) and everything in 32-bit."""
         self.ops.normed_mean_add(residual, [x], [self.weight], self.eps)
+
+
+@NORMS.register("layernorm")
+class LayerNorm(Norm):
+    """(v - mean) * rsqrt(variance + eps) * weight + bias over the last axis, the variance being the
+    mean of the squared deviations; 32-bit, fused with what is added to the stream before it: a
+    plain output, or one that is normed itself (``NormedUpdate``). Parameters: ``size``, ``eps``."""
+
+    @classmethod
+    def tensors(cls, spec):
+        return {"weight": TensorSpec((spec["size"],), "norm"), "bias": TensorSpec((spec["size"],), "bias")}
+
+    def __init__(self, spec, tensors, runtime):
+        super().__init__(spec, tensors, runtime)
+        self.weight, self.bias = self.vector(tensors["weight"]), self.vector(tensors["bias"])
+        self.eps = float(spec["eps"])
+
+    def forward(self, residual, delta, lazy=False, delta_scale=1.0):
+        return self.ops.add_norm(residual, delta, self.weight, self.bias, self.eps,
+                                 self.runtime.dtype, delta_scale=delta_scale)
+
+    def update(self, output):
+        """residual + norm(output), still to be added."""
+        return NormedUpdate(output, self.weight, self.bias, self.eps)

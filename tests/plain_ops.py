@@ -41,6 +41,15 @@ class PlainOps:
         inv = torch.rsqrt(residual.pow(2).mean(dim=-1, keepdim=True) + eps)
         return (residual * inv * weight).to(dtype)
 
+    def add_norm(self, residual, delta, weight, bias, eps, dtype, delta_scale=1.0):
+        if delta is not None and hasattr(delta, "applied"):
+            residual.copy_(delta.applied(residual))
+        elif delta is not None:
+            residual += delta.float() * delta_scale
+        x = residual if bias is None else residual - residual.mean(dim=-1, keepdim=True)
+        x = x * torch.rsqrt(x.pow(2).mean(dim=-1, keepdim=True) + eps) * weight
+        return (x if bias is None else x + bias).to(dtype)
+
     def gather_rows(self, residual, delta, rows):
         index = rows.long()
         return residual[index].clone(), None if delta is None else delta[index].clone()
@@ -59,9 +68,15 @@ class PlainOps:
     def linear_add(self, a, w, bias, residual, scale=1.0):
         return self.linear(a, w, bias)      # (the caller adds it, with its factor)
 
-    def linear_gated(self, a, gate_up, kind):
+    def linear_gated(self, a, gate_up, kind, limits=None):
         both = self.linear(a, gate_up)
         width = both.shape[1] // 2
+        if kind == "clamped":
+            first, second, boundary = limits
+            limit = torch.where(torch.arange(width) < boundary, first, second)
+            g = torch.minimum(both[:, :width].float(), limit)
+            u = torch.maximum(torch.minimum(both[:, width:].float(), limit), -limit)
+            return (g * torch.sigmoid(1.702 * g) * (u + 1)).to(a.dtype)
         return (self.activation(both[:, :width], kind).float() * both[:, width:].float()).to(a.dtype)
 
     def swiglu(self, gate_up):
@@ -105,12 +120,24 @@ class PlainOps:
 
     def qk_norm_rope_store(self, qkv, *, heads, kv_heads, head_dim, q_weight, k_weight, eps,
                            rotary, ctx, view, write, value_dim=None, amplitude=1.0,
-                           norm_after=False):
+                           norm_after=False, norm_rows=False, temperature=None, value_mix=None):
         tokens = qkv.shape[0]
         dtype = qkv.dtype
         value_dim = value_dim or head_dim
         row_dim = view.kv.shape[-1]
-        flat = qkv.float()
+        flat = qkv.float().clone()
+        q_size, k_size = heads * head_dim, kv_heads * head_dim
+        if norm_rows:
+            for lo, hi, weight in ((0, q_size, q_weight), (q_size, q_size + k_size, k_weight)):
+                flat[:, lo:hi] = self._normed(flat[:, lo:hi], weight, eps)
+            q_weight = k_weight = None
+        if temperature is not None:
+            coef, every = temperature
+            steps = torch.floor((ctx.positions.double() + 1) / every)
+            flat[:, :q_size] *= (1 + coef * torch.log(steps + 1)).float()[:, None]
+        if value_mix is not None:
+            factor, first = value_mix
+            flat[:, q_size + k_size:] = (1 - factor) * flat[:, q_size + k_size:] + factor * first.float()
         q = flat[:, :heads * head_dim].view(tokens, heads, head_dim)
         k = flat[:, heads * head_dim:(heads + kv_heads) * head_dim].view(tokens, kv_heads, head_dim)
         v = flat[:, (heads + kv_heads) * head_dim:].view(tokens, kv_heads, value_dim)
@@ -152,13 +179,14 @@ class PlainOps:
 
     def qkv_attention(self, qkv, *, heads, kv_heads, head_dim, q_weight, k_weight, eps, rotary,
                       scale, window, ctx, view, write, sinks=None, chunk=None, keep_first=0,
-                      **extra):
+                      score_cap=0.0, slopes=None, least_slope=0.0, **extra):
         q = self.qk_norm_rope_store(qkv, heads=heads, kv_heads=kv_heads, head_dim=head_dim,
                                     q_weight=q_weight, k_weight=k_weight, eps=eps, rotary=rotary,
                                     ctx=ctx, view=view, write=write, **extra)
         return self.paged_attention(q, heads=heads, kv_heads=kv_heads, head_dim=view.kv.shape[-1],
                                     scale=scale, window=window, ctx=ctx, view=view, sinks=sinks,
-                                    chunk=chunk, keep_first=keep_first)
+                                    chunk=chunk, keep_first=keep_first, score_cap=score_cap,
+                                    slopes=slopes)
 
     def concat_stream(self, residual, delta, token_ids, table, dtype, delta_scale=1.0):
         stream = residual if delta is None else residual + delta.float() * delta_scale
@@ -498,7 +526,8 @@ class PlainOps:
         return out.reshape(tokens, inner).to(projected.dtype)
 
     def paged_attention(self, q, *, heads, kv_heads, head_dim, scale, window, ctx, view,
-                        sinks=None, chunk=None, keep_first=0):
+                        sinks=None, chunk=None, keep_first=0, score_cap=0.0, slopes=None,
+                        least_slope=0.0):
         tokens = q.shape[0]
         out = torch.empty(tokens, heads, head_dim)
         positions = ctx.positions.tolist()
@@ -519,6 +548,10 @@ class PlainOps:
             k = k.repeat_interleave(group, dim=1)
             v = v.repeat_interleave(group, dim=1)
             scores = torch.einsum("hd,khd->hk", q[t].float(), k) * scale
+            if score_cap:
+                scores = score_cap * torch.tanh(scores / score_cap)
+            if slopes is not None:
+                scores = scores - slopes[:, None] * (p - torch.tensor(keys)).float()
             if sinks is not None:
                 # a column without a key or a value: it only takes its share of the weights
                 scores = torch.cat([scores, sinks.float()[:, None]], dim=1)
@@ -555,6 +588,26 @@ class PlainOps:
         elif activation is not None:
             raise ValueError(activation)
         return out.to(dtype)
+
+    def gated_recurrence(self, u, y, *, gates, gate_bias, rate, ctx, view, write):
+        tokens, width = u.shape
+        blocks, part = gates.shape[0], gates.shape[2]
+        flat = u.float()
+        z = torch.einsum("tbn,bmn->tbm", flat.view(tokens, blocks, part), gates.float()) + gate_bias
+        z = torch.sigmoid(z)
+        r, i = z[:, :, :part].reshape(tokens, width), z[:, :, part:].reshape(tokens, width)
+        log_a = rate * r
+        a, add = torch.exp(log_a), torch.sqrt(-torch.expm1(2 * log_a)) * i * flat
+        out = torch.empty(tokens, width)
+        starts, slots = ctx.request_start.tolist(), view.slots.tolist()
+        for q in range(ctx.requests):
+            state = view.state[slots[q]].clone()
+            for t in range(starts[q], starts[q + 1]):
+                state = a[t] * state + add[t]
+                out[t] = state
+            if write:
+                view.state[slots[q]] = state
+        return (out * self.activation(y.float(), "gelu_tanh")).to(u.dtype)
 
     def gate_heads(self, mixed, gate, *, heads, row_dim, value_dim, per_head):
         tokens = mixed.shape[0]
