@@ -8,10 +8,12 @@
 // on its position, never on how the tokens were cut into steps or batched. `sinks` (float32
 // [heads] or null) adds exp(sink) of the query's head to the softmax's denominator. With
 // `keep_first` the keys at positions below it stay visible behind a window: their blocks come
-// first, the blocks between them and the window's first are skipped.
+// first, the blocks between them and the window's first are skipped. With SHAPED a score passes a cap
+// and a distance bias ahead of the softmax (score_shape.cuh).
 //
 // This kernel serves the 32-bit engine and every shape that the faster kernels refuse.
 #include "common.cuh"
+#include "score_shape.cuh"
 
 namespace {
 
@@ -19,15 +21,15 @@ constexpr int WARPS = 4;
 constexpr int MAX_HEAD_DIM = 1024;
 constexpr int MAX_ACC = MAX_HEAD_DIM / 32;
 
-template <typename T>
+template <typename T, bool SHAPED>
 __global__ void __launch_bounds__(WARPS * 32)
 attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ kv,
                          const int* __restrict__ block_table, int table_width, int page_size,
                          long long kv_half, const int* __restrict__ positions,
                          const int* __restrict__ token_request, T* __restrict__ out, int tokens,
                          int heads, int kv_heads, int head_dim, float scale, int window,
-                         int keep_first, const float* __restrict__ sinks,
-                         int* __restrict__ error_flag) {
+                         int keep_first, const float* __restrict__ sinks, float cap,
+                         const float* __restrict__ slopes, int* __restrict__ error_flag) {
     extern __shared__ float shared[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long item = (long long)blockIdx.x * WARPS + warp;
@@ -73,6 +75,10 @@ attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ kv,
                 float dot = 0.f;
                 for (int e = 0; e < head_dim; ++e) dot = fmaf(query[e], to_float<T>(key_row[e]), dot);
                 score = dot;
+                if (SHAPED) {
+                    if (cap > 0.f) score = cap * tanhf(score / cap);
+                    if (slopes != nullptr) score = fmaf(-slopes[head], (float)(position - key), score);
+                }
             }
         }
         const float block_max = warp_max(score);
@@ -115,7 +121,8 @@ static int attention_generic_launch(const void* q, const void* kv, const int* bl
                                     const int* token_request, void* out, int tokens, int heads,
                                     int kv_heads, int head_dim, float scale, int window, int dtype,
                                     const float* sinks, int planes, int* error_flag,
-                                    cudaStream_t stream, int keep_first) {
+                                    cudaStream_t stream, int keep_first, float cap = 0.f,
+                                    const float* slopes = nullptr) {
     if (tokens == 0) return 0;
     MLXONE_REQUIRE(tokens > 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0,
                    "attention: %d heads cannot share %d key heads", heads, kv_heads);
@@ -127,19 +134,20 @@ static int attention_generic_launch(const void* q, const void* kv, const int* bl
     const size_t shared = (size_t)WARPS * head_dim * sizeof(float);
     MLXONE_REQUIRE(planes == 1 || planes == 2, "attention: one or two planes, not %d", planes);
     const long long kv_half = planes == 1 ? 0 : (long long)pages * kv_heads * page_size * head_dim;
+#define LAUNCH(T, SHAPED)                                                                          \
+    attention_generic_kernel<T, SHAPED><<<blocks, WARPS * 32, shared, stream>>>(                   \
+        (const T*)q, (const T*)kv, block_table, table_width, page_size, kv_half, positions,        \
+        token_request, (T*)out, tokens, heads, kv_heads, head_dim, scale, window, keep_first,      \
+        sinks, cap, slopes, error_flag)
+    const bool shaped = cap > 0.f || slopes != nullptr;
     if (dtype == MLXONE_BF16) {
-        using T = __nv_bfloat16;
-        attention_generic_kernel<T><<<blocks, WARPS * 32, shared, stream>>>(
-            (const T*)q, (const T*)kv, block_table, table_width, page_size, kv_half, positions,
-            token_request, (T*)out, tokens, heads, kv_heads, head_dim, scale, window, keep_first,
-            sinks, error_flag);
+        if (shaped) LAUNCH(__nv_bfloat16, true);
+        else LAUNCH(__nv_bfloat16, false);
     } else {
-        using T = float;
-        attention_generic_kernel<T><<<blocks, WARPS * 32, shared, stream>>>(
-            (const T*)q, (const T*)kv, block_table, table_width, page_size, kv_half, positions,
-            token_request, (T*)out, tokens, heads, kv_heads, head_dim, scale, window, keep_first,
-            sinks, error_flag);
+        if (shaped) LAUNCH(float, true);
+        else LAUNCH(float, false);
     }
+#undef LAUNCH
     MLXONE_LAUNCH_CHECK("attention_generic");
     return 0;
 }
@@ -183,4 +191,18 @@ MLXONE_API int mlxone_attention_generic_keep(const void* q, const void* kv, cons
     return attention_generic_launch(q, kv, block_table, table_width, page_size, pages, positions,
                                     token_request, out, tokens, heads, kv_heads, head_dim, scale,
                                     window, dtype, sinks, 2, error_flag, stream, keep_first);
+}
+
+// ... with scores s that become cap tanh(s / cap) (cap 0: none) and then lose slopes[head] (float32
+// [heads] or null) times the distance between query and key
+MLXONE_API int mlxone_attention_generic_shaped(const void* q, const void* kv, const int* block_table,
+                                               int table_width, int page_size, int pages,
+                                               const int* positions, const int* token_request,
+                                               void* out, int tokens, int heads, int kv_heads,
+                                               int head_dim, float scale, float cap,
+                                               const float* slopes, int dtype, int* error_flag,
+                                               cudaStream_t stream) {
+    return attention_generic_launch(q, kv, block_table, table_width, page_size, pages, positions,
+                                    token_request, out, tokens, heads, kv_heads, head_dim, scale, 0,
+                                    dtype, nullptr, 2, error_flag, stream, 0, cap, slopes);
 }

@@ -18,6 +18,7 @@
 #include <cuda_pipeline_primitives.h>
 
 #include "common.cuh"
+#include "score_shape.cuh"
 
 namespace {
 
@@ -149,13 +150,16 @@ __device__ __forceinline__ void load_tile(bf16* k_tile, bf16* v_tile, const Page
 // One warp: 16 query rows (their fragments in `qf`) against one tile of KEYS keys.
 // `limit_lo[i]`/`limit_hi[i]` (i = 0: row lane/4, 1: row lane/4 + 8) bound the keys that the row
 // may see; with MASKED false the caller has checked that every row sees the whole tile.
-// Updates the running max `m` (of score * scale * log2 e), the sum `l` and `o`.
-template <int HD, int KEYS, bool MASKED>
+// Updates the running max `m` (of score * scale * log2 e), the sum `l` and `o`. With SHAPED the scores
+// pass `shape` first, the distance bias with slope `slope` (in units of log2 e) from the rows'
+// positions `at` on.
+template <int HD, int KEYS, bool MASKED, bool SHAPED>
 __device__ __forceinline__ void attend_tile(const uint32_t (&qf)[HD / 16][4], const bf16* k_tile,
                                             const bf16* v_tile, int first, const int (&limit_lo)[2],
                                             const int (&limit_hi)[2], float scale_log2,
                                             float (&m)[2], float (&l)[2], float (&o)[HD / 8][4],
-                                            int lane, int kept = 0) {
+                                            int lane, int kept, const ScoreShape& shape, float slope,
+                                            const int (&at)[2]) {
     using T = Tile<HD>;
     float s[KEYS / 8][4];
 #pragma unroll
@@ -178,6 +182,21 @@ __device__ __forceinline__ void attend_tile(const uint32_t (&qf)[HD / 16][4], co
 
     // the tile's row maxima (of the raw scores; masked ones count as -inf)
     const int t2 = (lane & 3) * 2;
+    if (SHAPED) {
+#pragma unroll
+        for (int j = 0; j < KEYS / 8; j += 4) {
+            float piece[16];
+#pragma unroll
+            for (int c = 0; c < 16; ++c) piece[c] = s[j + (c >> 2)][c & 3];
+            shape_scores<16>(piece, shape);
+#pragma unroll
+            for (int c = 0; c < 16; ++c) {
+                const int key = first + (j + (c >> 2)) * 8 + t2 + (c & 1);
+                s[j + (c >> 2)][c & 3] = fmaf(-slope, (float)(at[(c >> 1) & 1] - key), piece[c]);
+            }
+        }
+        scale_log2 = 1.f;
+    }
     float tile_max[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int j = 0; j < KEYS / 8; ++j)
@@ -246,14 +265,14 @@ __device__ __forceinline__ void attend_tile(const uint32_t (&qf)[HD / 16][4], co
 constexpr int PREFILL_WARPS = 4;       // 8 warps (128 rows) measured the same on long prompts
 constexpr int ROWS = 16 * PREFILL_WARPS;      // query rows per block
 
-template <int HD>
+template <int HD, bool SHAPED>
 __global__ void __launch_bounds__(PREFILL_WARPS * 32)
 attention_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv, long long kv_half,
                          const int* __restrict__ block_table, int table_width, int page_size,
                          const int* __restrict__ request_start, const int* __restrict__ history,
                          bf16* __restrict__ out, int requests, int heads, int kv_heads,
                          float scale_log2, int window, const float* __restrict__ sinks,
-                         int keep_first) {
+                         int keep_first, ScoreShape shape) {
     using T = Tile<HD>;
     constexpr int KEYS = PREFILL_KEYS;
     extern __shared__ __align__(16) unsigned char shared_bytes[];
@@ -279,6 +298,11 @@ attention_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv
     if (request < 0) return;
     const int row_start = found[1];
     const int head = blockIdx.y;
+    float slope = 0.f;
+    if (SHAPED) {
+        if (shape.slopes != nullptr) slope = shape.slopes[head] * LOG2E;
+        window = shape_window(shape, head, 1);
+    }
     const int first_token = request_start[request];
     const int count = request_start[request + 1] - first_token;
     const int rows = min(ROWS, count - row_start);
@@ -314,11 +338,12 @@ attention_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv
     copy_commit();
 
     // per-thread rows: lane/4 and lane/4 + 8 of the warp's 16
-    int limit_lo[2], limit_hi[2];
+    int limit_lo[2], limit_hi[2], at[2];
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
         const int row = warp * 16 + (lane >> 2) + i * 8;
         const int position = first_position + row;
+        at[i] = position;
         limit_hi[i] = row < rows ? position : -1;
         limit_lo[i] = first_visible_key(position, window);
     }
@@ -372,11 +397,12 @@ attention_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv
             const bool open = warp_whole && tile * KEYS >= open_lo &&
                               tile * KEYS + KEYS - 1 <= warp_first;
             if (open)
-                attend_tile<HD, KEYS, false>(qf, k_now, v_now, tile * KEYS, limit_lo, limit_hi,
-                                             scale_log2, m, l, o, lane);
+                attend_tile<HD, KEYS, false, SHAPED>(qf, k_now, v_now, tile * KEYS, limit_lo, limit_hi,
+                                                     scale_log2, m, l, o, lane, 0, shape, slope, at);
             else
-                attend_tile<HD, KEYS, true>(qf, k_now, v_now, tile * KEYS, limit_lo, limit_hi,
-                                            scale_log2, m, l, o, lane, keep_first);
+                attend_tile<HD, KEYS, true, SHAPED>(qf, k_now, v_now, tile * KEYS, limit_lo, limit_hi,
+                                                    scale_log2, m, l, o, lane, keep_first, shape, slope,
+                                                    at);
         }
         __syncthreads();
     }
@@ -436,9 +462,10 @@ struct DecodePrep {
     int write_kv = 0;
     int* error_flag = nullptr;
     int keep_first = 0;                   // positions below this stay visible behind a window
+    ScoreShape shape;                     // what happens to the scores (with SHAPED)
 };
 
-template <int HD, bool CLUSTER, bool PREP>
+template <int HD, bool CLUSTER, bool PREP, bool SHAPED>
 __global__ void __launch_bounds__(DECODE_WARPS * 32)
 attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv, long long kv_half,
                         const int* __restrict__ block_table, int table_width, int page_size,
@@ -462,6 +489,15 @@ attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv,
     const int g = lane >> 2, t = lane & 3;
 
     const int position = positions[request];
+    float slope[2] = {0.f, 0.f};               // of this lane's heads 2t and 2t + 1, times log2 e
+    if (SHAPED) {
+        if (prep.shape.slopes != nullptr) {
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+                slope[i] = prep.shape.slopes[head0 + min(2 * t + i, rows - 1)] * LOG2E;
+        }
+        window = shape_window(prep.shape, head0, rows);
+    }
     const int lowest = first_visible_key(position, window);
     // Tiles are counted in the order they are walked: first those of the first positions that
     // stay visible behind a window, then the window's; tile_at gives a tile's place among the keys.
@@ -706,6 +742,17 @@ attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv,
                 mma_16816(s[mt], a, qb[kk][0], qb[kk][1]);
             }
         }
+        if (SHAPED) {
+            float piece[KEYS / 4];
+#pragma unroll
+            for (int c = 0; c < KEYS / 4; ++c) piece[c] = s[c >> 2][c & 3];
+            shape_scores<KEYS / 4>(piece, prep.shape);
+#pragma unroll
+            for (int c = 0; c < KEYS / 4; ++c) {
+                const int key = first + (c >> 2) * 16 + g + ((c >> 1) & 1) * 8;
+                s[c >> 2][c & 3] = fmaf(-slope[c & 1], (float)(position - key), piece[c]);
+            }
+        }
         float tile_max[2] = {-INFINITY, -INFINITY};
 #pragma unroll
         for (int mt = 0; mt < KEYS / 16; ++mt)
@@ -713,7 +760,7 @@ attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv,
             for (int c = 0; c < 4; ++c) {
                 const int key = first + mt * 16 + g + (c >> 1) * 8;
                 const bool seen = (key >= lowest || key < kept) && key <= position && head_live[c & 1];
-                s[mt][c] = seen ? s[mt][c] * scale_log2 : -INFINITY;
+                s[mt][c] = seen ? (SHAPED ? s[mt][c] : s[mt][c] * scale_log2) : -INFINITY;
                 tile_max[c & 1] = fmaxf(tile_max[c & 1], s[mt][c]);
             }
         float correction[2];
@@ -924,21 +971,22 @@ __global__ void attention_merge_kernel(const float* __restrict__ partial, bf16* 
     }
 }
 
-template <int HD>
+template <int HD, bool SHAPED = false>
 int launch_prefill(const void* q, const void* kv, long long kv_half, const int* block_table,
                    int table_width, int page_size, const int* request_start, const int* history,
                    void* out, int tokens, int requests, int heads, int kv_heads, float scale,
-                   int window, const float* sinks, cudaStream_t stream, int keep_first = 0) {
+                   int window, const float* sinks, cudaStream_t stream, int keep_first = 0,
+                   ScoreShape shape = ScoreShape()) {
     using T = Tile<HD>;
     const size_t shared = (size_t)(ROWS + 4 * PREFILL_KEYS) * T::STRIDE * 2;
-    auto kernel = attention_prefill_kernel<HD>;
+    auto kernel = attention_prefill_kernel<HD, SHAPED>;
     if (shared > 48 * 1024)
         cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
     const dim3 grid((tokens + ROWS - 1) / ROWS + requests, heads);
     kernel<<<grid, PREFILL_WARPS * 32, shared, stream>>>(
         (const bf16*)q, (const bf16*)kv, kv_half, block_table, table_width, page_size,
         request_start, history, (bf16*)out, requests, heads, kv_heads, scale * LOG2E, window,
-        sinks, keep_first);
+        sinks, keep_first, shape);
     return 0;
 }
 
@@ -948,7 +996,7 @@ size_t decode_shared_bytes(int head_dim) {
     return tiles > merge ? tiles : merge;
 }
 
-template <int HD, bool PREP>
+template <int HD, bool PREP, bool SHAPED = false>
 int launch_decode(const void* q, const void* kv, long long kv_half, const int* block_table,
                   int table_width, int page_size, const int* positions, void* out, float* partial,
                   int requests, int heads, int kv_heads, int splits, float scale, int window,
@@ -960,7 +1008,7 @@ int launch_decode(const void* q, const void* kv, long long kv_half, const int* b
     const float scale_log2 = scale * LOG2E;
     // 2 to 8 splits without a scratch buffer: a cluster of the splits' blocks merges them itself
     if (splits > 1 && splits <= 8 && partial == nullptr) {
-        auto kernel = attention_decode_kernel<HD, true, PREP>;
+        auto kernel = attention_decode_kernel<HD, true, PREP, SHAPED>;
         if (shared > 48 * 1024)
             cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
         cudaLaunchConfig_t config = {};
@@ -987,7 +1035,7 @@ int launch_decode(const void* q, const void* kv, long long kv_half, const int* b
         }
         return 0;
     }
-    auto kernel = attention_decode_kernel<HD, false, PREP>;
+    auto kernel = attention_decode_kernel<HD, false, PREP, SHAPED>;
     if (shared > 48 * 1024)
         cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
     launch_kernel(kernel, grid, dim3(DECODE_WARPS * 32), shared, stream, true, (const bf16*)q,
@@ -1145,6 +1193,61 @@ MLXONE_API int mlxone_attention_decode_keep(const void* q, const void* kv, const
     MLXONE_HEAD_DIMS(CALL)
 #undef CALL
     MLXONE_LAUNCH_CHECK("attention_decode");
+    return 0;
+}
+
+// ... with scores s that become cap tanh(s / cap) (cap 0: none) and then lose slopes[head] (float32
+// [heads] or null) times the distance between query and key
+MLXONE_API int mlxone_attention_decode_shaped(const void* q, const void* kv, const int* block_table,
+                                              int table_width, int page_size, int pages,
+                                              const int* positions, void* out, float* partial,
+                                              int requests, int heads, int kv_heads, int head_dim,
+                                              int splits, float scale, float cap,
+                                              const float* slopes, cudaStream_t stream) {
+    if (requests == 0) return 0;
+    MLXONE_REQUIRE(requests > 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0,
+                   "attention_decode: bad sizes");
+    MLXONE_REQUIRE(requests <= 65535 && splits >= 1 && splits <= 65535,
+                   "attention_decode: at most 65535 requests and splits");
+    MLXONE_REQUIRE(splits <= 8 || partial != nullptr,
+                   "attention_decode: more than 8 splits need a scratch buffer");
+    MLXONE_REQUIRE(page_size > 0 && pages > 0 && table_width > 0,
+                   "attention_decode: bad page geometry");
+    const long long kv_half = (long long)pages * kv_heads * page_size * head_dim;
+    DecodePrep prep;
+    prep.shape = make_score_shape(scale, cap, slopes);
+#define CALL(HD)                                                                               \
+    launch_decode<HD, false, true>(q, kv, kv_half, block_table, table_width, page_size,        \
+                                   positions, out, partial, requests, heads, kv_heads, splits, \
+                                   scale, 0, nullptr, stream, prep)
+    MLXONE_HEAD_DIMS(CALL)
+#undef CALL
+    MLXONE_LAUNCH_CHECK("attention_decode");
+    return 0;
+}
+
+// As mlxone_attention_prefill with capped and distance-biased scores.
+MLXONE_API int mlxone_attention_prefill_shaped(const void* q, const void* kv, const int* block_table,
+                                               int table_width, int page_size, int pages,
+                                               const int* request_start, const int* history,
+                                               void* out, int tokens, int requests, int heads,
+                                               int kv_heads, int head_dim, float scale, float cap,
+                                               const float* slopes, cudaStream_t stream) {
+    if (tokens == 0) return 0;
+    MLXONE_REQUIRE(tokens > 0 && requests > 0 && heads > 0 && kv_heads > 0 &&
+                       heads % kv_heads == 0, "attention_prefill: bad sizes");
+    MLXONE_REQUIRE(heads <= 65535, "attention_prefill: too many heads");
+    MLXONE_REQUIRE(page_size > 0 && pages > 0 && table_width > 0,
+                   "attention_prefill: bad page geometry");
+    const long long kv_half = (long long)pages * kv_heads * page_size * head_dim;
+    const ScoreShape shape = make_score_shape(scale, cap, slopes);
+#define CALL(HD)                                                                               \
+    launch_prefill<HD, true>(q, kv, kv_half, block_table, table_width, page_size,              \
+                             request_start, history, out, tokens, requests, heads, kv_heads,   \
+                             scale, 0, nullptr, stream, 0, shape)
+    MLXONE_HEAD_DIMS(CALL)
+#undef CALL
+    MLXONE_LAUNCH_CHECK("attention_prefill");
     return 0;
 }
 

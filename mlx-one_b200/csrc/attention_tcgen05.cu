@@ -39,6 +39,7 @@
 #include <cuda.h>
 
 #include "common.cuh"
+#include "score_shape.cuh"
 
 namespace {
 
@@ -211,6 +212,11 @@ __device__ __forceinline__ unsigned long long fma_pair(unsigned long long a, uns
     asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
     return d;
 }
+__device__ __forceinline__ unsigned long long mul_pair(unsigned long long a, unsigned long long b) {
+    unsigned long long d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
 __device__ __forceinline__ unsigned long long add_pair(unsigned long long a, unsigned long long b) {
     unsigned long long d;
     asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
@@ -260,6 +266,7 @@ struct Item {
     // from `tile_first` on.
     int kept_first;
     int kept_tiles;
+    int window;             // as the kernel's, or what the shape of the scores leaves to be seen
 };
 
 // the place among the keys of the j-th tile that an item walks
@@ -267,7 +274,55 @@ __device__ __forceinline__ int tile_of(const Item& item, int j) {
     return j < item.kept_tiles ? item.kept_first + j : item.tile_first + j - item.kept_tiles;
 }
 
-template <int KEYS, int PARTS>
+// What a thread does to its raw products v of one tile when scores are shaped: the cap, then the
+// distance bias. `ahead` is the distance of the query to the thread's first key. Two values an
+// instruction; lanes take the polynomial of the tanh or its general form together.
+template <int N>
+__device__ __forceinline__ void shape_tile(float (&v)[N], const ScoreShape& shape, float slope, float ahead) {
+    float top = 0.f;
+#pragma unroll
+    for (int i = 0; i < N; i += 2) top = max_of_three(top, fabsf(v[i]), fabsf(v[i + 1]));
+    const unsigned long long fall = pair_of(-slope, -slope);
+    unsigned long long away = pair_of(ahead, ahead - 1.f);
+    const unsigned long long nearer = pair_of(-2.f, -2.f);
+    if (shape.outer == 0.f) {
+        const unsigned long long plain = pair_of(shape.plain, shape.plain), none = pair_of(0.f, 0.f);
+#pragma unroll
+        for (int i = 0; i < N; i += 2) {
+            const unsigned long long bias = fma_pair(fall, away, none);
+            unpair(fma_pair(pair_of(v[i], v[i + 1]), plain, bias), v[i], v[i + 1]);
+            away = add_pair(away, nearer);
+        }
+    } else if (__any_sync(0xffffffffu, top * fabsf(shape.inner) > 1.f)) {
+#pragma unroll
+        for (int i = 0; i < N; ++i)
+            v[i] = fmaf(-slope, ahead - (float)i, shape.outer * tanh_any(v[i] * shape.inner));
+    } else {
+        // (t P(t^2) with t = inner v and the factor outer in the coefficients)
+        const float o = shape.outer;
+        const unsigned long long c0 = pair_of(o * MLXONE_TANH_C0, o * MLXONE_TANH_C0);
+        const unsigned long long c1 = pair_of(o * MLXONE_TANH_C1, o * MLXONE_TANH_C1);
+        const unsigned long long c2 = pair_of(o * MLXONE_TANH_C2, o * MLXONE_TANH_C2);
+        const unsigned long long c3 = pair_of(o * MLXONE_TANH_C3, o * MLXONE_TANH_C3);
+        const unsigned long long c4 = pair_of(o * MLXONE_TANH_C4, o * MLXONE_TANH_C4);
+        const unsigned long long c5 = pair_of(o * MLXONE_TANH_C5, o * MLXONE_TANH_C5);
+        const unsigned long long inner = pair_of(shape.inner, shape.inner);
+#pragma unroll
+        for (int i = 0; i < N; i += 2) {
+            const unsigned long long t = mul_pair(pair_of(v[i], v[i + 1]), inner);
+            const unsigned long long x = mul_pair(t, t);
+            unsigned long long p = fma_pair(x, c5, c4);
+            p = fma_pair(x, p, c3);
+            p = fma_pair(x, p, c2);
+            p = fma_pair(x, p, c1);
+            p = fma_pair(x, p, c0);
+            unpair(fma_pair(t, p, mul_pair(fall, away)), v[i], v[i + 1]);
+            away = add_pair(away, nearer);
+        }
+    }
+}
+
+template <int KEYS, int PARTS, bool SHAPED>
 __global__ void __launch_bounds__((4 * PARTS + 2) * 32, Shape<KEYS>::BLOCKS_PER_SM)
 attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q,
                          const __grid_constant__ CUtensorMap map_kv, long long value_rows,
@@ -276,7 +331,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q,
                          const int* __restrict__ history, bf16* __restrict__ out, int requests,
                          int heads, int kv_heads, float scale_log2, int window, int token_tiles,
                          int splits, float* __restrict__ partial, const float* __restrict__ sinks,
-                         int* __restrict__ error_flag, int keep_first) {
+                         int* __restrict__ error_flag, int keep_first, ScoreShape shape) {
     using S = Shape<KEYS>;
     constexpr int COPY_WARP = 4 * PARTS, MMA_WARP = 4 * PARTS + 1;
     constexpr int THREADS = (4 * PARTS + 2) * 32;     // softmax warps, the copy warp, the product warp
@@ -323,7 +378,8 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q,
                 item.tokens_here = min(tile_tokens, count - token_start);
                 item.first_position = history[r] + token_start;
                 const int last_position = item.first_position + item.tokens_here - 1;
-                const int lowest = first_visible_key(item.first_position, window);
+                item.window = SHAPED ? shape_window(shape, item.kv_head * group, group) : window;
+                const int lowest = first_visible_key(item.first_position, item.window);
                 item.tile_first = lowest / KEYS;
                 // the kept first positions' tiles that lie wholly ahead of the window's first
                 const int kept = min((min(keep_first, lowest) + KEYS - 1) / KEYS, item.tile_first);
@@ -413,7 +469,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q,
             ++taken;
             const int* table = block_table + (size_t)item.request * table_width;
             const int last_position = item.first_position + item.tokens_here - 1;
-            const int lowest = first_visible_key(item.first_position, window);
+            const int lowest = first_visible_key(item.first_position, item.window);
             // this lane's box of the item's tile j: its rows in the cache, if some query row
             // may see its keys
             auto box_row = [&](int j) {
@@ -551,11 +607,14 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q,
             const int position = item.first_position + token;
             const int last_position = item.first_position + item.tokens_here - 1;
             const int limit_hi = valid ? position : -1;
-            const int limit_lo = first_visible_key(position, window);
+            const int limit_lo = first_visible_key(position, item.window);
+            float slope = 0.f;
+            if (SHAPED && shape.slopes != nullptr)
+                slope = shape.slopes[item.kv_head * group + row % group] * 1.4426950408889634f;
             // keys that every row of the block sees: from the last row's lower limit to the
             // first row's position; a block with rows beyond the portion's end always masks
             const bool whole = item.tokens_here == tile_tokens;
-            const int open_lo = first_visible_key(last_position, window);
+            const int open_lo = first_visible_key(last_position, item.window);
             // m: the maximum that the exponentials are taken against. It follows the running
             // maximum only when that has moved by more than LAZY (in powers of two), so that the
             // output so far, which the product warp accumulates in tensor memory over the item's
@@ -576,6 +635,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q,
                 fence_after_sync();
                 float v[MY_KEYS];
                 tmem_load<MY_KEYS>(tmem_base + lanes + (t & 1) * KEYS + part * MY_KEYS, v);
+                if (SHAPED) shape_tile<MY_KEYS>(v, shape, slope, (float)(position - key0));
                 const bool open = whole && tile_key >= open_lo &&
                                   tile_key + KEYS - 1 <= item.first_position;
                 if (!open) {
@@ -596,7 +656,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q,
                     for (int other = 0; other < PARTS; ++other)
                         top = fmaxf(top, maxima[((t & 1) * PARTS + other) * ROWS + row]);
                 }
-                const float running = fmaxf(m, top * scale_log2);
+                const float running = fmaxf(m, SHAPED ? top : top * scale_log2);
                 // both threads of a row see the same maxima and take the same decision
                 const bool follow = running > m + LAZY || (m == -INFINITY && running > m);
                 const float moved = !follow ? 1.f : m == -INFINITY ? 0.f : fast_exp2(m - running);
@@ -626,8 +686,9 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q,
 #pragma unroll
                     for (int i = 0; i < 8; i += 2) {
                         float lo, hi;
-                        unpair(fma_pair(pair_of(v[piece * 8 + i], v[piece * 8 + i + 1]), scale_pair,
-                                        shift_pair), lo, hi);
+                        const unsigned long long scores = pair_of(v[piece * 8 + i], v[piece * 8 + i + 1]);
+                        unpair(SHAPED ? add_pair(scores, shift_pair)
+                                      : fma_pair(scores, scale_pair, shift_pair), lo, hi);
                         p[i] = fast_exp2(lo);                     // exp2(-inf) = 0
                         p[i + 1] = fast_exp2(hi);
                         partial[(i >> 1) & 1] = add_pair(partial[(i >> 1) & 1], pair_of(p[i], p[i + 1]));
@@ -785,7 +846,8 @@ static int prefill_tcgen05(const void* q, const void* kv, const int* block_table
                                                 void* out, int tokens, int requests, int heads,
                                                 int kv_heads, int head_dim, float scale, int window,
                                                 int splits, float* partial, const float* sinks,
-                                                int* error_flag, cudaStream_t stream, int keep_first) {
+                                                int* error_flag, cudaStream_t stream, int keep_first,
+                                                bool shaped = false, ScoreShape shape = ScoreShape()) {
     if (tokens == 0) return 0;
     MLXONE_REQUIRE(keep_first >= 0 && (keep_first == 0 || window > 0),
                    "attention_prefill_tcgen05: first positions are kept behind a window only");
@@ -854,9 +916,12 @@ static int prefill_tcgen05(const void* q, const void* kv, const int* block_table
     // item and walks its key tiles one after the other, so two threads share a row's softmax
     const bool shared_rows = !small_tiles && all_items < g_sm_count;
     const int threads = ((shared_rows ? 2 : 1) * 4 + 2) * 32;
-    auto kernel = small_tiles ? attention_tcgen05_kernel<64, 1>
-                              : shared_rows ? attention_tcgen05_kernel<128, 2>
-                                            : attention_tcgen05_kernel<128, 1>;
+    auto kernel = shaped ? (small_tiles ? attention_tcgen05_kernel<64, 1, true>
+                                        : shared_rows ? attention_tcgen05_kernel<128, 2, true>
+                                                      : attention_tcgen05_kernel<128, 1, true>)
+                         : (small_tiles ? attention_tcgen05_kernel<64, 1, false>
+                                        : shared_rows ? attention_tcgen05_kernel<128, 2, false>
+                                                      : attention_tcgen05_kernel<128, 1, false>);
     const cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, shared);
     if (err != cudaSuccess) {
         mlxone_set_error("attention_prefill_tcgen05: %s", cudaGetErrorString(err));
@@ -865,7 +930,7 @@ static int prefill_tcgen05(const void* q, const void* kv, const int* block_table
     kernel<<<dim3((unsigned)blocks), threads, shared, stream>>>(
         map_q, map_kv, value_rows, block_table, table_width, page_size, box_keys, request_start,
         history, static_cast<bf16*>(out), requests, heads, kv_heads, scale * 1.4426950408889634f,
-        window, token_tiles, splits, partial, sinks, error_flag, keep_first);
+        window, token_tiles, splits, partial, sinks, error_flag, keep_first, shape);
     MLXONE_LAUNCH_CHECK("attention_prefill_tcgen05");
     return 0;
 }
@@ -895,4 +960,20 @@ MLXONE_API int mlxone_attention_prefill_tcgen05_keep(const void* q, const void* 
     return prefill_tcgen05(q, kv, block_table, table_width, page_size, pages, request_start, history,
                            out, tokens, requests, heads, kv_heads, head_dim, scale, window, splits,
                            partial, sinks, error_flag, stream, keep_first);
+}
+
+// ... with scores s that become cap tanh(s / cap) (cap 0: none) and then lose slopes[head] (float32
+// [heads] or null) times the distance between query and key
+MLXONE_API int mlxone_attention_prefill_tcgen05_shaped(const void* q, const void* kv,
+                                                       const int* block_table, int table_width,
+                                                       int page_size, int pages,
+                                                       const int* request_start, const int* history,
+                                                       void* out, int tokens, int requests, int heads,
+                                                       int kv_heads, int head_dim, float scale,
+                                                       float cap, const float* slopes, int splits,
+                                                       float* partial, int* error_flag,
+                                                       cudaStream_t stream) {
+    return prefill_tcgen05(q, kv, block_table, table_width, page_size, pages, request_start, history,
+                           out, tokens, requests, heads, kv_heads, head_dim, scale, 0, splits, partial,
+                           nullptr, error_flag, stream, 0, true, make_score_shape(scale, cap, slopes));
 }

@@ -72,6 +72,14 @@ __device__ __forceinline__ float mlxone_activate(float z, int kind, float a = 0.
     }
 }
 
+// The hidden value of a clamped gated feed-forward: the gate cut at `limit` from above, the other
+// branch on both sides and shifted by one.
+__device__ __forceinline__ float mlxone_clamped(float gate, float up, float limit) {
+    const float g = fminf(gate, limit);
+    const float u = fminf(fmaxf(up, -limit), limit);
+    return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
+}
+
 // The first key that a query at `position` reads; the last one is its own. span > 0: a sliding
 // window of that many keys. span < 0: chunks of -span positions counted from 0, a query reads
 // the keys of its own chunk. 0: every earlier key. The result never falls as the position grows.

@@ -65,6 +65,9 @@ struct ConvUpdate {
     int gate = MLXONE_ACT_SILU;
     // (and for ACTIVATE: the two numbers of an activation that has some, as xielu)
     float act_a = 0.f, act_b = 0.f;
+    // (and for the gated epilogue with a positive act_a: the limits of the clamped form, act_a for
+    // columns below `boundary`, act_b behind it)
+    int boundary = 0;
 };
 
 __device__ __forceinline__ uint32_t shared_address(const void* p) {
@@ -616,10 +619,15 @@ skinny_gemm_kernel(const bf16* a, int lda, const bf16* __restrict__ w,
                 }
             } else if (EPILOGUE == SWIGLU) {
                 if (bias != nullptr) up += bias[up_offset + column];
-                const float gate = conv.gate == MLXONE_ACT_SILU ? value / (1.f + expf(-value))
-                                                                : mlxone_activate(value, conv.gate);
-                reinterpret_cast<bf16*>(out)[(size_t)token * ldo + column] =
-                    __float2bfloat16_rn(gate * up);
+                float hidden;
+                if (conv.act_a > 0.f) {
+                    hidden = mlxone_clamped(value, up, column < conv.boundary ? conv.act_a : conv.act_b);
+                } else {
+                    const float gate = conv.gate == MLXONE_ACT_SILU ? value / (1.f + expf(-value))
+                                                                    : mlxone_activate(value, conv.gate);
+                    hidden = gate * up;
+                }
+                reinterpret_cast<bf16*>(out)[(size_t)token * ldo + column] = __float2bfloat16_rn(hidden);
             } else if (EPILOGUE == STORE_BF16) {
                 reinterpret_cast<bf16*>(out)[(size_t)token * ldo + column] =
                     __float2bfloat16_rn(value);
@@ -774,6 +782,33 @@ MLXONE_API int mlxone_gemm_skinny_shaped(const void* a, int lda, const void* w, 
     shaped.act_b = act_b;
     const cudaError_t err = launch_for_rows<ACTIVATE>(a, lda, w, bias, out, ldo, m, n, k, activation,
                                                       stream, NormInput(), shaped);
+    if (err != cudaSuccess) {
+        mlxone_set_error("gemm_skinny: launch failed: %s", cudaGetErrorString(err));
+        return 2;
+    }
+    MLXONE_LAUNCH_CHECK("gemm_skinny");
+    return 0;
+}
+
+// As the gated epilogue of mlxone_gemm_skinny (w = [gate rows; up rows], n = 2 * width) with the
+// clamped form: limit `limit` for output columns below `boundary`, `second` behind it.
+MLXONE_API int mlxone_gemm_skinny_clamped(const void* a, int lda, const void* w, void* out, int ldo,
+                                          int m, int n, int k, float limit, float second,
+                                          int boundary, cudaStream_t stream) {
+    if (m == 0 || n == 0) return 0;
+    MLXONE_REQUIRE(m > 0 && m <= 32, "gemm_skinny: %d rows, at most 32", m);
+    MLXONE_REQUIRE(n > 0 && n % 2 == 0 && k > 0 && k % 8 == 0 && lda % 8 == 0,
+                   "gemm_skinny: K (%d) and the row stride of a (%d) must be multiples of 8", k, lda);
+    MLXONE_REQUIRE((reinterpret_cast<uintptr_t>(a) & 15) == 0 &&
+                       (reinterpret_cast<uintptr_t>(w) & 15) == 0,
+                   "gemm_skinny: operands must be 16-byte aligned");
+    MLXONE_REQUIRE(limit > 0.f && second > 0.f, "gemm_skinny: limits are positive");
+    ConvUpdate clamped;
+    clamped.act_a = limit;
+    clamped.act_b = second;
+    clamped.boundary = boundary;
+    const cudaError_t err = launch_for_rows<SWIGLU>(a, lda, w, nullptr, out, ldo, m, n, k, n / 2, stream,
+                                                    NormInput(), clamped);
     if (err != cudaSuccess) {
         mlxone_set_error("gemm_skinny: launch failed: %s", cudaGetErrorString(err));
         return 2;

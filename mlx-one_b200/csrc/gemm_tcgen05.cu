@@ -151,12 +151,13 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a,
                     const __grid_constant__ CUtensorMap map_w, const float* __restrict__ bias,
                     void* out, int ldo, int m, int n, int k, int up_offset, int tiles_m,
                     int total_tiles, int* __restrict__ error_flag,
-                    const int2* __restrict__ groups, int out_limit) {
+                    const int2* __restrict__ groups, int out_limit, float clamp) {
     // `groups` (null: one product): per tile of 128 rows of `a`, where its rows' weights lie in
     // `w` (x: first row, or -1 for a tile without rows, which is left out; y: first column).
     // Rows of `a` sorted by expert, each expert's rows padded to whole tiles, and the experts'
     // matrices stacked in `w`: a product per expert in one launch. `out_limit` is the number of
-    // output columns (the width of one expert's result).
+    // output columns (the width of one expert's result). `clamp` (SWIGLU): positive: the limit of the
+    // clamped gated form (mlxone_clamped) instead of silu(gate) * up.
     constexpr int A_BYTES = BM * BK * 2, W_BYTES = BN * BK * 2;
     constexpr int OUT_COLUMNS = EPILOGUE == SWIGLU ? BN / 2 : BN;
     extern __shared__ unsigned char shared_raw[];
@@ -286,8 +287,14 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a,
                             gate += bias[tile_n + c0 + i];
                             other += bias[up_offset + tile_n + c0 + i];
                         }
+                        float steep = 1.f;
+                        if (clamp > 0.f) {
+                            gate = fminf(gate, clamp);
+                            other = fminf(fmaxf(other, -clamp), clamp) + 1.f;
+                            steep = 1.702f;
+                        }
                         // the result is rounded to bfloat16; the fast exponential is exact enough
-                        value[i] = __fdividef(gate, 1.f + __expf(-gate)) * other;
+                        value[i] = __fdividef(gate, 1.f + __expf(-steep * gate)) * other;
                     }
                 } else if (bias != nullptr) {
 #pragma unroll
@@ -442,7 +449,7 @@ struct Grouping {
 template <int BN, int EPILOGUE, int STAGES>
 int launch(const void* a, int lda, const void* w, const float* bias, void* out, int ldo, int m,
            int n, int k, int up_offset, int* error_flag, cudaStream_t stream,
-           Grouping grouping = Grouping()) {
+           Grouping grouping = Grouping(), float clamp = 0.f) {
     CUtensorMap map_a, map_w;
     const int w_box = EPILOGUE == SWIGLU ? BN / 2 : BN;
     const bool grouped = grouping.groups != nullptr;
@@ -474,7 +481,7 @@ int launch(const void* a, int lda, const void* w, const float* bias, void* out, 
     }
     kernel<<<grid, THREADS, shared, stream>>>(map_a, map_w, bias, out, ldo, m, n, k, up_offset,
                                               tiles_m, total_tiles, error_flag, grouping.groups,
-                                              columns);
+                                              columns, clamp);
     return 0;
 }
 
@@ -525,18 +532,36 @@ MLXONE_API int mlxone_gemm_tcgen05(const void* a, int lda, const void* w, const 
     return 0;
 }
 
+// The gated product with the clamped form: out bf16 [m, n / 2] from w = [gate rows; up rows].
+MLXONE_API int mlxone_gemm_tcgen05_clamped(const void* a, int lda, const void* w, void* out, int ldo,
+                                           int m, int n, int k, float clamp, int* error_flag,
+                                           cudaStream_t stream) {
+    if (m == 0 || n == 0) return 0;
+    MLXONE_REQUIRE(find_encoder(), "gemm_tcgen05: the driver has no cuTensorMapEncodeTiled");
+    MLXONE_REQUIRE(m > 0 && n > 0 && n % 2 == 0 && k > 0 && k % 8 == 0 && lda % 8 == 0 && clamp > 0.f,
+                   "gemm_tcgen05: K (%d) and the row stride of a (%d) must be multiples of 8", k, lda);
+    MLXONE_REQUIRE((reinterpret_cast<uintptr_t>(a) & 15) == 0 &&
+                       (reinterpret_cast<uintptr_t>(w) & 15) == 0,
+                   "gemm_tcgen05: operands must be 16-byte aligned");
+    const int code = launch<256, SWIGLU, WIDE_STAGES>(a, lda, w, nullptr, out, ldo, m, n, k, n / 2,
+                                                      error_flag, stream, Grouping(), clamp);
+    if (code != 0) return code;
+    MLXONE_LAUNCH_CHECK("gemm_tcgen05");
+    return 0;
+}
+
 // One product per group of rows in one launch. a: [m, k] (row stride lda), its rows sorted by
 // group and every group's rows padded to whole tiles of 128; groups: int32 [m / 128, 2], per
 // tile the first row and the first column of its group's matrix inside the stacked w
 // [w_rows, w_columns] (row stride w_ld), or -1 for a tile without rows. epilogue 0: out bf16
 // [m, n] = a_tile w_group^T with w_group [n, k]; epilogue 1 (SwiGLU): w_group's n gate rows start
 // at the tile's row, its up rows `up_offset` rows further, out bf16 [m, n]; epilogue 4: as 0, the
-// square of max(z, 0) of every value z.
-MLXONE_API int mlxone_gemm_tcgen05_grouped(const void* a, int lda, const void* w, long long w_rows,
-                                           long long w_columns, long long w_ld, void* out, int ldo,
-                                           int m, int n, int k, int up_offset, int epilogue,
-                                           const int* groups, int* error_flag,
-                                           cudaStream_t stream) {
+// square of max(z, 0) of every value z. `clamp` (epilogue 1): positive: the limit of the clamped form.
+static int grouped_product(const void* a, int lda, const void* w, long long w_rows,
+                           long long w_columns, long long w_ld, void* out, int ldo,
+                           int m, int n, int k, int up_offset, int epilogue,
+                           const int* groups, int* error_flag,
+                           cudaStream_t stream, float clamp) {
     if (m == 0 || n == 0) return 0;
     MLXONE_REQUIRE(find_encoder(), "gemm_tcgen05: the driver has no cuTensorMapEncodeTiled");
     MLXONE_REQUIRE(m > 0 && m % BM == 0 && n > 0 && k > 0 && k % 8 == 0 && lda % 8 == 0 &&
@@ -555,7 +580,7 @@ MLXONE_API int mlxone_gemm_tcgen05_grouped(const void* a, int lda, const void* w
     int code;
     if (epilogue == SWIGLU)
         code = launch<256, SWIGLU, WIDE_STAGES>(a, lda, w, nullptr, out, ldo, m, n, k, up_offset,
-                                                error_flag, stream, grouping);
+                                                error_flag, stream, grouping, clamp);
     else if (epilogue == STORE_RELU2)
         code = n > 128 ? launch<256, STORE_RELU2, WIDE_STAGES>(a, lda, w, nullptr, out, ldo, m, n, k, 0,
                                                                error_flag, stream, grouping)
@@ -570,4 +595,24 @@ MLXONE_API int mlxone_gemm_tcgen05_grouped(const void* a, int lda, const void* w
     if (code != 0) return code;
     MLXONE_LAUNCH_CHECK("gemm_tcgen05_grouped");
     return 0;
+}
+
+MLXONE_API int mlxone_gemm_tcgen05_grouped(const void* a, int lda, const void* w, long long w_rows,
+                                           long long w_columns, long long w_ld, void* out, int ldo,
+                                           int m, int n, int k, int up_offset, int epilogue,
+                                           const int* groups, int* error_flag,
+                                           cudaStream_t stream) {
+    return grouped_product(a, lda, w, w_rows, w_columns, w_ld, out, ldo, m, n, k, up_offset, epilogue,
+                           groups, error_flag, stream, 0.f);
+}
+
+MLXONE_API int mlxone_gemm_tcgen05_grouped_clamped(const void* a, int lda, const void* w,
+                                                   long long w_rows, long long w_columns,
+                                                   long long w_ld, void* out, int ldo, int m, int n,
+                                                   int k, int up_offset, float clamp,
+                                                   const int* groups, int* error_flag,
+                                                   cudaStream_t stream) {
+    MLXONE_REQUIRE(clamp > 0.f, "gemm_tcgen05_grouped: the limit is positive");
+    return grouped_product(a, lda, w, w_rows, w_columns, w_ld, out, ldo, m, n, k, up_offset, SWIGLU,
+                           groups, error_flag, stream, clamp);
 }

@@ -210,7 +210,18 @@ qk_prep_wide_kernel(const __nv_bfloat16* __restrict__ qkv, const float* __restri
 // value_dim], rows ``ld`` values apart (a slice of a wider product). The rotation multiplies
 // cosine and sine by ``amplitude``. norm_mode 0: no norm;
 // 1: RMSNorm with the given weights before the rotation; 2: division by the root mean square
-// (over head_dim, eps inside the root) after the rotation, no weight. One warp per (token, head).
+// (over head_dim, eps inside the root) after the rotation, no weight; 3: RMSNorm over all query heads'
+// values at once, and over all key heads', with weights of those sizes, before the rotation (every
+// block of a token works the two sums out). One warp per (token, head). `extra`: a factor on the
+// queries that grows with the position, and values mixed with another layer's.
+struct PrepExtra {
+    float coef = 0.f;               // queries times 1 + coef ln(floor((p + 1) / every) + 1); 0: as they are
+    double every = 1.0;
+    const void* first = nullptr;    // v <- (1 - mix) v + mix first[t, :]; rows `first_ld` values apart
+    int first_ld = 0;
+    float mix = 0.f;
+};
+
 template <typename T>
 __global__ void __launch_bounds__(WARPS * 32)
 qk_prep_general_kernel(const T* __restrict__ qkv, const float* __restrict__ q_weight,
@@ -221,7 +232,7 @@ qk_prep_general_kernel(const T* __restrict__ qkv, const float* __restrict__ q_we
                        T* __restrict__ kv, const int* __restrict__ block_table, int table_width,
                        int page_size, long long kv_half, int tokens, int heads, int kv_heads,
                        int head_dim, int value_dim, int row_dim, int write_kv, int ld,
-                       int* __restrict__ error_flag) {
+                       int* __restrict__ error_flag, PrepExtra extra) {
     // Blocks (token, part): the angles' cosines and sines are worked out once for the block's
     // heads (rotary_dim / 2 of each, scaled), then its warps take their share of the token's
     // heads in turn: a warp has one head in a step of few tokens, two in a large one.
@@ -243,6 +254,24 @@ qk_prep_general_kernel(const T* __restrict__ qkv, const float* __restrict__ q_we
             cosines[j] = cosine * amplitude;
         }
     }
+    float whole[2] = {1.f, 1.f};               // 1 / rms of all queries, of all keys
+    if (norm_mode == 3) {
+        __shared__ float scratch[33];
+        const T* row = qkv + (size_t)t * ld;
+        for (int part = 0; part < 2; ++part) {
+            const int first = part == 0 ? 0 : heads * head_dim;
+            const int count = (part == 0 ? heads : kv_heads) * head_dim;
+            float sum = 0.f;
+            for (int e = threadIdx.x; e < count; e += blockDim.x) {
+                const float v = to_float<T>(row[first + e]);
+                sum = fmaf(v, v, sum);
+            }
+            whole[part] = rsqrtf(block_sum(sum, scratch) / (float)count + eps);
+        }
+    }
+    float warmth = 1.f;
+    if (extra.coef != 0.f)
+        warmth = fmaf(extra.coef, logf((float)(floor((double)(position + 1) / extra.every) + 1.0)), 1.f);
     __syncthreads();
     // where this token's keys and values go
     T* page_base = nullptr;
@@ -279,7 +308,13 @@ qk_prep_general_kernel(const T* __restrict__ qkv, const float* __restrict__ q_we
                 const float inv = rsqrtf(sum / (float)head_dim + eps);
                 for (int e = lane; e < head_dim; e += 32)
                     values[e] = values[e] * inv * (weight ? weight[e] : 1.f);
+            } else if (norm_mode == 3) {
+                const int first = (is_q ? slot : slot - heads) * head_dim;
+                const float inv = is_q ? whole[0] : whole[1];
+                for (int e = lane; e < head_dim; e += 32) values[e] = values[e] * inv * weight[first + e];
             }
+            if (is_q && warmth != 1.f)          // (a factor on the row: before or after the rotation alike)
+                for (int e = lane; e < head_dim; e += 32) values[e] *= warmth;
             __syncwarp();
             float squares = 0.f;
             if (inv_freq != nullptr) {
@@ -298,6 +333,11 @@ qk_prep_general_kernel(const T* __restrict__ qkv, const float* __restrict__ q_we
                 const float inv = 1.f / sqrtf(squares / (float)head_dim + eps);
                 for (int e = lane; e < head_dim; e += 32) values[e] *= inv;
             }
+        } else if (extra.first != nullptr) {
+            const T* first = static_cast<const T*>(extra.first) + (size_t)t * extra.first_ld +
+                             (size_t)(slot - heads - kv_heads) * value_dim;
+            for (int e = lane; e < value_dim; e += 32)
+                values[e] = fmaf(extra.mix, to_float<T>(first[e]), (1.f - extra.mix) * values[e]);
         }
         __syncwarp();
         T* dst;
@@ -374,14 +414,14 @@ MLXONE_API int mlxone_qk_prep(const void* qkv, const float* q_weight, const floa
     return 0;
 }
 
-MLXONE_API int mlxone_qk_prep_general(const void* qkv, const float* q_weight, const float* k_weight,
-                                      float eps, const float* inv_freq, int rotary_dim,
-                                      float amplitude, int norm_mode, const int* positions,
-                                      const int* token_request, void* q_out, void* kv,
-                                      const int* block_table, int table_width, int page_size,
-                                      int pages, int tokens, int heads, int kv_heads, int head_dim,
-                                      int value_dim, int row_dim, int write_kv, int ld, int dtype,
-                                      int* error_flag, cudaStream_t stream) {
+static int qk_prep_general(const void* qkv, const float* q_weight, const float* k_weight,
+                           float eps, const float* inv_freq, int rotary_dim,
+                           float amplitude, int norm_mode, const int* positions,
+                           const int* token_request, void* q_out, void* kv,
+                           const int* block_table, int table_width, int page_size,
+                           int pages, int tokens, int heads, int kv_heads, int head_dim,
+                           int value_dim, int row_dim, int write_kv, int ld, int dtype,
+                           int* error_flag, PrepExtra extra, cudaStream_t stream) {
     if (tokens == 0) return 0;
     MLXONE_REQUIRE(tokens > 0 && heads > 0 && kv_heads > 0, "qk_prep: bad sizes");
     MLXONE_REQUIRE(head_dim >= 1 && value_dim >= 1 && row_dim >= head_dim && row_dim >= value_dim &&
@@ -392,7 +432,11 @@ MLXONE_API int mlxone_qk_prep_general(const void* qkv, const float* q_weight, co
                        (rotary_dim > 0 && rotary_dim % 2 == 0 && rotary_dim <= head_dim),
                    "qk_prep: rotary size %d must be even and at most the head size %d", rotary_dim,
                    head_dim);
-    MLXONE_REQUIRE(norm_mode >= 0 && norm_mode <= 2, "qk_prep: unknown norm mode %d", norm_mode);
+    MLXONE_REQUIRE(norm_mode >= 0 && norm_mode <= 3, "qk_prep: unknown norm mode %d", norm_mode);
+    MLXONE_REQUIRE(norm_mode != 3 || (q_weight != nullptr && k_weight != nullptr),
+                   "qk_prep: a norm over whole rows has weights");
+    MLXONE_REQUIRE(extra.every > 0.0 && (extra.first == nullptr || extra.first_ld >= kv_heads * value_dim),
+                   "qk_prep: bad temperature or value rows");
     MLXONE_REQUIRE(ld >= (heads + kv_heads) * head_dim + kv_heads * value_dim,
                    "qk_prep: rows %d apart are shorter than their heads", ld);
     MLXONE_REQUIRE(page_size > 0 && pages > 0 && table_width > 0, "qk_prep: bad page geometry");
@@ -407,15 +451,50 @@ MLXONE_API int mlxone_qk_prep_general(const void* qkv, const float* q_weight, co
                       (const T*)qkv, q_weight, k_weight, eps, inv_freq, rotary_dim, amplitude,
                       norm_mode, positions, token_request, (T*)q_out, (T*)kv, block_table,
                       table_width, page_size, kv_half, tokens, heads, kv_heads, head_dim, value_dim,
-                      row_dim, write_kv, ld, error_flag);
+                      row_dim, write_kv, ld, error_flag, extra);
     } else {
         using T = float;
         launch_kernel(qk_prep_general_kernel<T>, blocks, dim3(WARPS * 32), shared, stream, true,
                       (const T*)qkv, q_weight, k_weight, eps, inv_freq, rotary_dim, amplitude,
                       norm_mode, positions, token_request, (T*)q_out, (T*)kv, block_table,
                       table_width, page_size, kv_half, tokens, heads, kv_heads, head_dim, value_dim,
-                      row_dim, write_kv, ld, error_flag);
+                      row_dim, write_kv, ld, error_flag, extra);
     }
     MLXONE_LAUNCH_CHECK("qk_prep_general");
     return 0;
+}
+
+MLXONE_API int mlxone_qk_prep_general(const void* qkv, const float* q_weight, const float* k_weight,
+                                      float eps, const float* inv_freq, int rotary_dim,
+                                      float amplitude, int norm_mode, const int* positions,
+                                      const int* token_request, void* q_out, void* kv,
+                                      const int* block_table, int table_width, int page_size,
+                                      int pages, int tokens, int heads, int kv_heads, int head_dim,
+                                      int value_dim, int row_dim, int write_kv, int ld, int dtype,
+                                      int* error_flag, cudaStream_t stream) {
+    return qk_prep_general(qkv, q_weight, k_weight, eps, inv_freq, rotary_dim, amplitude, norm_mode,
+                           positions, token_request, q_out, kv, block_table, table_width, page_size,
+                           pages, tokens, heads, kv_heads, head_dim, value_dim, row_dim, write_kv, ld,
+                           dtype, error_flag, PrepExtra(), stream);
+}
+
+// ... with queries times 1 + coef ln(floor((p + 1) / every) + 1) (coef 0: as they are), and values
+// (1 - mix) v + mix first[t, :] (first: rows of kv_heads * value_dim values, `first_ld` apart; null: as
+// they are).
+MLXONE_API int mlxone_qk_prep_mixed(const void* qkv, const float* q_weight, const float* k_weight,
+                                    float eps, const float* inv_freq, int rotary_dim,
+                                    float amplitude, int norm_mode, float coef, double every,
+                                    const void* first, int first_ld, float mix, const int* positions,
+                                    const int* token_request, void* q_out, void* kv,
+                                    const int* block_table, int table_width, int page_size, int pages,
+                                    int tokens, int heads, int kv_heads, int head_dim, int value_dim,
+                                    int row_dim, int write_kv, int ld, int dtype, int* error_flag,
+                                    cudaStream_t stream) {
+    PrepExtra extra;
+    extra.coef = coef; extra.every = every;
+    extra.first = first; extra.first_ld = first_ld; extra.mix = mix;
+    return qk_prep_general(qkv, q_weight, k_weight, eps, inv_freq, rotary_dim, amplitude, norm_mode,
+                           positions, token_request, q_out, kv, block_table, table_width, page_size,
+                           pages, tokens, heads, kv_heads, head_dim, value_dim, row_dim, write_kv, ld,
+                           dtype, error_flag, extra, stream);
 }

@@ -141,6 +141,63 @@ __global__ void gated_activation_kernel(const T* __restrict__ gate_up, T* __rest
     out[i] = from_float<T>(mlxone_activate(gate, kind) * up);
 }
 
+// out = mlxone_clamped(gate, up) with one limit for columns below `boundary` and another behind it.
+// VEC neighbouring values a thread (8: bfloat16 with 16-byte rows).
+template <typename T, int VEC>
+__global__ void gated_clamped_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int width,
+                                     long long total, float limit, float second, int boundary) {
+    griddep_launch();
+    griddep_wait();
+    gate_up = settled(gate_up);
+    const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+    if (i >= total) return;
+    const long long t = i / width;
+    const int f = (int)(i - t * width);
+    const T* row = gate_up + t * 2 * width + f;
+    __align__(16) T g[VEC];
+    __align__(16) T u[VEC];
+    __align__(16) T result[VEC];
+    if (VEC == 8) {
+        *reinterpret_cast<uint4*>(g) = *reinterpret_cast<const uint4*>(row);
+        *reinterpret_cast<uint4*>(u) = *reinterpret_cast<const uint4*>(row + width);
+    } else {
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) { g[j] = row[j]; u[j] = row[width + j]; }
+    }
+#pragma unroll
+    for (int j = 0; j < VEC; ++j)
+        result[j] = from_float<T>(mlxone_clamped(to_float<T>(g[j]), to_float<T>(u[j]),
+                                                 f + j < boundary ? limit : second));
+    if (VEC == 8) {
+        *reinterpret_cast<uint4*>(out + i) = *reinterpret_cast<const uint4*>(result);
+    } else {
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) out[i + j] = result[j];
+    }
+}
+
+MLXONE_API int mlxone_gated_clamped(const void* gate_up, void* out, int rows, int width, float limit,
+                                    float second, int boundary, int dtype, cudaStream_t stream) {
+    if (rows == 0) return 0;
+    MLXONE_REQUIRE(rows > 0 && width > 0, "gated_clamped: bad sizes");
+    const long long total = (long long)rows * width;
+    const int blocks = ceil_div_host(total, 256);
+    if (dtype == MLXONE_BF16 && width % 8 == 0 && (reinterpret_cast<uintptr_t>(gate_up) & 15) == 0 &&
+        (reinterpret_cast<uintptr_t>(out) & 15) == 0)
+        launch_kernel(gated_clamped_kernel<__nv_bfloat16, 8>, dim3(ceil_div_host(total / 8, 256)),
+                      dim3(256), 0, stream, true, (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out,
+                      width, total, limit, second, boundary);
+    else if (dtype == MLXONE_BF16)
+        launch_kernel(gated_clamped_kernel<__nv_bfloat16, 1>, dim3(blocks), dim3(256), 0, stream, true,
+                      (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, width, total, limit, second,
+                      boundary);
+    else
+        launch_kernel(gated_clamped_kernel<float, 1>, dim3(blocks), dim3(256), 0, stream, true,
+                      (const float*)gate_up, (float*)out, width, total, limit, second, boundary);
+    MLXONE_LAUNCH_CHECK("gated_clamped");
+    return 0;
+}
+
 MLXONE_API int mlxone_gated_activation(const void* gate_up, void* out, int rows, int width, int kind,
                                        int dtype, cudaStream_t stream) {
     if (rows == 0) return 0;

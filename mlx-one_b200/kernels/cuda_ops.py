@@ -17,7 +17,7 @@ from typing import Any
 
 import torch
 
-from ..parts.base import NormedInput
+from ..parts.base import NormedInput, NormedUpdate
 from .build import KernelBuildError, library_path
 
 _F32, _BF16 = 0, 1
@@ -60,6 +60,7 @@ class CudaOps:
         self.lib.mlxone_channel_delta_scratch.restype = ctypes.c_longlong
         self.lib.mlxone_lightning_scratch.restype = ctypes.c_longlong
         self.lib.mlxone_state_space_scratch.restype = ctypes.c_longlong
+        self.lib.mlxone_gated_recurrence_scratch.restype = ctypes.c_longlong
         if self.lib.mlxone_abi_version() != 1:
             raise KernelBuildError("the CUDA extension is of another version; rebuild it")
         self.error_flag = torch.zeros(1, dtype=torch.int32, device=self.device)
@@ -116,6 +117,8 @@ class CudaOps:
         self.skinny_fused_max_rows = 16
         # latent attention of few tokens: the key up-projection with the queries' rotation in one kernel
         self.fused_latent = True
+        # the gated recurrence of few single tokens: the gates' product in the recurrence's kernel
+        self.fused_recurrence = True
         self._sample_scratch: torch.Tensor | None = None
         self._device_index = self.device.index if self.device.index is not None else torch.cuda.current_device()
 
@@ -200,6 +203,37 @@ class CudaOps:
         self._call("mlxone_add_rmsnorm", _c_void_p(_ptr(residual)), _c_void_p(_ptr(delta)),
                    _c_void_p(_ptr(weight)), _c_void_p(_ptr(out)), _c_int(rows), _c_int(hidden),
                    _c_float(eps), _c_int(_dtype_code(dtype)), _c_float(delta_scale))
+        return out
+
+    def add_norm(self, residual, delta, weight, bias, eps, dtype, delta_scale=1.0):
+        """What ``add_rmsnorm`` does, for norms with a bias (layer norms; ``bias`` None: RMSNorm) and
+        for a ``delta`` that is a ``NormedUpdate``: an output that is normed itself before it is
+        added. One kernel."""
+        self._need(residual, torch.float32, "residual")
+        update = delta if isinstance(delta, NormedUpdate) else None
+        output = delta if update is None else update.output
+        rows, hidden = residual.shape
+        vectors = [(weight, "norm weight"), (bias, "norm bias")]
+        if update is not None:
+            vectors += [(update.weight, "update weight"), (update.bias, "update bias")]
+        for vector, what in vectors:
+            if vector is not None:
+                self._need(vector, torch.float32, what)
+                if vector.numel() != hidden:
+                    raise KernelError(f"{what} has {vector.numel()} entries, rows have {hidden}")
+        if output is not None:
+            self._need(output, dtype, "delta")
+            if output.shape != residual.shape:
+                raise KernelError("delta and residual differ in shape")
+        out = torch.empty((rows, hidden), dtype=dtype, device=self.device)
+        post = (None, None, 0, 0.0)
+        if update is not None:
+            post = (update.weight, update.bias, 1 if update.bias is None else 2, update.eps)
+        self._call("mlxone_stream_norm", _c_void_p(_ptr(residual)), _c_void_p(_ptr(output)),
+                   _c_float(delta_scale), _c_void_p(_ptr(post[0])), _c_void_p(_ptr(post[1])),
+                   _c_int(post[2]), _c_float(post[3]), _c_void_p(_ptr(weight)), _c_void_p(_ptr(bias)),
+                   _c_int(1 if bias is None else 2), _c_float(eps), _c_void_p(_ptr(out)), _c_int(rows),
+                   _c_int(hidden), _c_int(_dtype_code(dtype)))
         return out
 
     def gather_rows(self, residual, delta, rows):
@@ -412,11 +446,14 @@ class CudaOps:
             return None
         return self.linear(a, w, bias)
 
-    def linear_gated(self, a, gate_up, kind):
+    def linear_gated(self, a, gate_up, kind, limits=None):
         """act(a @ gate^T) * (a @ up^T) with gate_up = [gate rows; up rows], for the activations
         of ``ACTIVATIONS``: silu takes the fused kernels of ``linear_swiglu``; for the others the
         gate is the skinny product's epilogue for few rows (also with the norm of its input
-        applied while loading), else the product and one kernel for the gate."""
+        applied while loading), else the product and one kernel for the gate. ``clamped`` (see
+        ``_linear_clamped``) takes ``limits``."""
+        if kind == "clamped":
+            return self._linear_clamped(a, gate_up, *limits)
         if kind == "silu":
             return self.linear_swiglu(a, gate_up)
         if kind not in self.ACTIVATIONS:
@@ -437,6 +474,37 @@ class CudaOps:
         out = torch.empty((rows, twice // 2), dtype=both.dtype, device=self.device)
         self._call("mlxone_gated_activation", _c_void_p(_ptr(both)), _c_void_p(_ptr(out)),
                    _c_int(rows), _c_int(twice // 2), _c_int(self.ACTIVATIONS[kind]),
+                   _c_int(_dtype_code(both.dtype)))
+        return out
+
+    def _linear_clamped(self, a, gate_up, limit, second, boundary):
+        """g sigmoid(1.702 g) (u + 1) with g = min(a @ gate^T, limit) and u = a @ up^T cut to [-limit,
+        limit]; output columns from ``boundary`` on have the limit ``second``. The epilogue of the
+        skinny or (one limit for all columns) the tcgen05 product, else the product and one kernel."""
+        if isinstance(a, NormedInput):
+            a = a.materialize()
+        self._check_product(a, gate_up)
+        rows, width = a.shape[0], gate_up.shape[0] // 2
+        if self._skinny(a, gate_up, fused=True):
+            out = torch.empty((rows, width), dtype=a.dtype, device=self.device)
+            self._call("mlxone_gemm_skinny_clamped", _c_void_p(_ptr(a)), _c_int(a.stride(0)),
+                       _c_void_p(_ptr(gate_up)), _c_void_p(_ptr(out)), _c_int(width), _c_int(rows),
+                       _c_int(gate_up.shape[0]), _c_int(a.shape[1]), _c_float(limit), _c_float(second),
+                       _c_int(boundary))
+            return out
+        if boundary >= width or boundary <= 0 or limit == second:
+            if self._tcgen05(a, gate_up, self._SWIGLU):
+                out = torch.empty((rows, width), dtype=a.dtype, device=self.device)
+                self._call("mlxone_gemm_tcgen05_clamped", _c_void_p(_ptr(a)), _c_int(a.stride(0)),
+                           _c_void_p(_ptr(gate_up)), _c_void_p(_ptr(out)), _c_int(width), _c_int(rows),
+                           _c_int(gate_up.shape[0]), _c_int(a.shape[1]),
+                           _c_float(limit if boundary > 0 else second),
+                           _c_void_p(_ptr(self.error_flag)))
+                return out
+        both = self.linear(a, gate_up)
+        out = torch.empty((rows, width), dtype=both.dtype, device=self.device)
+        self._call("mlxone_gated_clamped", _c_void_p(_ptr(both)), _c_void_p(_ptr(out)), _c_int(rows),
+                   _c_int(width), _c_float(limit), _c_float(second), _c_int(boundary),
                    _c_int(_dtype_code(both.dtype)))
         return out
 
@@ -1028,16 +1096,18 @@ class CudaOps:
 
     def routed_experts_sorted(self, x, weights, gate_up, down, *, experts, width, top,
                               shared_gate_up=None, shared_down=None, shared_scale=None,
-                              activation=None):
+                              activation=None, limit=0.0, shared_limits=None):
         """The weighted sum of every token's chosen experts (+ the shared expert's output), with
         the tokens sorted by expert: gate_up [2 stack, hidden] holds the experts' gate rows, then
         (``stack`` rows further) their up rows; down [hidden, stack] their down matrices side by
-        side. ``activation`` (relu2): experts without a gate, gate_up [stack, hidden] holds their
-        up rows alone. weights [tokens, experts] float32, zero where an expert was not chosen."""
+        side. ``activation``: ``relu2``: experts without a gate, gate_up [stack, hidden] holds their
+        up rows alone; ``clamped``: the gated form of ``_linear_clamped`` with ``limit``, the shared
+        expert's with ``shared_limits``. weights [tokens, experts] float32, zero where an expert was not chosen."""
         tokens, hidden = x.shape
-        if activation not in (None, "relu2"):
+        if activation not in (None, "relu2", "clamped"):
             raise KernelError(f"no grouped product with the activation {activation!r}")
-        stack = gate_up.shape[0] if activation else gate_up.shape[0] // 2
+        ungated = activation == "relu2"
+        stack = gate_up.shape[0] if ungated else gate_up.shape[0] // 2
         tiles = -(-(tokens * top + experts * 127) // 128)
         rows = tiles * 128
         pair_row = torch.empty((tokens, experts), dtype=torch.int32, device=self.device)
@@ -1052,11 +1122,14 @@ class CudaOps:
                    _c_void_p(_ptr(pair_row)), _c_void_p(_ptr(sorted_x)), _c_int(tokens),
                    _c_int(hidden), _c_int(experts), _c_int(rows), _c_int(_dtype_code(x.dtype)))
         gated = torch.empty((rows, width), dtype=x.dtype, device=self.device)
-        self._call("mlxone_gemm_tcgen05_grouped", _c_void_p(_ptr(sorted_x)), _c_int(hidden),
+        clamped = activation == "clamped"
+        form = (_c_float(limit),) if clamped else \
+            (_c_int(self._GROUPED_RELU2 if ungated else self._SWIGLU),)
+        self._call("mlxone_gemm_tcgen05_grouped" + ("_clamped" if clamped else ""),
+                   _c_void_p(_ptr(sorted_x)), _c_int(hidden),
                    _c_void_p(_ptr(gate_up)), _c_ll(gate_up.shape[0]), _c_ll(hidden), _c_ll(hidden),
                    _c_void_p(_ptr(gated)), _c_int(width), _c_int(rows), _c_int(width),
-                   _c_int(hidden), _c_int(0 if activation else stack),
-                   _c_int(self._GROUPED_RELU2 if activation else self._SWIGLU),
+                   _c_int(hidden), _c_int(0 if ungated else stack), *form,
                    _c_void_p(_ptr(groups[0])), _c_void_p(_ptr(self.error_flag)))
         y = torch.empty((rows, hidden), dtype=x.dtype, device=self.device)
         self._call("mlxone_gemm_tcgen05_grouped", _c_void_p(_ptr(gated)), _c_int(width),
@@ -1066,7 +1139,8 @@ class CudaOps:
                    _c_void_p(_ptr(self.error_flag)))
         shared_out = None
         if shared_gate_up is not None:
-            shared_gated = self.linear_swiglu(x, shared_gate_up)
+            shared_gated = self._linear_clamped(x, shared_gate_up, *shared_limits) if clamped \
+                else self.linear_swiglu(x, shared_gate_up)
             if shared_scale is not None:
                 # (one number per token on the shared expert's output, applied ahead of its down
                 # product, which is linear)
@@ -1110,6 +1184,55 @@ class CudaOps:
                    _c_int(ctx.max_portion), _c_int(heads), _c_int(key_dim), _c_int(value_dim),
                    _c_int(1 if write else 0), _c_int(_dtype_code(projected.dtype)))
         self.launches += 1 if ctx.max_portion < 128 else 3
+        return out
+
+    def gated_recurrence(self, u, y, *, gates, gate_bias, rate, ctx, view, write):
+        """The gated linear recurrence per channel. u [tokens, width]; gates [blocks, 2 n, n] in u's
+        dtype with bias float32 [blocks, 2 n] (per part of n channels the rows of r, then those of
+        i); r, i = sigmoid of their 32-bit products with the parts of u; log a = ``rate`` r, S = a S
+        + sqrt(1 - a^2) i u over each request's tokens on its 32-bit state [width]. Returns S *
+        gelu_tanh(y) [tokens, width] (``y`` may be a slice of wider rows). Up to 16 single tokens one
+        kernel; else the gates' product, then one kernel, or for longer portions three."""
+        self._need(u, u.dtype, "u")
+        self._need_rows(y, u.dtype, "y")
+        self._need(gates, u.dtype, "gates")
+        for tensor, what in ((gate_bias, "gate bias"), (rate, "rate"), (view.state, "state")):
+            self._need(tensor, torch.float32, what)
+        tokens, width = u.shape
+        blocks, part = gates.shape[0], gates.shape[2]
+        if (gates.shape != (blocks, 2 * part, part) or blocks * part != width or y.shape != u.shape
+                or gate_bias.numel() != 2 * width or rate.numel() != width
+                or view.state[0].numel() != width):
+            raise KernelError("the recurrence's channels, gates and state do not match")
+        out = torch.empty((tokens, width), dtype=u.dtype, device=self.device)
+        sizes = (_c_int(width), _c_int(blocks), _c_int(1 if write else 0), _c_int(_dtype_code(u.dtype)))
+        if (self.fused_recurrence and ctx.max_portion == 1 and tokens == ctx.requests
+                and self.lib.mlxone_gated_recurrence_step_fits(_c_int(tokens), _c_int(part))):
+            self._call("mlxone_gated_recurrence_step", _c_void_p(_ptr(u)), _c_void_p(_ptr(y)),
+                       _c_int(y.stride(0)), _c_void_p(_ptr(gates)), _c_void_p(_ptr(gate_bias)),
+                       _c_void_p(_ptr(rate)), _c_void_p(_ptr(view.state)), _c_void_p(_ptr(view.slots)),
+                       _c_void_p(_ptr(out)), _c_int(tokens), *sizes)
+            return out
+        # the gates' products stay in 32-bit: [parts, tokens, 2 n], or token by token in 32-bit storage
+        parts = u.view(tokens, blocks, part)
+        if u.dtype == torch.float32:
+            z = self.linear_heads(parts, gates)
+            z_token, z_block = z.stride(0), z.stride(1)
+        else:
+            z = torch.bmm(parts.transpose(0, 1), gates.transpose(1, 2), out_dtype=torch.float32)
+            z_token, z_block = z.stride(1), z.stride(0)
+        scratch = None
+        size = self.lib.mlxone_gated_recurrence_scratch(tokens, ctx.requests, ctx.max_portion, width)
+        if size:
+            scratch = torch.empty(size, dtype=torch.float32, device=self.device)
+        self._call("mlxone_gated_recurrence", _c_void_p(_ptr(u)), _c_void_p(_ptr(y)),
+                   _c_int(y.stride(0)), _c_void_p(_ptr(z)), _c_ll(z_token), _c_ll(z_block),
+                   _c_void_p(_ptr(gate_bias)), _c_void_p(_ptr(rate)), _c_void_p(_ptr(view.state)),
+                   _c_void_p(_ptr(view.slots)), _c_void_p(_ptr(ctx.request_start)),
+                   _c_void_p(_ptr(scratch)), _c_void_p(_ptr(out)), _c_int(tokens),
+                   _c_int(ctx.requests), _c_int(ctx.max_portion), *sizes)
+        if scratch is not None:
+            self.launches += 2
         return out
 
     def normed_mean_add(self, residual, outputs, weights, eps):
@@ -1344,17 +1467,21 @@ class CudaOps:
 
     def qk_norm_rope_store(self, qkv, *, heads, kv_heads, head_dim, q_weight, k_weight, eps,
                            rotary, ctx, view, write, value_dim=None, amplitude=1.0,
-                           norm_after=False):
+                           norm_after=False, norm_rows=False, temperature=None, value_mix=None):
         """Queries [tokens, heads, row] ready for attention; keys and values written to the
         pages. ``value_dim``, ``amplitude`` (a factor on cosine and sine) and ``norm_after``
         (queries and keys divided by their root mean square after the rotation, no weight)
         select the general kernel, which pads queries, keys and values with zeros to the
-        pages' row size."""
+        pages' row size. So do ``norm_rows`` (the norm is taken over all heads of the queries, and
+        of the keys, at once, the weights are of those sizes), ``temperature`` (coef, every: queries
+        at position p times 1 + coef ln(floor((p + 1) / every) + 1)) and ``value_mix`` (m, first:
+        values (1 - m) v + m first, ``first`` [tokens, kv_heads * value_dim])."""
         tokens = qkv.shape[0]
         inv_freq, rotary_dim = (None, 0) if rotary is None else rotary
         row_dim = view.kv.shape[-1]
         value_dim = value_dim or head_dim
-        general = value_dim != head_dim or row_dim != head_dim or amplitude != 1.0 or norm_after
+        general = (value_dim != head_dim or row_dim != head_dim or amplitude != 1.0 or norm_after
+                   or norm_rows or temperature is not None or value_mix is not None)
         if general:
             self._need_rows(qkv, view.kv.dtype, "qkv")
         else:
@@ -1365,11 +1492,27 @@ class CudaOps:
             if norm_after and eps is None:
                 raise KernelError("a norm after the rotation needs its eps")
             mode = 2 if norm_after else (1 if q_weight is not None else 0)
+            if norm_rows:
+                mode = 3
+                if eps is None or q_weight is None or q_weight.numel() != heads * head_dim or \
+                        k_weight.numel() != kv_heads * head_dim:
+                    raise KernelError("a norm over whole rows needs its eps and weights of the rows' sizes")
+            mixed = ()
+            if temperature is not None or value_mix is not None:
+                coef, every = temperature or (0.0, 1.0)
+                factor, first = value_mix or (0.0, None)
+                if first is not None:
+                    self._need_rows(first, qkv.dtype, "the first values")
+                    if first.shape != (tokens, kv_heads * value_dim):
+                        raise KernelError("values of different sizes cannot be mixed")
+                mixed = (_c_float(coef), ctypes.c_double(every), _c_void_p(_ptr(first)),
+                         _c_int(0 if first is None else first.stride(0)), _c_float(factor))
             q = torch.empty((tokens, heads, row_dim), dtype=qkv.dtype, device=self.device)
-            self._call("mlxone_qk_prep_general", _c_void_p(_ptr(qkv)), _c_void_p(_ptr(q_weight)),
+            self._call("mlxone_qk_prep_mixed" if mixed else "mlxone_qk_prep_general",
+                       _c_void_p(_ptr(qkv)), _c_void_p(_ptr(q_weight)),
                        _c_void_p(_ptr(k_weight)), _c_float(0.0 if eps is None else eps),
                        _c_void_p(_ptr(inv_freq)), _c_int(rotary_dim), _c_float(amplitude),
-                       _c_int(mode), _c_void_p(_ptr(ctx.positions)),
+                       _c_int(mode), *mixed, _c_void_p(_ptr(ctx.positions)),
                        _c_void_p(_ptr(ctx.token_request)), _c_void_p(_ptr(q)),
                        _c_void_p(_ptr(view.kv)), _c_void_p(_ptr(view.block_table)),
                        _c_int(view.block_table.shape[1]), _c_int(view.page_size),
@@ -1405,7 +1548,7 @@ class CudaOps:
 
     def qkv_attention(self, qkv, *, heads, kv_heads, head_dim, q_weight, k_weight, eps, rotary,
                       scale, window, ctx, view, write, sinks=None, chunk=None, keep_first=0,
-                      **extra):
+                      score_cap=0.0, slopes=None, least_slope=0.0, **extra):
         """From the fused projection qkv [tokens, (heads + 2 kv_heads) * head_dim] to the mixed
         heads [tokens, heads * head_dim]: per-head norm of queries and keys, rotation, keys and
         values appended to the pages, attention. A step of single tokens in bfloat16 whose head
@@ -1414,6 +1557,9 @@ class CudaOps:
         tokens = qkv.shape[0]
         inv_freq, rotary_dim = (None, 0) if rotary is None else rotary
         window = self._span(window, chunk)
+        shaped = {}
+        if score_cap or slopes is not None:
+            shaped = dict(score_cap=score_cap, slopes=slopes, least_slope=least_slope)
         if extra:
             # (value size, amplitude, norm after the rotation: see qk_norm_rope_store) the
             # general preparation, then attention over rows of the pages' size; the output has
@@ -1423,8 +1569,9 @@ class CudaOps:
                                         rotary=rotary, ctx=ctx, view=view, write=write, **extra)
             return self.paged_attention(q, heads=heads, kv_heads=kv_heads,
                                         head_dim=view.kv.shape[-1], scale=scale, window=window,
-                                        ctx=ctx, view=view, sinks=sinks, keep_first=keep_first)
-        if (self.fused_decode_attention and qkv.dtype == torch.bfloat16
+                                        ctx=ctx, view=view, sinks=sinks, keep_first=keep_first,
+                                        **shaped)
+        if (not shaped and self.fused_decode_attention and qkv.dtype == torch.bfloat16
                 and ctx.max_portion == 1 and tokens == ctx.requests
                 and self.tensor_core_attention and not keep_first
                 and self.lib.mlxone_attention_decode_fused_supports(_c_int(head_dim))
@@ -1455,15 +1602,23 @@ class CudaOps:
                                     ctx=ctx, view=view, write=write)
         return self.paged_attention(q, heads=heads, kv_heads=kv_heads, head_dim=head_dim,
                                     scale=scale, window=window, ctx=ctx, view=view, sinks=sinks,
-                                    keep_first=keep_first)
+                                    keep_first=keep_first, **shaped)
 
     def paged_attention(self, q, *, heads, kv_heads, head_dim, scale, window, ctx, view,
-                        sinks=None, chunk=None, keep_first=0):
+                        sinks=None, chunk=None, keep_first=0, score_cap=0.0, slopes=None,
+                        least_slope=0.0):
         """Attention of every token over its request's pages. ``keep_first``: behind a window the
         first ``keep_first`` positions of a sequence stay visible. bfloat16 with a head size that
         is a multiple of 16 up to 128 runs on tensor cores: the split-key decode kernel when
         every request brings one token, else the prefill kernel. Everything else (float32,
-        other head sizes) runs the general kernel."""
+        other head sizes) runs the general kernel. ``score_cap`` c (0: none): scores s become c
+        tanh(s / c); ``slopes`` (float32 [heads] or None): then they lose slope * (query's position
+        - key's); ``least_slope`` is their minimum on the host."""
+        if score_cap or slopes is not None:
+            if window or chunk or keep_first or sinks is not None:
+                raise KernelError("shaped scores go without windows, chunks and sinks")
+            return self._shaped_attention(q, heads, kv_heads, head_dim, scale, ctx, view,
+                                          float(score_cap), slopes, float(least_slope))
         tokens = q.shape[0]
         out = torch.empty((tokens, heads * head_dim), dtype=q.dtype, device=self.device)
         width = view.block_table.shape[1]
@@ -1556,6 +1711,79 @@ class CudaOps:
                    _c_void_p(_ptr(out)), _c_int(tokens), _c_int(heads), _c_int(kv_heads),
                    _c_int(head_dim), _c_float(scale), _c_int(window or 0),
                    _c_int(code), _c_void_p(_ptr(sinks)), _c_void_p(_ptr(self.error_flag)))
+        return out
+
+    def _shaped_attention(self, q, heads, kv_heads, head_dim, scale, ctx, view, cap, slopes, least_slope):
+        """paged_attention with capped or distance-biased scores, on the same kernels built with the
+        shaping of scores. With both, a key so far back that its weight underflows beside the
+        query's own is not read (the kernels find the bound per head): the host bounds the splits of
+        the keys by the farthest that any head reads."""
+        tokens = q.shape[0]
+        if slopes is not None:
+            self._need(slopes, torch.float32, "slopes")
+            if slopes.numel() != heads:
+                raise KernelError("one slope per query head")
+        out = torch.empty((tokens, heads * head_dim), dtype=q.dtype, device=self.device)
+        width, pages = view.block_table.shape[1], view.kv.shape[1]
+        code = _dtype_code(q.dtype)
+        shape = (_c_float(scale), _c_float(cap), _c_void_p(_ptr(slopes)))
+        if not (self.tensor_core_attention and self.lib.mlxone_attention_mma_supports(head_dim, code)):
+            self._call("mlxone_attention_generic_shaped", _c_void_p(_ptr(q)), _c_void_p(_ptr(view.kv)),
+                       _c_void_p(_ptr(view.block_table)), _c_int(width), _c_int(view.page_size),
+                       _c_int(pages), _c_void_p(_ptr(ctx.positions)),
+                       _c_void_p(_ptr(ctx.token_request)), _c_void_p(_ptr(out)), _c_int(tokens),
+                       _c_int(heads), _c_int(kv_heads), _c_int(head_dim), *shape, _c_int(code),
+                       _c_void_p(_ptr(self.error_flag)))
+            return out
+        bound = min(ctx.max_context, width * view.page_size)
+        reach = None
+        if cap > 0 and least_slope > 0:
+            reach = int((2 * cap + 88) / least_slope) + 2
+        # the requests at the head of the step that bring one token each (all of a step of single
+        # tokens) go to the split-key kernel, the rest to the prefill kernel
+        single_step = ctx.max_portion == 1 and tokens == ctx.requests
+        singles = ctx.requests if single_step else min(getattr(ctx, "leading_single", 0), ctx.requests)
+        if singles < self.split_singles_from:
+            singles = 0
+        if singles:
+            splits, partial = self._decode_plan(singles, heads, kv_heads, head_dim, width, reach, view)
+            self._call("mlxone_attention_decode_shaped", _c_void_p(_ptr(q)), _c_void_p(_ptr(view.kv)),
+                       _c_void_p(_ptr(view.block_table)), _c_int(width), _c_int(view.page_size),
+                       _c_int(pages), _c_void_p(_ptr(ctx.positions)), _c_void_p(_ptr(out)),
+                       _c_void_p(_ptr(partial)), _c_int(singles), _c_int(heads), _c_int(kv_heads),
+                       _c_int(head_dim), _c_int(splits), *shape)
+            if partial is not None:
+                self.launches += 1          # the merge kernel
+        if single_step:
+            return out
+        rest = ctx.requests - singles
+        table, starts, history = (view.block_table[singles:], ctx.request_start[singles:],
+                                  ctx.history[singles:])
+        common = (_c_void_p(_ptr(q)), _c_void_p(_ptr(view.kv)), _c_void_p(_ptr(table)), _c_int(width),
+                  _c_int(view.page_size), _c_int(pages), _c_void_p(_ptr(starts)),
+                  _c_void_p(_ptr(history)), _c_void_p(_ptr(out)), _c_int(tokens), _c_int(rest),
+                  _c_int(heads), _c_int(kv_heads), _c_int(head_dim), *shape)
+        if not (self.tcgen05_attention and self.lib.mlxone_attention_tcgen05_supports(
+                _c_int(head_dim), _c_int(heads), _c_int(kv_heads), _c_int(view.page_size))):
+            self._call("mlxone_attention_prefill_shaped", *common)
+            return out
+        splits = 1
+        if reach is not None:
+            bound = min(bound, reach + ctx.max_portion)
+        if self.prefill_key_splits:
+            splits = self.lib.mlxone_attention_tcgen05_splits(
+                _c_int(tokens - singles), _c_int(rest), _c_int(heads), _c_int(kv_heads), _c_int(bound))
+        partial = None
+        if splits > 1:
+            partial = torch.empty(tokens * heads * splits * (head_dim + 2), dtype=torch.float32,
+                                  device=self.device)
+        self._call("mlxone_attention_prefill_tcgen05_shaped", *common, _c_int(splits),
+                   _c_void_p(_ptr(partial)), _c_void_p(_ptr(self.error_flag)))
+        if partial is not None:
+            skip = singles * heads * splits * (head_dim + 2)
+            self._call("mlxone_attention_merge", _c_void_p(_ptr(partial[skip:])),
+                       _c_void_p(_ptr(out[singles:])), _c_int((tokens - singles) * heads),
+                       _c_int(splits), _c_int(head_dim))
         return out
 
     def _decode_attention(self, q, out, requests, heads, kv_heads, head_dim, scale, window, ctx,
