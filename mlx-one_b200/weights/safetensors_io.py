@@ -160,4 +160,4 @@ def write_safetensors(path: str | Path, tensors: Mapping[str, torch.Tensor],
         out.write(blob)
         for name in order:
             tensor = tensors[name].detach().cpu().contiguous()
-            out.write(tensor.view(torch.uint8).numpy().tobytes() if tensor.numel() else b"")
+            out.write(tensor.reshape(-1).view(torch.uint8).numpy().tobytes() if tensor.numel() else b"")
