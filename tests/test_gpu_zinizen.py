@@ -160,7 +160,7 @@ SHAPED = [
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("heads, kv_heads, dim, cap, sloped, scale", SHAPED)
 def test_capped_and_distance_biased_scores(ops, dtype, heads, kv_heads, dim, cap, sloped, scale):
-    """One key near the start of 700 matches the last queries by far and is worth 3 in its values,
+    """One key near the start of 700 matches the last queries by far and is worth 45 in its values,
     several near ones match by less: what the far one is worth depends on the cap and on the
     distance, head by head. In whole prompts, portions beside single tokens, and single tokens at
     page and tile borders whose keys are cut into runs."""
@@ -171,14 +171,14 @@ def test_capped_and_distance_biased_scores(ops, dtype, heads, kv_heads, dim, cap
     T, page = 700, 16
     q, k, v = 0.4 * draw(T, heads, dim), 0.4 * draw(T, kv_heads, dim), 0.5 * draw(T, kv_heads, dim)
     q[-50:, :, 1] = 5.0
-    k[5, :, 1], v[5] = 9.0, 3.0
+    k[5, :, 1], v[5] = 9.0, 45.0
     k[T - 90:T - 60:7, :, 1] = 1.5
     q, k, v = q.to(dtype), k.to(dtype), v.to(dtype)
     slope = plain.slopes(heads, torch.float32) * 0.25 if sloped else torch.zeros(heads)
     want = plain_scores(q, k, v, scale, cap, slope)
     near = plain_scores(q[8:], k[8:], v[8:], scale, cap, slope)         # without the far key
     if float(slope.min()) * T < 15:
-        assert (want[-1] - near[-1]).abs().max() > 0.3                   # it shows
+        assert (want[-1] - near[-1]).abs().max() > 0.2                   # it shows
     table, pool = page_tables((T,), page, generator)
     kv = torch.full((2, pool, kv_heads, page, dim), 100.0).to(dtype)
     for t in range(T):
@@ -200,7 +200,8 @@ def test_capped_and_distance_biased_scores(ops, dtype, heads, kv_heads, dim, cap
         got = ops.paged_attention(on(q[positions]).contiguous(), heads=heads, kv_heads=kv_heads,
                                   head_dim=dim, scale=scale, window=None, ctx=ctx, view=view, **shape)
         got = got.view(len(positions), heads, dim).cpu().double()
-        assert (got - want[positions]).abs().max() < tolerance, str(portions)
+        bound = tolerance * torch.clamp(want[positions].abs() / 3, min=1.0)
+        assert ((got - want[positions]).abs() < bound).all(), str(portions)
     ops.check_errors()
 
 
@@ -433,6 +434,9 @@ def test_channels_that_keep_and_channels_that_forget(ops, dtype):
     decoding and in a prompt of several chunks."""
     width = 64
     case = recurrence_case(width, 4, dtype, 3)
+    for name in ("ra", "ri", "ra_b"):
+        case[name].zero_()
+    case["ri_b"].fill_(3.0)
     case["lam"] = torch.cat([torch.full((32,), -13.0), torch.full((16,), -8.0), torch.full((16,), 30.0)])
     generator = torch.Generator().manual_seed(9)
     u = 0.3 * torch.randn(1100, width, generator=generator)
@@ -449,7 +453,8 @@ def test_channels_that_keep_and_channels_that_forget(ops, dtype):
         assert torch.isfinite(got).all()
         error = ((got - want).abs() / torch.clamp(want.abs(), min=0.1))
         assert error.max() < (2e-3 if dtype == torch.float32 else 0.03), str(portions)
-        bound = 2e-5 if dtype == torch.float32 else 0.02
+        # (a decay that close to 1 is off by half a unit of 2^-24 in 32-bit, and so token after token)
+        bound = 1e-4 if dtype == torch.float32 else 0.02
         assert ((got - want).abs() < bound * torch.clamp(want.abs(), min=1.0)).all(), str(portions)
 
 

@@ -79,7 +79,7 @@ Z2 = {"architecture": "Zinizen", "vocab": 257, "width": 52, "norm": {"eps": 1e-6
 # one head, one key head, one part, one expert, six taps, no second table; keys and values of
 # equal size
 Z3 = {"architecture": "Zinizen", "vocab": 64, "width": 36, "norm": {"eps": 1e-5},
-      "layers": [attention(1, 1, 16, 16, 0.4, moe(1, 1, 16, 0.7, 1.0, (8, 2.0)), 50.0, (1.0, 1), True),
+      "layers": [attention(1, 1, 16, 16, 0.4, moe(1, 1, 16, 0.7, 1.0, (8, 2.0)), 50.0, (0.3, 1), True),
                  rglru(8, 1, 6, moe(4, 4, 24, 0.9, 0.7)),
                  latent(1, 8, 2, 12, 16, 8, 0.5, dense(40), base=100.0)]}
 
