@@ -17,6 +17,8 @@ Two more workloads, each printing one JSON line of its own (the default line is 
 
     python bench.py --case batching     continuous batching of 128 requests at the LFM2-700M shape
     python bench.py --case long         4 x 32,768-token prompts at the LFM2-350M shape, then decoding
+    python bench.py --case zinizen      Zinizen beside Tirudra and Susalorn at equal width, depth and
+                                        vocabulary: decode and prefill, and the new kernels alone
     python bench.py --case susalorn     Susalorn beside Lamisun and Galarax at equal width, depth and
                                         vocabulary: decode and prefill, and the new kernels alone
     python bench.py --case lamisun      Lamisun beside LFM2 at equal width, depth and vocabulary:
@@ -252,6 +254,9 @@ def model_flops(spec, tokens):
             elif part.kind == "channel_delta":
                 # 32-bit multiply-adds of the recurrence (not tensor-core work, but work)
                 flops += 6 * tokens * part["heads"] * part["key_dim"] * part["value_dim"]
+            elif part.kind == "rglru":
+                # the gates' block-diagonal products
+                flops += 4 * tokens * part["width"] * (part["width"] // part["blocks"])
             elif part.kind == "mamba2":
                 flops += 4 * tokens * part["heads"] * part["state"] * part["value_dim"]
     return flops
@@ -1919,6 +1924,277 @@ def case_susalorn(args) -> int:
     return 0
 
 
+# --------------------------------------------------------------------------- Zinizen beside Tirudra and Susalorn
+
+
+def zinizen_shape(width: int, layers: int, vocab: int = 65536) -> dict:
+    """A Zinizen of the sizes that a model of this width has: gated recurrences as wide as the model
+    (gates in parts of 256 channels, four taps) in every other layer, between them in turn attention
+    with a distance bias (heads of 64, one key head per four query heads, values mixed) and attention
+    over latent rows (as Susalorn's); eight routed experts of the model's width of which a token uses
+    three, beside a shared one (as Tirudra's)."""
+    rot_dim, latent = (32, 256) if width <= 1024 else (64, 512)
+    attention = {"heads": width // 64, "kv_heads": width // 256, "dim": 64, "vdim": 64, "scale": 0.125,
+                 "softcap": 50.0, "q_temp": {"coef": 0.1, "every": 4096}, "v_mix": True}
+    rows = {"heads": width // 64, "dim": 64, "rot_dim": rot_dim, "vdim": 64, "kv_rank": latent,
+            "q_rank": width // 2, "scale": (64 + rot_dim) ** -0.5, "rot": {"base": 10000.0, "dims": rot_dim}}
+    recurrence = {"width": width, "blocks": width // 256, "conv": 4}
+    moe = {"kind": "moe", "expert": {"ff": width, "limit": 7.0}, "shared": {"ff": width, "limit": 7.0},
+           "router": {"experts": 8, "top": 3, "scale": 1.0}}
+    entries = []
+    for index in range(layers):
+        mixer = (("rglru", recurrence), ("attention", attention), ("rglru", recurrence),
+                 ("latent_attention", rows))[index % 4]
+        entries.append({"type": mixer[0], "mixer": mixer[1], "mlp": moe})
+    return {"architecture": "Zinizen", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "embedding": {"bigram": {"buckets": vocab - 1, "mul_prev": 1000003, "mul_cur": 31}},
+            "layers": entries}
+
+
+def zinizen_kernels(width, batch, peak):
+    """The kernels that Zinizen adds, alone, beside the like kernels of Tirudra, for a decode step of
+    ``batch`` tokens over 2,048 earlier ones and a prompt of PREFILL_TOKENS tokens: algorithmic
+    bytes (or flops) / time against the measured peaks. Arguments rotate over copies that together
+    exceed L2."""
+    import torch
+
+    from mlx_one_b200.kernels import default_ops
+    from mlx_one_b200.parts import (FixedState, NormedUpdate, PagedKeyValues, PagedView, StateView,
+                                    StepContext)
+
+    ops, device = default_ops("cuda:0"), "cuda:0"
+    ints = lambda values: torch.tensor(values, dtype=torch.int32, device=device)
+    bf16 = lambda *shape: torch.randn(*shape, device=device).bfloat16()
+
+    def ctx_of(portions, histories):
+        positions, owner, starts = [], [], [0]
+        for r, (n, before) in enumerate(zip(portions, histories)):
+            positions += list(range(before, before + n))
+            owner += [r] * n
+            starts.append(starts[-1] + n)
+        return StepContext(tokens=len(positions), requests=len(portions),
+                           token_ids=ints([0] * len(positions)), positions=ints(positions),
+                           token_request=ints(owner), request_start=ints(starts),
+                           history=ints(histories), max_portion=max(portions),
+                           max_context=max(p + h for p, h in zip(portions, histories)))
+
+    def entry(seconds, moved=None, flops=None):
+        out = {"us": round(seconds * 1e6, 2)}
+        if moved is not None:
+            out["gbs"] = round(moved / seconds / 1e9, 1)
+            out["hbm_frac"] = round(moved / seconds / 1e9 / peak["hbm_gbs"], 4)
+        if flops is not None:
+            out["tflops"] = round(flops / seconds / 1e12, 2)
+            out["tensor_frac"] = round(flops / seconds / 1e12 / peak["bf16_tflops"], 4)
+        return out
+
+    out = {}
+    for label, portions, histories in (("decode", [1] * batch, [2048] * batch),
+                                       ("prefill", [PREFILL_TOKENS], [0])):
+        ctx = ctx_of(portions, histories)
+        tokens, requests = ctx.tokens, ctx.requests
+        # ---- a part's output normed into the stream and the next norm, beside Tirudra's two kernels
+        copies = 16 if label == "prefill" else 4
+        residual = [torch.zeros(tokens, width, device=device) for _ in range(copies)]
+        delta = [bf16(tokens, width) for _ in range(copies)]
+        vector = torch.ones(width, device=device)
+        moved = tokens * width * (4 + 4 + 2 + 2)
+        seconds = graph_seconds(lambda i: ops.add_norm(
+            residual[i], NormedUpdate(delta[i], vector, vector, 1e-6), vector, vector, 1e-6,
+            torch.bfloat16), copies, 2 * copies)
+        out[f"{label}_layer_norms"] = entry(seconds, moved)
+
+        def two_norms(i):
+            ops.normed_mean_add(residual[i], [delta[i]], [vector], 1e-6)
+            ops.add_rmsnorm(residual[i], None, vector, 1e-6, torch.bfloat16)
+
+        out[f"{label}_two_norms_tirudra"] = entry(graph_seconds(two_norms, copies, 2 * copies), moved)
+        del residual, delta
+        # ---- the recurrence (with its gates' product) beside the state space
+        part = 256
+        blocks = width // part
+        copies = 24
+        state = torch.zeros(copies * requests, width, device=device)
+        slots = [ints(list(range(c * requests, (c + 1) * requests))) for c in range(copies)]
+        views = [StateView(state, slots[c], FixedState((width,), "float32")) for c in range(copies)]
+        u = [bf16(tokens, width) for _ in range(copies)]
+        both = [bf16(tokens, 2 * width) for _ in range(copies)]
+        gates = [bf16(blocks, 2 * part, part) * 0.06 for _ in range(copies)]
+        bias, rate = torch.zeros(blocks, 2 * part, device=device), torch.full((width,), -0.3, device=device)
+        seconds = graph_seconds(lambda i: ops.gated_recurrence(
+            u[i], both[i][:, width:], gates=gates[i], gate_bias=bias, rate=rate, ctx=ctx, view=views[i],
+            write=True), copies, 2 * copies)
+        moved = tokens * width * 2 * 3 + 2 * width * part * 2 + 2 * requests * width * 4
+        out[f"{label}_gated_recurrence"] = entry(seconds, moved)
+        if label == "prefill":
+            product = lambda i: torch.bmm(u[i].view(tokens, blocks, part).transpose(0, 1),
+                                          gates[i].transpose(1, 2), out_dtype=torch.float32)
+            alone = graph_seconds(product, copies, 2 * copies)
+            out[f"{label}_gates_product"] = entry(alone, tokens * width * (2 + 8), 4.0 * tokens * width * part)
+            out[f"{label}_recurrence_alone"] = entry(seconds - alone, tokens * width * (2 + 8 + 2 + 2))
+        taps = 4
+        kept = torch.zeros(copies * requests, taps - 1, width, device=device).bfloat16()
+        conv_views = [StateView(kept, slots[c], FixedState((taps - 1, width))) for c in range(copies)]
+        kernel, conv_bias = torch.randn(width, taps, device=device), torch.zeros(width, device=device)
+        for name, act in (("channel_conv", None), ("channel_conv_tirudra", "silu")):
+            seconds = graph_seconds(lambda i: ops.channel_conv(
+                both[i][:, :width], kernel, conv_bias, taps=taps, activation=act, ctx=ctx,
+                view=conv_views[i], write=True), copies, 2 * copies)
+            out[f"{label}_{name}"] = entry(seconds, tokens * width * 4 + 2 * requests * (taps - 1) * width * 2)
+        del state, views, u, both, gates, kept, conv_views
+        H, P, N = width // 64, 64, 128
+        size, few = H * N * P, 8
+        state = torch.zeros(few * requests, size, device=device)
+        views = [StateView(state, slots[c], FixedState((size,), "float32")) for c in range(few)]
+        mixed = [bf16(tokens, H * P + 2 * N) for _ in range(few)]
+        raw = [bf16(tokens, H) for _ in range(few)]
+        seconds = graph_seconds(lambda i: ops.state_space_scan(
+            mixed[i], raw[i], a_log=vector[:H],
+            dt_bias=vector[:H], skip=vector[:H], ctx=ctx, view=views[i], write=True, heads=H,
+            value_dim=P, state_dim=N, groups=1), few, 2 * few)
+        out[f"{label}_state_space_tirudra"] = entry(
+            seconds, tokens * ((H * P + 2 * N + H) * 2 + H * P * 4) + 2 * requests * size * 4)
+        del state, views, mixed, raw
+        # ---- attention: the preparation (norms over rows, temperature, mixed values, page write) beside
+        # Tirudra's (norms per head, scaled rotation), then attention with and without the scores' shape
+        for head in (64, 128):
+            heads, kv_heads = width // head, width // (4 * head)
+            span = histories[0] + portions[0]
+            pages = -(-span // PAGE_SIZE)
+            table = ints([[r * pages + b for b in range(pages)] for r in range(requests)])
+            kv = (torch.randn(2, requests * pages + 1, kv_heads, PAGE_SIZE, head, device=device) * 0.3).bfloat16()
+            view = PagedView(kv, table, PAGE_SIZE, PagedKeyValues(kv_heads, head))
+            copies = 8
+            wide = (heads + 2 * kv_heads) * head
+            qkv = [bf16(tokens, wide) for _ in range(copies)]
+            q = [bf16(tokens, heads, head) * 0.5 for _ in range(copies)]
+            ones = torch.ones(wide, device=device)
+            common = dict(heads=heads, kv_heads=kv_heads, head_dim=head, eps=1e-6, ctx=ctx, view=view,
+                          write=True)
+            seconds = graph_seconds(lambda i: ops.qk_norm_rope_store(
+                qkv[i], q_weight=ones[:heads * head], k_weight=ones[:kv_heads * head], rotary=None,
+                norm_rows=True, temperature=(0.1, 4096.0),
+                value_mix=(0.4, qkv[(i + 1) % copies][:, wide - kv_heads * head:]), **common),
+                copies, 2 * copies)
+            out[f"{label}_prep_rows_{head}"] = entry(seconds, tokens * (2 * wide + kv_heads * head) * 2)
+            rotary = (torch.rand(head // 2, device=device), head)
+            seconds = graph_seconds(lambda i: ops.qk_norm_rope_store(
+                qkv[i], q_weight=ones[:head], k_weight=ones[:head], rotary=rotary, amplitude=1.2, **common),
+                copies, 2 * copies)
+            out[f"{label}_prep_tirudra_{head}"] = entry(seconds, tokens * 2 * wide * 2)
+            slopes = [2.0 ** (-8.0 * (h + 1) / heads) for h in range(heads)]
+            shape = dict(score_cap=50.0, slopes=torch.tensor(slopes, device=device), least_slope=min(slopes))
+            # (keys that a head's slope leaves without weight are not read: count what is)
+            reach = [188.0 / s for s in slopes]
+            seen = lambda h: sum(min(b + i + 1, reach[h]) for n, b in zip(portions, histories) for i in range(n))
+            all_seen = sum(b + i + 1 for n, b in zip(portions, histories) for i in range(n))
+            group = heads // kv_heads
+            keys = sum(min(span, max(reach[g * group:(g + 1) * group]) + portions[0]) for g in range(kv_heads))
+            own = tokens * heads * head * 2 * 2
+            for name, extra, flops, read in (
+                    ("attention_shaped", shape, 4.0 * head * sum(seen(h) for h in range(heads)), keys),
+                    ("attention_biased_uncapped", dict(shape, score_cap=0.0), 4.0 * head * heads * all_seen, kv_heads * span),
+                    ("attention_plain", {}, 4.0 * head * heads * all_seen, kv_heads * span)):
+                seconds = graph_seconds(lambda i: ops.paged_attention(
+                    q[i], heads=heads, kv_heads=kv_heads, head_dim=head, scale=0.125, window=None, ctx=ctx,
+                    view=view, **extra), copies, 2 * copies)
+                out[f"{label}_{name}_{head}"] = entry(seconds, requests * read * head * 2 * 2 + own, flops)
+            # every key within reach: what the shaping itself costs
+            flat = dict(shape, slopes=torch.full((heads,), 1e-4, device=device), least_slope=1e-4)
+            seconds = graph_seconds(lambda i: ops.paged_attention(
+                q[i], heads=heads, kv_heads=kv_heads, head_dim=head, scale=0.125, window=None, ctx=ctx,
+                view=view, **flat), copies, 2 * copies)
+            out[f"{label}_attention_shaped_all_keys_{head}"] = entry(
+                seconds, requests * kv_heads * span * head * 2 * 2 + own, 4.0 * head * heads * all_seen)
+            del kv, qkv, q
+        # ---- the routed feed-forward with clamped gates beside Tirudra's with silu, equal sizes
+        experts, top, ff, shared = 8, 3, width, width
+        copies = max(2, min(12, int(300e6 // ((experts * ff + shared) * width * 6))))
+        stack = experts * ff + shared
+        gate_up = [bf16(2 * stack, width) * 0.02 for _ in range(copies)]
+        down = [bf16(width, stack) * 0.02 for _ in range(copies)]
+        x = bf16(tokens, width)
+        at = experts * ff
+        alone = [(torch.cat([g[at:at + shared], g[stack + at:stack + at + shared]]).contiguous(),
+                  d[:, at:].contiguous()) for g, d in zip(gate_up, down)]
+        router, correction = torch.randn(experts, width, device=device), torch.zeros(experts, device=device)
+
+        def routed(i, clamped):
+            weights, _ = ops.route_general(x, router, correction, experts=experts, identity=0, top=top,
+                                           scores="softmax", normalize=True, shared_gate=False)
+            if ops.sorts_experts(x, experts=experts, width=ff, top=top, stack=stack):
+                form = dict(activation="clamped", limit=7.0, shared_limits=(7.0, 7.0, 0)) if clamped else {}
+                return ops.routed_experts_sorted(x, weights, gate_up[i], down[i], experts=experts, width=ff,
+                                                 top=top, shared_gate_up=alone[i][0],
+                                                 shared_down=alone[i][1], **form)
+            gated = ops.linear_gated(x, gate_up[i], "clamped", limits=(7.0, 7.0, at)) if clamped \
+                else ops.linear_swiglu(x, gate_up[i])
+            ops.scale_expert_columns(gated, weights, ff)
+            return ops.linear(gated, down[i])
+
+        touched = min(experts, tokens * top) * ff + shared
+        for name, clamped in (("routed_ff_clamped", True), ("routed_ff_tirudra", False)):
+            seconds = graph_seconds(lambda i: routed(i, clamped), copies, 2 * copies)
+            out[f"{label}_{name}"] = entry(
+                seconds, touched * width * 6 if label == "decode" else None,
+                6.0 * tokens * (top * ff + shared) * width if label == "prefill" else None)
+        del gate_up, down, alone
+        torch.cuda.empty_cache()
+    return out
+
+
+def case_zinizen(args) -> int:
+    """Zinizen beside Tirudra (norms ahead of and behind every part, a recurrent mixer with a
+    convolution ahead, routed experts with a shared one) and Susalorn (attention over latent rows with
+    a query latent), the closest of the engine's models, at equal width, depth and vocabulary, random
+    weights: decode tokens/s at ``--batch`` and ``--context`` (device-timed graph replays of the
+    engine's step), prefill tokens/s of one 2,048-token prompt, each against its bound, and the new
+    kernels alone."""
+    import gc
+
+    import torch
+
+    peak = peaks()
+    warmup, steps = max(args.warmup, 3), min(args.steps, 128)
+    context = args.context or 2048
+    layers = min(args.layers, 8)
+    results = {}
+    for width in (1024, 2048):
+        for label, data in ((f"zinizen_w{width}", zinizen_shape(width, layers)),
+                            (f"tirudra_w{width}", tirudra_shape(width, layers)),
+                            (f"susalorn_w{width}", susalorn_shape(width, layers))):
+            engine = engine_of(data, args.batch, context, warmup + steps, f"random-{label}")
+            model, spec = engine.model, engine.model.spec
+            weight_bytes = model.weight_bytes()
+            kv_per_token = engine.cache_bytes_per_token()
+            state_bytes = sum(g.storage[:, 0].numel() * g.storage.element_size()
+                              for g in engine.cache.states)
+            seconds, _, mean_context, launches = time_decode(engine, args.batch, context, warmup,
+                                                             steps, seed=3)
+            step_bytes = weight_bytes + args.batch * (mean_context * kv_per_token + 2 * state_bytes)
+            prefill_seconds = time_prefill(engine, PREFILL_TOKENS, 2, 3, seed=5)
+            flops = model_flops(spec, PREFILL_TOKENS)
+            results[label] = {
+                "layers": layers, "weight_mb": round(weight_bytes / 1e6, 1),
+                "state_mb_per_request": round(state_bytes / 1e6, 2),
+                "decode_tokens_per_s": round(args.batch * steps / seconds, 1),
+                "decode_ms_per_step": round(seconds / steps * 1e3, 4),
+                "decode_hbm_frac": round(step_bytes / (seconds / steps) / 1e9 / peak["hbm_gbs"], 4),
+                "launches_per_step": launches,
+                "prefill_tokens_per_s": round(PREFILL_TOKENS / prefill_seconds, 1),
+                "prefill_ms": round(prefill_seconds * 1e3, 3),
+                "prefill_tensor_frac": round(flops / prefill_seconds / (peak["bf16_tflops"] * 1e12), 4)}
+            del engine, model
+            gc.collect()
+            torch.cuda.empty_cache()
+        results[f"kernels_w{width}"] = zinizen_kernels(width, args.batch, peak)
+    print(json.dumps({"case": "zinizen", "batch": args.batch, "context": context, "steps": steps,
+                      "warmup": warmup, "dtype": "bf16", "peaks": peak["source"],
+                      "data": "synthetic: random weights, seeded uniform-random token ids",
+                      "results": results}))
+    return 0
+
+
 def decode_step_case(batch: int, context: int) -> int:
     """A few eager decode steps of the whole model at the benchmark's sizes, for a list of the
     step's launches (`ncu --metrics gpu__time_duration.sum`): the prompts are fed first, the last
@@ -2352,7 +2628,7 @@ def main() -> int:
     parser.add_argument("--context", type=int, default=None,
                         help="context length (default 4096; --case long: prompt tokens, 32768)")
     parser.add_argument("--case", default="decode", choices=["decode", "batching", "long", "galarax", "farorax", "lamisun",
-                                                               "tirudra", "susalorn"],
+                                                               "tirudra", "susalorn", "zinizen"],
                         help="decode: the default line; batching: 128 requests batched "
                              "continuously (LFM2-700M shape); long: 4 x 32,768 tokens "
                              "(LFM2-350M shape)")
@@ -2391,6 +2667,8 @@ def main() -> int:
         return case_lamisun(args)
     if args.case == "susalorn":
         return case_susalorn(args)
+    if args.case == "zinizen":
+        return case_zinizen(args)
     if args.case == "tirudra":
         return case_tirudra(args)
     args.context = args.context or 4096
