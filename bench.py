@@ -2516,6 +2516,35 @@ def kernel_case(name: str, batch: int, context: int) -> int:
         run = lambda i: ops.channel_delta_rule(rows[i % 4], *ups, view=views[i % 4], **constants)
         work = (f"{ctx.tokens} tokens of {len(portions)} requests, 16 heads of 128 x 128 on 8 key heads, "
                 f"state {slot * 4 / 1e6:.1f} MB a request")
+    elif name in ("recurrence_prefill", "recurrence_decode"):
+        # the gated linear recurrence at the shape of a 2048-wide model: one prompt of 2,048 tokens (the
+        # gates' product, build, chain, walk) or `batch` single tokens (one kernel)
+        from mlx_one_b200.parts import FixedState, StateView
+
+        channels, part = 2048, 256
+        portions = [1] * batch if name == "recurrence_decode" else [PREFILL_TOKENS]
+        ctx, _ = batch_context(portions, [context if name == "recurrence_decode" else 0] * len(portions))
+        state = torch.zeros(4 * len(portions), channels, device=device)
+        views = [StateView(state, torch.arange(c * len(portions), (c + 1) * len(portions), dtype=torch.int32,
+                                               device=device), FixedState((channels,), "float32")) for c in range(4)]
+        rows = [torch.randn(ctx.tokens, channels, device=device).bfloat16() for _ in range(4)]
+        both = [torch.randn(ctx.tokens, 2 * channels, device=device).bfloat16() for _ in range(4)]
+        gates = [(torch.randn(channels // part, 2 * part, part, device=device) / 16).bfloat16() for _ in range(4)]
+        constants = dict(gate_bias=torch.zeros(channels // part, 2 * part, device=device),
+                         rate=torch.full((channels,), -0.3, device=device), ctx=ctx, write=True)
+        run = lambda i: ops.gated_recurrence(rows[i % 4], both[i % 4][:, channels:], gates=gates[i % 4],
+                                             view=views[i % 4], **constants)
+        work = f"{ctx.tokens} tokens of {len(portions)} requests, {channels} channels, gates in parts of {part}"
+    elif name in ("shaped_attention_prefill", "shaped_attention_decode"):
+        # prefill or decode attention with capped scores and a distance bias within every key's reach
+        portions = [1] * batch if name == "shaped_attention_decode" else [PREFILL_TOKENS]
+        ctx, view = batch_context(portions, [context if name == "shaped_attention_decode" else 0] * len(portions))
+        q = torch.randn(ctx.tokens, heads, head_dim, device=device).bfloat16() * 0.5
+        shape = dict(score_cap=50.0, slopes=torch.full((heads,), 1e-4, device=device), least_slope=1e-4)
+        run = lambda i: ops.paged_attention(q, heads=heads, kv_heads=kv_heads, head_dim=head_dim,
+                                            scale=head_dim ** -0.5, window=None, ctx=ctx, view=view, **shape)
+        seen = sum(h + i + 1 for n, h in zip(portions, ctx.history.tolist()) for i in range(n))
+        work = f"{4 * heads * head_dim * seen / 1e9:.1f} GFLOP"
     elif name in ("latent_prefill", "latent_decode"):
         # attention over latent rows at the sizes of a Lamisun 1024 wide: one 2,048-token prompt
         # (the kernel whose warps own 16 rows) or `batch` single tokens (key runs and their merge)
@@ -2644,7 +2673,8 @@ def main() -> int:
                              "swapped_swiglu, mixed_attention, sampling, delta_prefill, delta_decode, lightning_prefill, "
                              "lightning_decode, experts_sorted, latent_prefill, latent_decode, state_space_prefill, "
                              "state_space_decode, channel_conv_prefill, channel_delta_prefill, "
-                             "channel_delta_decode, decode_step (the "
+                             "channel_delta_decode, recurrence_prefill, recurrence_decode, "
+                             "shaped_attention_prefill, shaped_attention_decode, decode_step (the "
                              "whole step, eager, for a launch list), decode_timeline (where "
                              "the graph-replayed step's time goes, kernel by kernel)")
     parser.add_argument("--dependent-launches", type=int, default=1,

@@ -269,8 +269,12 @@ struct Item {
     int window;             // as the kernel's, or what the shape of the scores leaves to be seen
 };
 
-// the place among the keys of the j-th tile that an item walks
+// the place among the keys of the j-th tile that an item walks. Shaped scores fall with the distance, so
+// their tiles are walked from the query's own backwards: the running maximum then hardly moves, where
+// it would climb (and the output be rescaled) tile by tile on the way towards the query.
+template <bool SHAPED>
 __device__ __forceinline__ int tile_of(const Item& item, int j) {
+    if (SHAPED) return item.tile_first + item.tile_count - 1 - j;
     return j < item.kept_tiles ? item.kept_first + j : item.tile_first + j - item.kept_tiles;
 }
 
@@ -474,7 +478,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q,
             // may see its keys
             auto box_row = [&](int j) {
                 long long row = -1;
-                const int key = tile_of(item, j) * KEYS + lane * box_keys;
+                const int key = tile_of<SHAPED>(item, j) * KEYS + lane * box_keys;
                 if (lane < boxes && key <= last_position &&
                     (key + box_keys - 1 >= lowest || key < keep_first)) {
                     const int block = key / page_size;
@@ -628,7 +632,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q,
                 return true;
             };
             for (int j = 0; j < item.tile_count && ok; ++j, ++t) {
-                const int tile_key = tile_of(item, j) * KEYS;
+                const int tile_key = tile_of<SHAPED>(item, j) * KEYS;
                 const int key0 = tile_key + part * MY_KEYS;
                 ok = barrier_wait(s_ready(t & 1), (t >> 1) & 1, error_flag);
                 if (!ok) break;

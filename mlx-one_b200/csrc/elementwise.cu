@@ -379,13 +379,33 @@ __global__ void add_bias_kernel(T* __restrict__ x, const float* __restrict__ bia
     x[i] = from_float<T>(to_float<T>(x[i]) + bias[i % width]);
 }
 
+// The same for bfloat16 with width % 8 == 0: eight neighbouring values a thread, 16-byte accesses.
+__global__ void add_bias_wide_kernel(__nv_bfloat16* __restrict__ x, const float* __restrict__ bias,
+                                     int groups_per_row, long long groups) {
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= groups) return;
+    const int f = (int)(i % groups_per_row) * 8;
+    uint4 v = *reinterpret_cast<const uint4*>(x + i * 8);
+    const float4 lo = *reinterpret_cast<const float4*>(bias + f), hi = *reinterpret_cast<const float4*>(bias + f + 4);
+    __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&v);
+    p[0] = __floats2bfloat162_rn(__low2float(p[0]) + lo.x, __high2float(p[0]) + lo.y);
+    p[1] = __floats2bfloat162_rn(__low2float(p[1]) + lo.z, __high2float(p[1]) + lo.w);
+    p[2] = __floats2bfloat162_rn(__low2float(p[2]) + hi.x, __high2float(p[2]) + hi.y);
+    p[3] = __floats2bfloat162_rn(__low2float(p[3]) + hi.z, __high2float(p[3]) + hi.w);
+    *reinterpret_cast<uint4*>(x + i * 8) = v;
+}
+
 MLXONE_API int mlxone_add_bias(void* x, const float* bias, int rows, int width, int dtype,
                                cudaStream_t stream) {
     if (rows == 0) return 0;
     MLXONE_REQUIRE(rows > 0 && width > 0, "add_bias: bad sizes");
     const long long total = (long long)rows * width;
     const int blocks = ceil_div_host(total, 256);
-    if (dtype == MLXONE_BF16)
+    if (dtype == MLXONE_BF16 && width % 8 == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0 &&
+        (reinterpret_cast<uintptr_t>(bias) & 15) == 0)
+        add_bias_wide_kernel<<<ceil_div_host(total / 8, 256), 256, 0, stream>>>((__nv_bfloat16*)x, bias,
+                                                                               width / 8, total / 8);
+    else if (dtype == MLXONE_BF16)
         add_bias_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>((__nv_bfloat16*)x, bias, width,
                                                                   total);
     else

@@ -66,52 +66,34 @@ struct Math<float> {
     static __device__ __forceinline__ float gelu(float z) { return mlxone_activate(z, MLXONE_ACT_GELU_TANH); }
 };
 
-// V neighbouring values of a row.
+// V (1 or 2) neighbouring values of a row.
 template <int V>
 __device__ __forceinline__ void load_values(const float* p, float (&v)[V]) {
-    if (V == 4) {
-        const float4 x = *reinterpret_cast<const float4*>(p);
-        v[0] = x.x; v[1 % V] = x.y; v[2 % V] = x.z; v[3 % V] = x.w;
+    if (V == 2) {
+        const float2 x = *reinterpret_cast<const float2*>(p);
+        v[0] = x.x; v[V - 1] = x.y;
     } else {
-#pragma unroll
-        for (int i = 0; i < V; ++i) v[i] = p[i];
+        v[0] = *p;
     }
 }
 template <int V>
 __device__ __forceinline__ void load_values(const __nv_bfloat16* p, float (&v)[V]) {
-    if (V == 4) {
-        const uint2 x = *reinterpret_cast<const uint2*>(p);
-        const __nv_bfloat162 lo = *reinterpret_cast<const __nv_bfloat162*>(&x.x);
-        const __nv_bfloat162 hi = *reinterpret_cast<const __nv_bfloat162*>(&x.y);
-        v[0] = __low2float(lo); v[1 % V] = __high2float(lo);
-        v[2 % V] = __low2float(hi); v[3 % V] = __high2float(hi);
+    if (V == 2) {
+        const __nv_bfloat162 x = *reinterpret_cast<const __nv_bfloat162*>(p);
+        v[0] = __low2float(x); v[V - 1] = __high2float(x);
     } else {
-#pragma unroll
-        for (int i = 0; i < V; ++i) v[i] = __bfloat162float(p[i]);
+        v[0] = __bfloat162float(*p);
     }
 }
 template <int V>
 __device__ __forceinline__ void store_values(float* p, const float (&v)[V]) {
-    if (V == 4) {
-        *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1 % V], v[2 % V], v[3 % V]);
-    } else {
-#pragma unroll
-        for (int i = 0; i < V; ++i) p[i] = v[i];
-    }
+    if (V == 2) *reinterpret_cast<float2*>(p) = make_float2(v[0], v[V - 1]);
+    else *p = v[0];
 }
 template <int V>
 __device__ __forceinline__ void store_values(__nv_bfloat16* p, const float (&v)[V]) {
-    if (V == 4) {
-        const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1 % V]);
-        const __nv_bfloat162 hi = __floats2bfloat162_rn(v[2 % V], v[3 % V]);
-        uint2 x;
-        x.x = *reinterpret_cast<const uint32_t*>(&lo);
-        x.y = *reinterpret_cast<const uint32_t*>(&hi);
-        *reinterpret_cast<uint2*>(p) = x;
-    } else {
-#pragma unroll
-        for (int i = 0; i < V; ++i) p[i] = __float2bfloat16_rn(v[i]);
-    }
+    if (V == 2) *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v[0], v[V - 1]);
+    else *p = __float2bfloat16_rn(v[0]);
 }
 
 struct Operands {
@@ -179,33 +161,44 @@ gated_recurrence_kernel(Operands o, float* __restrict__ carry, int alone) {
     const T* y_row = static_cast<const T*>(o.y) + c;
     T* out_row = static_cast<T*>(o.out) + c;
     const float* z_row = o.z + (size_t)block * o.z_block + within;
-    constexpr int AHEAD = 4;                     // tokens whose operands are asked for together
-    for (int t0 = first; t0 < last; t0 += AHEAD) {
-        float u[AHEAD][V], y[AHEAD][V], zr[AHEAD][V], zi[AHEAD][V];
+    // the operands of the next AHEAD tokens are on their way while the current ones are worked on
+    constexpr int AHEAD = 4;
+    struct Group { float u[AHEAD][V], y[AHEAD][V], zr[AHEAD][V], zi[AHEAD][V]; };
+    auto fetch = [&](Group& g, int t0) {
 #pragma unroll
         for (int k = 0; k < AHEAD; ++k) {
             const int t = min(t0 + k, last - 1);
-            load_values<V>(z_row + (size_t)t * o.z_token, zr[k]);
-            load_values<V>(z_row + (size_t)t * o.z_token + o.part, zi[k]);
-            load_values<V>(u_row + (size_t)t * o.width, u[k]);
-            if (WALK) load_values<V>(y_row + (size_t)t * o.y_ld, y[k]);
+            load_values<V>(z_row + (size_t)t * o.z_token, g.zr[k]);
+            load_values<V>(z_row + (size_t)t * o.z_token + o.part, g.zi[k]);
+            load_values<V>(u_row + (size_t)t * o.width, g.u[k]);
+            if (WALK) load_values<V>(y_row + (size_t)t * o.y_ld, g.y[k]);
         }
+    };
+    auto work = [&](const Group& g, int t0) {
 #pragma unroll
         for (int k = 0; k < AHEAD; ++k) {
             if (t0 + k >= last) break;
             float result[V];
 #pragma unroll
             for (int i = 0; i < V; ++i) {
-                const float r = Math<T>::sigmoid(zr[k][i] + bias_r[i]);
-                const float gate = Math<T>::sigmoid(zi[k][i] + bias_i[i]);
+                const float r = Math<T>::sigmoid(g.zr[k][i] + bias_r[i]);
+                const float gate = Math<T>::sigmoid(g.zi[k][i] + bias_i[i]);
                 float a, rest;
                 Math<T>::decay(rate[i] * r, a, rest);
-                s[i] = fmaf(a, s[i], rest * gate * u[k][i]);
-                if (WALK) result[i] = s[i] * Math<T>::gelu(y[k][i]);
+                s[i] = fmaf(a, s[i], rest * gate * g.u[k][i]);
+                if (WALK) result[i] = s[i] * Math<T>::gelu(g.y[k][i]);
                 else product[i] *= a;
             }
             if (WALK) store_values<V>(out_row + (size_t)(t0 + k) * o.width, result);
         }
+    };
+    Group even, odd;
+    fetch(even, first);
+    for (int t0 = first; t0 < last; t0 += 2 * AHEAD) {
+        fetch(odd, t0 + AHEAD);
+        work(even, t0);
+        fetch(even, t0 + 2 * AHEAD);
+        work(odd, t0 + AHEAD);
     }
     if (!WALK) {
         store_values<V>(mine, product);
@@ -370,22 +363,22 @@ int chunk_length(int tokens, int max_portion) {
 template <typename T>
 void run(const Operands& o, float* carry, int tokens, int max_portion, cudaStream_t stream) {
     auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-    const bool four = o.part % 4 == 0 && o.y_ld % 4 == 0 && o.z_token % 4 == 0 && o.z_block % 4 == 0 &&
-                      aligned(o.u) && (reinterpret_cast<uintptr_t>(o.y) & (sizeof(T) * 4 - 1)) == 0 &&
+    const bool pairs = o.part % 2 == 0 && o.y_ld % 2 == 0 && o.z_token % 2 == 0 && o.z_block % 2 == 0 &&
+                      aligned(o.u) && (reinterpret_cast<uintptr_t>(o.y) & (sizeof(T) * 2 - 1)) == 0 &&
                       aligned(o.z) && aligned(o.gate_bias) && aligned(o.rate) && aligned(o.state) &&
                       aligned(o.out);
     const bool alone = max_portion <= o.chunk;
     const int chunks = alone ? o.requests : ceil_div_host(tokens, o.chunk) + o.requests;
-    const int columns = four ? 4 : 1;
+    const int columns = pairs ? 2 : 1;
     const dim3 grid(ceil_div_host(o.width, 128 * columns), chunks);
     if (!alone) {
-        if (four) launch_kernel(gated_recurrence_kernel<T, 4, false>, grid, dim3(128), 0, stream, true, o, carry, 0);
+        if (pairs) launch_kernel(gated_recurrence_kernel<T, 2, false>, grid, dim3(128), 0, stream, true, o, carry, 0);
         else launch_kernel(gated_recurrence_kernel<T, 1, false>, grid, dim3(128), 0, stream, true, o, carry, 0);
         launch_kernel(gated_recurrence_chain_kernel, dim3(ceil_div_host(o.width, 32), o.requests),
                       dim3(RUNS * 32), 0, stream, true, o, carry);
     }
-    if (four)
-        launch_kernel(gated_recurrence_kernel<T, 4, true>, grid, dim3(128), 0, stream, true, o, carry, alone ? 1 : 0);
+    if (pairs)
+        launch_kernel(gated_recurrence_kernel<T, 2, true>, grid, dim3(128), 0, stream, true, o, carry, alone ? 1 : 0);
     else
         launch_kernel(gated_recurrence_kernel<T, 1, true>, grid, dim3(128), 0, stream, true, o, carry, alone ? 1 : 0);
 }

@@ -352,6 +352,123 @@ qk_prep_general_kernel(const T* __restrict__ qkv, const float* __restrict__ q_we
     }
 }
 
+// Norm mode 3 without a rotation, for bfloat16 rows whose heads are multiples of 8 values: one block per
+// token, the whole row in registers (C pieces of 16 bytes a thread), one pass over memory.
+template <int C>
+__global__ void __launch_bounds__(C == 4 ? 768 : 1024)
+qk_prep_rows_kernel(const __nv_bfloat16* __restrict__ qkv, const float* __restrict__ q_weight,
+                    const float* __restrict__ k_weight, float eps, const int* __restrict__ positions,
+                    const int* __restrict__ token_request, __nv_bfloat16* __restrict__ q_out,
+                    __nv_bfloat16* __restrict__ kv, const int* __restrict__ block_table, int table_width,
+                    int page_size, long long kv_half, int heads, int kv_heads, int head_dim,
+                    int value_dim, int row_dim, int write_kv, int ld, int* __restrict__ error_flag,
+                    PrepExtra extra) {
+    using T = __nv_bfloat16;
+    __shared__ float sums[2][32];
+    griddep_launch();
+    const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int q_size = heads * head_dim, k_size = kv_heads * head_dim, v_size = kv_heads * value_dim;
+    const int pieces = (q_size + k_size + v_size) / 8;
+    griddep_wait();
+    const T* row = settled(qkv) + (size_t)t * ld;
+    const T* first = extra.first == nullptr ? nullptr
+        : settled(static_cast<const T*>(extra.first)) + (size_t)t * extra.first_ld;
+    uint4 raw[C], other[C];
+#pragma unroll
+    for (int c = 0; c < C; ++c) {
+        const int at = (c * blockDim.x + threadIdx.x) * 8;
+        raw[c] = other[c] = make_uint4(0u, 0u, 0u, 0u);
+        if (at < pieces * 8) {
+            raw[c] = *reinterpret_cast<const uint4*>(row + at);
+            if (first != nullptr && at >= q_size + k_size)
+                other[c] = *reinterpret_cast<const uint4*>(first + at - q_size - k_size);
+        }
+    }
+    const int position = positions[t];
+    T* page_base = nullptr;
+    if (write_kv) {
+        const int block = position / page_size;
+        const int page = block < table_width
+                             ? block_table[(size_t)token_request[t] * table_width + block] : -1;
+        if (page >= 0)
+            page_base = kv + ((size_t)page * kv_heads * page_size + position % page_size) * row_dim;
+        else if (threadIdx.x == 0)
+            atomicExch(error_flag, 2);
+    }
+    float warmth = 1.f;
+    if (extra.coef != 0.f)
+        warmth = fmaf(extra.coef, logf((float)(floor((double)(position + 1) / extra.every) + 1.0)), 1.f);
+    float squares[2] = {0.f, 0.f};
+#pragma unroll
+    for (int c = 0; c < C; ++c) {
+        const int at = (c * blockDim.x + threadIdx.x) * 8;
+        const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw[c]);
+        float sum = 0.f;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const float a = __low2float(p[i]), b = __high2float(p[i]);
+            sum = fmaf(a, a, fmaf(b, b, sum));
+        }
+        if (at < q_size) squares[0] += sum;
+        else if (at < q_size + k_size) squares[1] += sum;
+    }
+    const int warps = blockDim.x >> 5;
+#pragma unroll
+    for (int part = 0; part < 2; ++part) {
+        squares[part] = warp_sum(squares[part]);
+        if (lane == 0) sums[part][warp] = squares[part];
+    }
+    __syncthreads();
+    const float q_inv = rsqrtf(warp_sum(lane < warps ? sums[0][lane] : 0.f) / (float)q_size + eps) * warmth;
+    const float k_inv = rsqrtf(warp_sum(lane < warps ? sums[1][lane] : 0.f) / (float)k_size + eps);
+#pragma unroll
+    for (int c = 0; c < C; ++c) {
+        const int at = (c * blockDim.x + threadIdx.x) * 8;
+        if (at >= pieces * 8) continue;
+        const bool is_q = at < q_size, is_k = !is_q && at < q_size + k_size;
+        if (!is_q && page_base == nullptr) continue;
+        const int within = is_q ? at : is_k ? at - q_size : at - q_size - k_size;
+        const int size = is_q || is_k ? head_dim : value_dim;
+        const int head = within / size, place = within - head * size;
+        __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&raw[c]);
+        const __nv_bfloat162* o = reinterpret_cast<const __nv_bfloat162*>(&other[c]);
+        if (is_q || is_k) {
+            const float* weight = (is_q ? q_weight : k_weight) + within;
+            const float4 lo = *reinterpret_cast<const float4*>(weight), hi = *reinterpret_cast<const float4*>(weight + 4);
+            const float w[8] = {lo.x, lo.y, lo.z, lo.w, hi.x, hi.y, hi.z, hi.w};
+            const float inv = is_q ? q_inv : k_inv;
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+                p[i] = __floats2bfloat162_rn(__low2float(p[i]) * inv * w[2 * i],
+                                             __high2float(p[i]) * inv * w[2 * i + 1]);
+        } else if (first != nullptr) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+                p[i] = __floats2bfloat162_rn(
+                    fmaf(extra.mix, __low2float(o[i]), (1.f - extra.mix) * __low2float(p[i])),
+                    fmaf(extra.mix, __high2float(o[i]), (1.f - extra.mix) * __high2float(p[i])));
+        }
+        T* dst = is_q ? q_out + ((size_t)t * heads + head) * row_dim
+                      : page_base + (is_k ? 0 : kv_half) + (size_t)head * page_size * row_dim;
+        *reinterpret_cast<uint4*>(dst + place) = raw[c];
+    }
+    // the zeros behind rows that are shorter than the pages'
+    const int q_pad = (row_dim - head_dim) / 8, v_pad = (row_dim - value_dim) / 8;
+    const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+    for (int i = threadIdx.x; i < (heads + kv_heads) * q_pad; i += blockDim.x) {
+        const int head = i / q_pad, place = head_dim + (i - head * q_pad) * 8;
+        if (head < heads)
+            *reinterpret_cast<uint4*>(q_out + ((size_t)t * heads + head) * row_dim + place) = zero;
+        else if (page_base != nullptr)
+            *reinterpret_cast<uint4*>(page_base + (size_t)(head - heads) * page_size * row_dim + place) = zero;
+    }
+    if (page_base != nullptr)
+        for (int i = threadIdx.x; i < kv_heads * v_pad; i += blockDim.x) {
+            const int head = i / v_pad, place = value_dim + (i - head * v_pad) * 8;
+            *reinterpret_cast<uint4*>(page_base + kv_half + (size_t)head * page_size * row_dim + place) = zero;
+        }
+}
+
 template <int HD>
 static void launch_qk_prep_wide(const void* qkv, const float* q_weight, const float* k_weight,
                                 float eps, const float* inv_freq, const int* positions,
@@ -445,6 +562,23 @@ static int qk_prep_general(const void* qkv, const float* q_weight, const float* 
     const dim3 blocks(tokens, parts < 1 ? 1 : parts);
     const size_t shared = (size_t)(rotary_dim + WARPS * row_dim) * sizeof(float);
     const long long kv_half = (long long)pages * kv_heads * page_size * row_dim;
+    auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    const int pieces = ((heads + kv_heads) * head_dim + kv_heads * value_dim) / 8;
+    if (dtype == MLXONE_BF16 && norm_mode == 3 && inv_freq == nullptr && head_dim % 8 == 0 &&
+        value_dim % 8 == 0 && row_dim % 8 == 0 && ld % 8 == 0 && pieces <= 3072 && aligned(qkv) &&
+        aligned(q_out) && aligned(kv) && aligned(q_weight) && aligned(k_weight) && aligned(extra.first) &&
+        extra.first_ld % 8 == 0) {
+        const int each = pieces > 2048 ? 4 : tokens >= 256 || pieces > 1024 ? 2 : 1;
+        const int threads = (ceil_div_host(pieces, each) + 31) / 32 * 32;
+        auto kernel = each == 4 ? qk_prep_rows_kernel<4> : each == 2 ? qk_prep_rows_kernel<2>
+                                                                     : qk_prep_rows_kernel<1>;
+        launch_kernel(kernel, dim3(tokens), dim3(threads), 0, stream, true, (const __nv_bfloat16*)qkv,
+                      q_weight, k_weight, eps, positions, token_request, (__nv_bfloat16*)q_out,
+                      (__nv_bfloat16*)kv, block_table, table_width, page_size, kv_half, heads, kv_heads,
+                      head_dim, value_dim, row_dim, write_kv, ld, error_flag, extra);
+        MLXONE_LAUNCH_CHECK("qk_prep_rows");
+        return 0;
+    }
     if (dtype == MLXONE_BF16) {
         using T = __nv_bfloat16;
         launch_kernel(qk_prep_general_kernel<T>, blocks, dim3(WARPS * 32), shared, stream, true,

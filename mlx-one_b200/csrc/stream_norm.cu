@@ -64,11 +64,45 @@ __device__ __forceinline__ float row_sum(float v, float* scratch) {
     return warp_sum(lane < warps ? scratch[lane] : 0.f);
 }
 
+// The weight and bias of a norm at this thread's places: held in registers (few rows: they are asked for
+// before the kernel ahead has finished) or read where they are used.
+template <int VEC, bool HELD>
+struct Affine {
+    float w[HELD ? VEC : 1][4], b[HELD ? VEC : 1][4];
+    const float* weight;
+    const float* bias;
+    int hidden, first, step;
+
+    __device__ __forceinline__ Affine(const float* weight_, const float* bias_, int hidden_, int first_, int step_)
+        : weight(weight_), bias(bias_), hidden(hidden_), first(first_), step(step_) {
+        if (HELD)
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) fetch(j, w[HELD ? j : 0], b[HELD ? j : 0]);
+    }
+    __device__ __forceinline__ void fetch(int j, float (&wj)[4], float (&bj)[4]) const {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) wj[i] = bj[i] = 0.f;
+        if (first + j * step >= hidden) return;
+        if (weight != nullptr) load4<float>(weight + first + j * step, wj);
+        if (bias != nullptr) load4<float>(bias + first + j * step, bj);
+    }
+    __device__ __forceinline__ void apply(int j, float (&v)[4], float inv) const {
+        if (HELD) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) v[i] = fmaf(v[i] * inv, w[HELD ? j : 0][i], b[HELD ? j : 0][i]);
+        } else {
+            float wj[4], bj[4];
+            fetch(j, wj, bj);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) v[i] = fmaf(v[i] * inv, wj[i], bj[i]);
+        }
+    }
+};
+
 // Norms this thread's share of a row in place. `scratch`: two rows of 32 floats.
-template <int VEC, bool WARP>
+template <int VEC, bool WARP, bool HELD>
 __device__ __forceinline__ void norm_row(float (&v)[VEC][4], int hidden, int first, int step, int kind,
-                                         float eps, const float (&w)[VEC][4], const float (&b)[VEC][4],
-                                         float* scratch) {
+                                         float eps, const Affine<VEC, HELD>& affine, float* scratch) {
     float mean = 0.f;
     if (kind == 2) {
         float sum = 0.f;
@@ -89,25 +123,12 @@ __device__ __forceinline__ void norm_row(float (&v)[VEC][4], int hidden, int fir
             }
     const float inv = 1.f / sqrtf(row_sum<WARP>(squares, scratch + 32) / (float)hidden + eps);
 #pragma unroll
-    for (int j = 0; j < VEC; ++j)
-#pragma unroll
-        for (int i = 0; i < 4; ++i) v[j][i] = fmaf(v[j][i] * inv, w[j][i], b[j][i]);
-}
-
-template <int VEC>
-__device__ __forceinline__ void load_vector(float (&w)[VEC][4], const float* p, int hidden, int first,
-                                            int step) {
-#pragma unroll
-    for (int j = 0; j < VEC; ++j) {
-#pragma unroll
-        for (int i = 0; i < 4; ++i) w[j][i] = 0.f;
-        if (p != nullptr && first + j * step < hidden) load4<float>(p + first + j * step, w[j]);
-    }
+    for (int j = 0; j < VEC; ++j) affine.apply(j, v[j], inv);
 }
 
 // One row per block (WARP false) or per warp (WARP true), the row in registers: 4 VEC values a thread.
-template <typename T, int VEC, bool WARP>
-__global__ void __launch_bounds__(WARP ? 256 : VEC <= 2 ? 1024 : 512)
+template <typename T, int VEC, bool WARP, bool HELD>
+__global__ void __launch_bounds__(WARP ? 256 : HELD ? 1024 : 512)
 stream_norm_kernel(float* __restrict__ residual, const T* __restrict__ delta, T* __restrict__ out,
                    int rows, int hidden, StreamNorm n) {
     __shared__ float scratch[4 * 32];
@@ -115,17 +136,9 @@ stream_norm_kernel(float* __restrict__ residual, const T* __restrict__ delta, T*
     const int threads = WARP ? 32 : blockDim.x;
     const int row = WARP ? blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5) : blockIdx.x;
     const int first = (WARP ? (threadIdx.x & 31) : threadIdx.x) * 4, step = threads * 4;
-    // the norms' weights do not depend on the kernel before this one (a block asks for them ahead of
-    // the wait; warps with whole rows, of which there are many, when they come to them)
-    float w[VEC][4], b[VEC][4], post_w[VEC][4], post_b[VEC][4];
-    if (!WARP) {
-        load_vector<VEC>(w, n.weight, hidden, first, step);
-        load_vector<VEC>(b, n.bias, hidden, first, step);
-        if (n.post_kind != 0) {
-            load_vector<VEC>(post_w, n.post_weight, hidden, first, step);
-            load_vector<VEC>(post_b, n.post_bias, hidden, first, step);
-        }
-    }
+    // the norms' weights do not depend on the kernel before this one
+    const Affine<VEC, HELD> post(n.post_weight, n.post_bias, hidden, first, step);
+    const Affine<VEC, HELD> next(n.weight, n.bias, hidden, first, step);
     griddep_wait();
     delta = settled(delta);
     if (row >= rows) return;                      // (whole warps; a block has one row)
@@ -143,11 +156,7 @@ stream_norm_kernel(float* __restrict__ residual, const T* __restrict__ delta, T*
     if (delta != nullptr) {
         float factor = n.delta_scale;
         if (n.post_kind != 0) {
-            if (WARP) {
-                load_vector<VEC>(post_w, n.post_weight, hidden, first, step);
-                load_vector<VEC>(post_b, n.post_bias, hidden, first, step);
-            }
-            norm_row<VEC, WARP>(y, hidden, first, step, n.post_kind, n.post_eps, post_w, post_b, scratch);
+            norm_row<VEC, WARP, HELD>(y, hidden, first, step, n.post_kind, n.post_eps, post, scratch);
             factor = 1.f;
         }
 #pragma unroll
@@ -158,11 +167,7 @@ stream_norm_kernel(float* __restrict__ residual, const T* __restrict__ delta, T*
                 store4<float>(residual + base + first + j * step, x[j]);
             }
     }
-    if (WARP) {
-        load_vector<VEC>(w, n.weight, hidden, first, step);
-        load_vector<VEC>(b, n.bias, hidden, first, step);
-    }
-    norm_row<VEC, WARP>(x, hidden, first, step, n.kind, n.eps, w, b, scratch + 64);
+    norm_row<VEC, WARP, HELD>(x, hidden, first, step, n.kind, n.eps, next, scratch + 64);
 #pragma unroll
     for (int j = 0; j < VEC; ++j)
         if (first + j * step < hidden) store4<T>(out + base + first + j * step, x[j]);
@@ -218,25 +223,25 @@ cudaError_t launch(float* residual, const void* delta, void* out, int rows, int 
                          aligned16(n.post_bias);
     const T* d = (const T*)delta;
     T* o = (T*)out;
-#define ROWS(VEC)                                                                                   \
-    launch_kernel(stream_norm_kernel<T, VEC, false>, dim3(rows), dim3(threads), 0, stream, true,    \
-                  residual, d, o, rows, hidden, n)
-#define WARPS(VEC)                                                                                  \
-    launch_kernel(stream_norm_kernel<T, VEC, true>, dim3((rows + 7) / 8), dim3(256), 0, stream,     \
+#define ROWS(VEC, HELD)                                                                             \
+    launch_kernel(stream_norm_kernel<T, VEC, false, HELD>, dim3(rows), dim3(threads), 0, stream,    \
                   true, residual, d, o, rows, hidden, n)
-    if (aligned && rows >= 1536 && hidden <= 1024) {
+#define WARPS(VEC)                                                                                  \
+    launch_kernel(stream_norm_kernel<T, VEC, true, false>, dim3((rows + 7) / 8), dim3(256), 0,      \
+                  stream, true, residual, d, o, rows, hidden, n)
+    if (aligned && rows >= 1536 && hidden <= 512) {
         if (hidden <= 256) return WARPS(2);
-        if (hidden <= 512) return WARPS(4);
-        return WARPS(8);
+        return WARPS(4);
     }
     if (aligned && hidden <= 8192) {
         // many rows: fewer threads a row and more rows at a time; few rows: as many threads as there are
         const int quads = hidden / 4;
-        const int each = rows >= 1024 ? 4 : (quads <= 1024 ? 1 : 2);
+        const bool many = rows >= 592 && quads > 64;
+        const int each = many && quads > 1024 ? 4 : many || quads > 1024 ? 2 : 1;
         const int threads = ((quads + each - 1) / each + 31) / 32 * 32;
-        if (each == 1) return ROWS(1);
-        if (each == 2) return ROWS(2);
-        return ROWS(4);
+        if (each == 1) return ROWS(1, true);
+        if (each == 2) return many ? ROWS(2, false) : ROWS(2, true);
+        return ROWS(4, false);
     }
 #undef ROWS
 #undef WARPS
