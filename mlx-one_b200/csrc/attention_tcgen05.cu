@@ -289,13 +289,44 @@ __device__ __forceinline__ void shape_tile(float (&v)[N], const ScoreShape& shap
     const unsigned long long fall = pair_of(-slope, -slope);
     unsigned long long away = pair_of(ahead, ahead - 1.f);
     const unsigned long long nearer = pair_of(-2.f, -2.f);
+    // the bias of eight keys: the first pair's worked out, the other three pairs' by an addition
+    const unsigned long long further[4] = {pair_of(0.f, 0.f), pair_of(2.f * slope, 2.f * slope),
+                                           pair_of(4.f * slope, 4.f * slope), pair_of(6.f * slope, 6.f * slope)};
+    const float steep = fabsf(shape.inner);
     if (shape.outer == 0.f) {
-        const unsigned long long plain = pair_of(shape.plain, shape.plain), none = pair_of(0.f, 0.f);
+        const unsigned long long plain = pair_of(shape.plain, shape.plain);
 #pragma unroll
-        for (int i = 0; i < N; i += 2) {
-            const unsigned long long bias = fma_pair(fall, away, none);
-            unpair(fma_pair(pair_of(v[i], v[i + 1]), plain, bias), v[i], v[i + 1]);
-            away = add_pair(away, nearer);
+        for (int i = 0; i < N; i += 8) {
+            const unsigned long long base = mul_pair(fall, pair_of(ahead - (float)i, ahead - (float)(i + 1)));
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                const unsigned long long bias = k == 0 ? base : add_pair(base, further[k]);
+                unpair(fma_pair(pair_of(v[i + 2 * k], v[i + 2 * k + 1]), plain, bias), v[i + 2 * k],
+                       v[i + 2 * k + 1]);
+            }
+        }
+    } else if (steep >= 1e-4f && !__any_sync(0xffffffffu, top * steep > 0.5f)) {
+        // outer tanh(inner v) = v Q(v^2): the factors in the coefficients (inner^7 is no smaller than
+        // 1e-28 here)
+        const float in1 = shape.inner * shape.outer, in2 = shape.inner * shape.inner;
+        const float in3 = in1 * in2, in5 = in3 * in2, in7 = in5 * in2;
+        const unsigned long long c0 = pair_of(in1 * MLXONE_TANH_HALF_C0, in1 * MLXONE_TANH_HALF_C0);
+        const unsigned long long c1 = pair_of(in3 * MLXONE_TANH_HALF_C1, in3 * MLXONE_TANH_HALF_C1);
+        const unsigned long long c2 = pair_of(in5 * MLXONE_TANH_HALF_C2, in5 * MLXONE_TANH_HALF_C2);
+        const unsigned long long c3 = pair_of(in7 * MLXONE_TANH_HALF_C3, in7 * MLXONE_TANH_HALF_C3);
+#pragma unroll
+        for (int i = 0; i < N; i += 8) {
+            const unsigned long long base = mul_pair(fall, pair_of(ahead - (float)i, ahead - (float)(i + 1)));
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                const unsigned long long s = pair_of(v[i + 2 * k], v[i + 2 * k + 1]);
+                const unsigned long long x = mul_pair(s, s);
+                unsigned long long p = fma_pair(x, c3, c2);
+                p = fma_pair(x, p, c1);
+                p = fma_pair(x, p, c0);
+                const unsigned long long bias = k == 0 ? base : add_pair(base, further[k]);
+                unpair(fma_pair(s, p, bias), v[i + 2 * k], v[i + 2 * k + 1]);
+            }
         }
     } else if (__any_sync(0xffffffffu, top * fabsf(shape.inner) > 1.f)) {
 #pragma unroll

@@ -54,6 +54,12 @@ __device__ __forceinline__ int shape_window(const ScoreShape& shape, int first_h
 #define MLXONE_TANH_C4 0.016743037849664688f
 #define MLXONE_TANH_C5 -0.0030670284759253263f
 
+// ... and for |t| <= 1/2, of degree 3 (5.5e-7)
+#define MLXONE_TANH_HALF_C0 0.999999463558197f
+#define MLXONE_TANH_HALF_C1 -0.33326318860054016f
+#define MLXONE_TANH_HALF_C2 0.13190296292304993f
+#define MLXONE_TANH_HALF_C3 -0.04440220445394516f
+
 __device__ __forceinline__ float tanh_small(float t) {
     const float x = t * t;
     float p = fmaf(x, MLXONE_TANH_C5, MLXONE_TANH_C4);
