@@ -86,7 +86,7 @@ Z3 = {"architecture": "Zinizen", "vocab": 64, "width": 36, "norm": {"eps": 1e-5}
 # rows of 64 values (prompts on the tcgen05 kernel), four query heads on a key head, parts of 64
 # channels, one value mixer that no later layer follows
 Z4 = {"architecture": "Zinizen", "vocab": 512, "width": 128, "norm": {"eps": 2e-6},
-      "embedding": bigram(1000, 31, 17),
+      "embedding": bigram(1000, 29, 11),
       "layers": [rglru(192, 3, 4, dense(192)),
                  attention(8, 2, 64, 48, 0.125, moe(8, 2, 64, 1.1, 2.0, (64, 0.6)), 30.0, (0.3, 32), True),
                  latent(5, 32, 32, 48, 128, 64, 0.15, dense(200), base=1000000.0),
