@@ -357,7 +357,7 @@ gated_recurrence_step_kernel(Operands o, const T* __restrict__ gates, int tokens
 
 int chunk_length(int tokens, int max_portion) {
     if (max_portion <= 32) return 32;
-    return tokens <= 1024 ? 16 : tokens <= 4096 ? 32 : 64;
+    return tokens <= 4096 ? 16 : 32;
 }
 
 template <typename T>

@@ -241,6 +241,7 @@ qk_prep_general_kernel(const T* __restrict__ qkv, const float* __restrict__ q_we
     float* sines = shared + rotary_dim / 2;
     griddep_launch();
     griddep_wait();
+    qkv = settled(qkv);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int slots_per_token = heads + 2 * kv_heads;
     const int t = blockIdx.x;

@@ -428,6 +428,22 @@ def test_gated_recurrence_alone(ops, dtype, width, blocks):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
+def test_gated_recurrence_over_a_long_prompt(ops, dtype):
+    """Thousands of tokens (longer chunks, many a channel) beside a short request, and the same in two
+    portions of which the second is long again."""
+    case = recurrence_case(16, 2, dtype, 1, lam=-5.0)
+    generator = torch.Generator().manual_seed(2)
+    inputs, gates_in = ([torch.randn(n, 16, generator=generator).to(dtype) for n in (4500, 40)] for _ in range(2))
+    want = [plain_recurrence(x, y, case) for x, y in zip(inputs, gates_in)]
+    for portions in (((5000,), (5000,)), ((201, 5000), (39, 1)), ((4300, 200), (40,))):
+        state = torch.zeros(2, 16, device=DEVICE)
+        got = run_recurrence(ops, case, inputs, gates_in, portions, state, [1, 0])
+        for r, b in enumerate(want):
+            error = (got[r] - b).abs().max() / max(1.0, float(b.abs().max()))
+            assert error < (2e-4 if dtype == torch.float32 else 0.03), f"request {r} portions {portions[r]}"
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
 def test_channels_that_keep_and_channels_that_forget(ops, dtype):
     """Decays within a millionth of 1 (where 1 - a^2 taken as a difference would be noise) and decays
     that underflow: what the third token brought still moves some channels 1100 tokens later, by
